@@ -8,6 +8,7 @@
 //                     S <- f * S (rows) + (1 - f) v^T;  o = S^T q
 //   retention_scan  linear attention with one fixed decay per head and no denominator:
 //                     S <- decay S + k v^T;  o = S^T q
+//   lightning_scan  the same recurrence on q = silu(.), k = silu(.), v = silu(.)
 //   head_norm_gate  out = o / rms(o) per head, times a weight (or none), times sigmoid(gate) or silu(gate)
 // What does not depend on the state (unit vectors, decays, gates) is computed for all rows at once by a preparing
 // kernel, in place. A scan block then takes one (head, request, run of value columns) and walks the request's rows of
@@ -242,6 +243,28 @@ __global__ void retention_prepare_kernel(float* __restrict__ proj, int ld, int q
       head[i + half] = (b * c + a * sn) * mul;
     } else if (which) {
       head[rot + (i - half)] *= mul;
+    }
+  }
+}
+
+// Per row, in place, of a 32-bit projection: `n` values from column col0 on become silu of themselves.
+template <int V>
+__global__ void __launch_bounds__(256)
+silu_columns_kernel(float* __restrict__ proj, int ld, int col0, int n, const int* __restrict__ seq_of_row, int n_rows) {
+  pdl_trigger();
+  pdl_wait();
+  const int per_row = n / V;
+  for (size_t e = (size_t)blockIdx.x * blockDim.x + threadIdx.x; e < (size_t)n_rows * per_row;
+       e += (size_t)gridDim.x * blockDim.x) {
+    const size_t row = e / per_row;
+    if (seq_of_row[row] < 0) continue;
+    float* at = proj + row * ld + col0 + (e % per_row) * V;
+    if (V == 4) {
+      float4 v = *reinterpret_cast<float4*>(at);
+      v.x *= sigmoidf_(v.x); v.y *= sigmoidf_(v.y); v.z *= sigmoidf_(v.z); v.w *= sigmoidf_(v.w);
+      *reinterpret_cast<float4*>(at) = v;
+    } else {
+      *at *= sigmoidf_(*at);
     }
   }
 }
@@ -717,6 +740,34 @@ CUCA_API int cuca_forget_scan(float* proj, int ld, int q_col, int f_col, int v_c
   return 0;
 }
 
+// S <- decay[h] S + k v^T, o = S^T q along every request's rows of a prepared 32-bit projection
+static int launch_decay_scan(const char* name, const float* proj, int ld, int q_col, int k_col, int v_col, const float* decay,
+                             float* state, float* out, const int* req_row0, const int* req_count, const int* slots,
+                             int n_seqs, int H, int d, int dv, cudaStream_t stream) {
+  int ns, nr;
+  CUCA_REQUIRE(split_rows(d, (long long)n_seqs * H * dv, &ns, &nr), "%s: %d key channels exceed %d", name, d, 32 * MAXR);
+  int pb = block_threads(ns, nr) / ns;
+  pb = pb > dv ? dv : pb;
+  const int threads = (pb * ns + 31) / 32 * 32;
+  const int per = (2 * ns * (nr == 4 ? 4 : nr + 4) + pb + 3) & ~3;
+  int tc = 46000 / (2 * per * 4);
+  tc = tc > 16 ? 16 : tc;
+  CUCA_REQUIRE(tc >= 1, "%s: a token of %d key channels does not fit shared memory", name, d);
+  const size_t smem = (size_t)2 * tc * per * 4;
+  const int wide = d % 4 == 0 && ld % 4 == 0 && q_col % 4 == 0 && k_col % 4 == 0 && ((uintptr_t)proj & 15) == 0;
+  dim3 grid(H, n_seqs, (dv + pb - 1) / pb);
+#define RS(NR)                                                                                                     \
+  cuca_launch(forget_scan_kernel<NR, true>, grid, dim3(threads), smem, stream, true, proj, ld, q_col,  \
+              k_col, v_col, decay, state, out, req_row0, req_count, slots, H, d, dv, ns, pb, tc, wide)
+  if (nr == 4) RS(4);
+  else if (nr == 8) RS(8);
+  else if (nr == 16) RS(16);
+  else RS(32);
+#undef RS
+  CUCA_CHECK_LAUNCH(name);
+  return 0;
+}
+
 // Retention along every request's rows. proj: 32-bit rows of stride ld holding q heads at q_col, k heads at k_col (H
 // heads of d each) and v heads at v_col (H heads of dv). The preparing kernel turns the first `rot` values of every q
 // and k head by the row's position (pairs (i, i + rot/2); cos_t/sin_t: [table_rows, rot/2]) and multiplies k by
@@ -731,8 +782,6 @@ CUCA_API int cuca_retention_scan(float* proj, int ld, int q_col, int k_col, int 
   CUCA_REQUIRE(H > 0 && d > 0 && dv > 0, "retention_scan: bad sizes heads=%d dim=%d vdim=%d", H, d, dv);
   CUCA_REQUIRE(rot >= 0 && rot <= d && rot % 2 == 0, "retention_scan: rotary size %d does not fit head size %d", rot, d);
   CUCA_REQUIRE(n_seqs <= 65535, "retention_scan: %d requests exceed the launch limit", n_seqs);
-  int ns, nr;
-  CUCA_REQUIRE(split_rows(d, (long long)n_seqs * H * dv, &ns, &nr), "retention_scan: %d key channels exceed %d", d, 32 * MAXR);
   {
     size_t blocks = ((size_t)n_rows * 2 * H * (d - rot / 2) + 255) / 256;
     blocks = blocks > 8192 ? 8192 : blocks;
@@ -740,26 +789,29 @@ CUCA_API int cuca_retention_scan(float* proj, int ld, int q_col, int k_col, int 
                 cos_t, sin_t, table_rows, rot, k_scale, positions, seq_of_row, n_rows, H, d, err);
     CUCA_CHECK_LAUNCH("retention_prepare");
   }
-  int pb = block_threads(ns, nr) / ns;
-  pb = pb > dv ? dv : pb;
-  const int threads = (pb * ns + 31) / 32 * 32;
-  const int per = (2 * ns * (nr == 4 ? 4 : nr + 4) + pb + 3) & ~3;
-  int tc = 46000 / (2 * per * 4);
-  tc = tc > 16 ? 16 : tc;
-  CUCA_REQUIRE(tc >= 1, "retention_scan: a token of %d key channels does not fit shared memory", d);
-  const size_t smem = (size_t)2 * tc * per * 4;
-  const int wide = d % 4 == 0 && ld % 4 == 0 && q_col % 4 == 0 && k_col % 4 == 0 && ((uintptr_t)proj & 15) == 0;
-  dim3 grid(H, n_seqs, (dv + pb - 1) / pb);
-#define RS(NR)                                                                                                     \
-  cuca_launch(forget_scan_kernel<NR, true>, grid, dim3(threads), smem, stream, true, (const float*)proj, ld, q_col,  \
-              k_col, v_col, decay, state, out, req_row0, req_count, slots, H, d, dv, ns, pb, tc, wide)
-  if (nr == 4) RS(4);
-  else if (nr == 8) RS(8);
-  else if (nr == 16) RS(16);
-  else RS(32);
-#undef RS
-  CUCA_CHECK_LAUNCH("retention_scan");
-  return 0;
+  return launch_decay_scan("retention_scan", proj, ld, q_col, k_col, v_col, decay, state, out, req_row0, req_count, slots,
+                           n_seqs, H, d, dv, stream);
+}
+
+// Lightning attention along every request's rows. proj as for retention; q, k and v (contiguous from col0 on: H heads of
+// d, H heads of d, H heads of dv) hold pre-activations and become silu of themselves in place; then retention's scan.
+CUCA_API int cuca_lightning_scan(float* proj, int ld, int col0, const float* decay, float* state, float* out,
+                                 const int* seq_of_row, const int* req_row0, const int* req_count, const int* slots,
+                                 int n_rows, int n_seqs, int H, int d, int dv, cudaStream_t stream) {
+  if (n_seqs == 0 || n_rows == 0) return 0;
+  CUCA_REQUIRE(H > 0 && d > 0 && dv > 0, "lightning_scan: bad sizes heads=%d dim=%d vdim=%d", H, d, dv);
+  CUCA_REQUIRE(n_seqs <= 65535, "lightning_scan: %d requests exceed the launch limit", n_seqs);
+  const int n = H * (2 * d + dv);
+  const bool wide = n % 4 == 0 && ld % 4 == 0 && col0 % 4 == 0 && ((uintptr_t)proj & 15) == 0;
+  size_t blocks = ((size_t)n_rows * n / (wide ? 4 : 1) + 255) / 256;
+  blocks = blocks > 8192 ? 8192 : blocks;
+  if (wide)
+    cuca_launch(silu_columns_kernel<4>, dim3((unsigned)blocks), dim3(256), 0, stream, true, proj, ld, col0, n, seq_of_row, n_rows);
+  else
+    cuca_launch(silu_columns_kernel<1>, dim3((unsigned)blocks), dim3(256), 0, stream, true, proj, ld, col0, n, seq_of_row, n_rows);
+  CUCA_CHECK_LAUNCH("silu_columns");
+  return launch_decay_scan("lightning_scan", proj, ld, col0, col0 + H * d, col0 + 2 * H * d, decay, state, out, req_row0,
+                           req_count, slots, n_seqs, H, d, dv, stream);
 }
 
 // gate_act 0: the gate's factor is sigmoid(gate); 1: silu(gate). w null: no weight.

@@ -7,8 +7,13 @@
 //   moe_route_scored scores are a softmax over ALL router outputs; the choice goes by score + a correction per output,
 //                    the weights are the chosen scores over their sum; the last outputs may stand for experts that
 //                    return their input (their weights are summed per token for `moe_identity_add`)
+//   moe_route_grouped  scores are sigmoids; experts form equal groups of neighbours, only those of the best groups (by
+//                    the sum of a group's two largest scores) can be chosen; the weights are the chosen scores times a
+//                    constant. A shared expert rides along as one more entry, weighted by the sigmoid of its own logit
 //   moe_glu_dense    a[t, c] = silu(g[t, c]) u[t, c] * weight[t, expert of c]: gated experts, and behind them the
 //                    columns of a shared expert that every token uses with weight 1
+//   moe_glu_capped_dense  the same for capped gated units (see `capped_unit`); the shared columns have a cap and a
+//                    weight per token of their own
 // Routing arithmetic is 32-bit. A token's experts are summed in a fixed order, whatever else is in the batch.
 #include "common.cuh"
 #include <math.h>
@@ -138,6 +143,141 @@ moe_route_scored_kernel(const float* __restrict__ logits, const float* __restric
   if (ident && lane == 0) ident[t] = iw;
 }
 
+// The capped gated unit: g = min(gate, limit), u = clamp(up, -limit, limit), g sigmoid(alpha g) (u + 1).
+__device__ __forceinline__ float capped_unit(float gate, float up, float limit, float alpha) {
+  const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+  return g / (1.f + expf(-alpha * g)) * (u + 1.f);
+}
+
+// Scores s = sigmoid(z) of E experts in `groups` equal groups of neighbours. A group's score is the sum of its two
+// largest (of its one, where it has one); the `keep` best groups' experts can be chosen, the `top` largest of them are
+// (the lower number on a tie), with weights s * scale. Column E of a row of logits, where has_shared, belongs to a shared
+// expert that every token uses, with weight sigmoid(z): it becomes entry `top` of idx / wts (number E) and column E of
+// dense. A warp per token; lane l holds experts l, l + 32, ...
+__global__ void __launch_bounds__(128)
+moe_route_grouped_kernel(const float* __restrict__ logits, int T, int E, int groups, int keep, int top, float scale,
+                         int has_shared, int* __restrict__ idx, float* __restrict__ wts, float* __restrict__ dense) {
+  __shared__ float group_score[4][MAX_EXPERTS];
+  pdl_trigger();
+  pdl_wait();
+  const int warp = threadIdx.x >> 5, t = blockIdx.x * 4 + warp, lane = threadIdx.x & 31;
+  if (t >= T) return;
+  const int n_out = E + (has_shared ? 1 : 0), entries = top + (has_shared ? 1 : 0);
+  const float* z = logits + (size_t)t * n_out;
+  auto score = [&](int e) {  // (a row of padding may hold anything: every lane must still see one order)
+    const float v = z[e];
+    return v == v ? 1.f / (1.f + expf(-v)) : -1.f;
+  };
+  unsigned open = 0xffffffffu;  // bit k: this lane's expert lane + 32 k can be chosen
+  if (groups > 1 && keep < groups) {
+    const int size = E / groups;
+    float* gs = group_score[warp];
+    if (size <= 32) {  // a lane per group
+      for (int g = lane; g < groups; g += 32) {
+        float a = -INFINITY, b = -INFINITY;
+        for (int i = 0; i < size; ++i) {
+          const float v = score(g * size + i);
+          if (v > a) { b = a; a = v; } else if (v > b) b = v;
+        }
+        gs[g] = size > 1 ? a + b : a;
+      }
+    } else {  // few large groups: the warp's lanes share each
+      for (int g = 0; g < groups; ++g) {
+        float a = -INFINITY, b = -INFINITY;
+        for (int i = lane; i < size; i += 32) {
+          const float v = score(g * size + i);
+          if (v > a) { b = a; a = v; } else if (v > b) b = v;
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+          const float oa = __shfl_xor_sync(0xffffffffu, a, o), ob = __shfl_xor_sync(0xffffffffu, b, o);
+          const float hi = fmaxf(a, oa), lo = fminf(a, oa);
+          b = fmaxf(lo, fmaxf(b, ob));
+          a = hi;
+        }
+        if (lane == 0) gs[g] = a + b;
+      }
+    }
+    __syncwarp();
+    open = 0;
+    for (int k = 0; lane + 32 * k < E; ++k) {  // an expert is open if fewer than `keep` groups come before its own
+      const int g = (lane + 32 * k) / size;
+      const float mine = gs[g];
+      int before = 0;
+      for (int i = 0; i < groups; ++i) before += (gs[i] > mine || (gs[i] == mine && i < g)) ? 1 : 0;
+      if (before < keep) open |= 1u << k;
+    }
+  }
+  float my_s = 0.f;
+  int my_e = 0;
+  for (int j = 0; j < top; ++j) {
+    float best = -INFINITY;
+    int be = 0x7fffffff;
+    for (int k = 0; lane + 32 * k < E; ++k) {
+      if (!((open >> k) & 1u)) continue;
+      const int e = lane + 32 * k;
+      const float v = score(e);
+      if (v > best || be == 0x7fffffff) { best = v; be = e; }  // (ascending numbers: the first of equals stays)
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+      const int oe = __shfl_xor_sync(0xffffffffu, be, o);
+      if (oe != 0x7fffffff && (be == 0x7fffffff || ov > best || (ov == best && oe < be))) { best = ov; be = oe; }
+    }
+    if (be < E && (be & 31) == lane) open &= ~(1u << (be >> 5));
+    if (lane == j) { my_s = best; my_e = be < E ? be : 0; }
+  }
+  const float w = my_s * scale;
+  if (dense)
+    for (int e = lane; e < n_out; e += 32) dense[(size_t)t * n_out + e] = 0.f;
+  __syncwarp();
+  if (lane < top) {
+    idx[(size_t)t * entries + lane] = my_e;
+    wts[(size_t)t * entries + lane] = w;
+    if (dense) dense[(size_t)t * n_out + my_e] = w;
+  }
+  if (has_shared && lane == 0) {
+    const float sw = 1.f / (1.f + expf(-z[E]));
+    idx[(size_t)t * entries + top] = E;
+    wts[(size_t)t * entries + top] = sw;
+    if (dense) dense[(size_t)t * n_out + E] = sw;
+  }
+}
+
+// gu: [T, 2 C] (gates, then ups); a[t, c] = capped_unit(g, u) w; c < EF: expert c / F's columns, w = dense[t, c / F] and
+// cap `limit`; behind: the shared expert's, w = dense[t, EF / F] and cap `limit_s`. V values a thread (16 bytes), or 1.
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+moe_glu_capped_dense_kernel(const T* __restrict__ gu, const float* __restrict__ dense, int ld_dense, T* __restrict__ a,
+                            size_t n_vec, int C, int EF, int F, float limit, float limit_s, float alpha) {
+  pdl_trigger();
+  pdl_wait();
+  const int cv = C / V;
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n_vec; i += (size_t)gridDim.x * blockDim.x) {
+    const size_t t = i / cv;
+    const int c = (int)(i % cv) * V;
+    const bool shared = c >= EF;
+    const float w = dense[t * ld_dense + (shared ? EF / F : c / F)];
+    const float lim = shared ? limit_s : limit;
+    const T* gp = gu + t * 2 * C + c;
+    if (V == 1) {
+      a[t * C + c] = from_f32<T>(w == 0.f ? 0.f : capped_unit(to_f32(gp[0]), to_f32(gp[C]), lim, alpha) * w);
+      continue;
+    }
+    uint4 out4 = make_uint4(0u, 0u, 0u, 0u);
+    if (w != 0.f) {  // (an expert the token did not choose: its rows are not read)
+      const uint4 g4 = *reinterpret_cast<const uint4*>(gp), u4 = *reinterpret_cast<const uint4*>(gp + C);
+      const T* g = reinterpret_cast<const T*>(&g4);
+      const T* u = reinterpret_cast<const T*>(&u4);
+      T* o = reinterpret_cast<T*>(&out4);
+#pragma unroll
+      for (int e = 0; e < V; ++e) o[e] = from_f32<T>(capped_unit(to_f32(g[e]), to_f32(u[e]), lim, alpha) * w);
+    }
+    *reinterpret_cast<uint4*>(a + t * C + c) = out4;
+  }
+}
+
 // gu: [T, 2 C] (gates, then ups); a[t, c] = silu(g) u w with w = dense[t, c / F] for c < EF (ld_dense outputs a row),
 // 1 for the columns behind (a shared expert).
 template <typename T>
@@ -231,49 +371,55 @@ __device__ __forceinline__ float warp_dot(const __nv_bfloat16* w, const __nv_bfl
   return warp_sum(acc);
 }
 
-// a[pair, f] = act(W[e(pair)] . h[t]) * weight(pair); pair = t * top + j. GLU false: W_up [E F, K], act = relu(.)^2.
-// GLU true: w_up holds every expert's gate rows and, `up_rows` rows further on, its up rows; act = silu(gate) up.
-// A pair whose expert number is n_real or more has no weights (it returns its input): nothing is written for it.
-template <typename T, bool GLU>
+// What a sparse launch's experts compute. ACT 0: relu(up)^2; 1: silu(gate) up; 2: `capped_unit`.
+struct SparseUnit {
+  float limit, limit_s, alpha;  // ACT 2: the caps of the experts and of the shared expert
+};
+
+// a[pair, f] = act(W[e(pair)] . h[t]) * weight(pair); pair = t * entries + j. ACT 0: W_up [E F, K]. ACT 1 and 2: w_up
+// holds every expert's gate rows and, `up_rows` rows further on, its up rows. Entry number n_real is the shared expert
+// where Fs > 0: its Fs rows follow the experts'. Any other number from n_real on has no weights (such an expert
+// returns its input): nothing is written for it. Rows of a are lda values.
+template <typename T, int ACT>
 __global__ void __launch_bounds__(256)
 moe_up_sparse_kernel(const T* __restrict__ h, const T* __restrict__ w_up, const int* __restrict__ idx,
-                     const float* __restrict__ wts, T* __restrict__ a, int top, int F, int K, int n_real, size_t up_rows) {
+                     const float* __restrict__ wts, T* __restrict__ a, int lda, int entries, int F, int Fs, int K,
+                     int n_real, size_t up_rows, const SparseUnit unit) {
   pdl_trigger();
   pdl_wait();
   const int pair = blockIdx.y, f = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (f >= F) return;
   const int e = idx[pair];
-  if (e >= n_real) return;
+  if (f >= (e < n_real ? F : (e == n_real ? Fs : 0))) return;
   const T* wr = w_up + ((size_t)e * F + f) * K;
-  const T* hr = h + (size_t)(pair / top) * K;
-  const float acc = warp_dot(wr, hr, K, lane);
+  const T* hr = h + (size_t)(pair / entries) * K;
   float v;
-  if (GLU) {
-    const float u = warp_dot(wr + up_rows * K, hr, K, lane);
-    v = acc / (1.f + expf(-acc)) * u;
-  } else {
-    v = fmaxf(acc, 0.f);
+  if (ACT == 0) {
+    v = fmaxf(warp_dot(wr, hr, K, lane), 0.f);
     v = v * v;
+  } else {
+    const float g = warp_dot(wr, hr, K, lane), u = warp_dot(wr + up_rows * K, hr, K, lane);
+    v = ACT == 1 ? g / (1.f + expf(-g)) * u : capped_unit(g, u, e == n_real ? unit.limit_s : unit.limit, unit.alpha);
   }
-  if (lane == 0) a[(size_t)pair * F + f] = from_f32<T>(v * wts[pair]);
+  if (lane == 0) a[(size_t)pair * lda + f] = from_f32<T>(v * wts[pair]);
 }
 
-// y[t, o] (+)= sum_j W_down[o, e(t, j) F ..] . a[t * top + j]; W_down: [N, ld] (ld columns a row)
+// y[t, o] (+)= sum_j W_down[o, e(t, j) F ..] . a[t * entries + j]; W_down: [N, ld] (ld columns a row)
 template <typename T>
 __global__ void __launch_bounds__(256)
-moe_down_sparse_kernel(const T* __restrict__ a, const T* __restrict__ w_down, const int* __restrict__ idx,
-                       float* __restrict__ y, int store, int top, int F, int ld, int N, int n_real) {
+moe_down_sparse_kernel(const T* __restrict__ a, int lda, const T* __restrict__ w_down, const int* __restrict__ idx,
+                       float* __restrict__ y, int store, int entries, int F, int Fs, int ld, int N, int n_real) {
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.y, o = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (o >= N) return;
   float acc = 0.f;
-  for (int j = 0; j < top; ++j) {
-    const int e = idx[(size_t)t * top + j];
-    if (e >= n_real) continue;
+  for (int j = 0; j < entries; ++j) {
+    const int e = idx[(size_t)t * entries + j];
+    const int n = e < n_real ? F : (e == n_real ? Fs : 0);
+    if (n == 0) continue;
     const T* wr = w_down + (size_t)o * ld + (size_t)e * F;
-    const T* ar = a + ((size_t)t * top + j) * F;
-    acc += warp_dot(wr, ar, F, lane);
+    const T* ar = a + ((size_t)t * entries + j) * lda;
+    acc += warp_dot(wr, ar, n, lane);
   }
   if (lane == 0) y[(size_t)t * N + o] = store ? acc : y[(size_t)t * N + o] + acc;
 }
@@ -311,33 +457,84 @@ CUCA_API int cuca_moe_act_dense(const void* u, const float* dense, void* a, int 
   return 0;
 }
 
-// glu 0: relu(up)^2 experts, w_up [E F, K], w_down [N, E F]. glu 1: gated experts, w_up [2 C, K] (every expert's gate
-// rows, then C rows on every expert's up rows), w_down [N, C]; C >= E F (what lies behind belongs to a shared expert,
-// which this launch leaves alone). Pairs that name expert E or more are skipped.
-CUCA_API int cuca_moe_sparse(const void* h, const void* w_up, const void* w_down, const int* idx, const float* wts,
-                             void* a, float* y, int store, int dtype, int T, int top, int E, int F, int K, int N,
-                             int glu, int C, cudaStream_t stream) {
+// act 0: relu(up)^2 experts, w_up [E F, K], w_down [N, E F]. act 1 (silu-gated) and 2 (capped units): w_up [2 C, K] (every
+// expert's gate rows, then C rows on every expert's up rows), w_down [N, C]; C >= E F. `entries` idx / wts a token. Fs > 0:
+// number E is a shared expert of Fs rows behind the experts' (with cap limit_s); numbers beyond (with Fs = 0: from E
+// on) are skipped. a: [T * entries, lda], lda >= max(F, Fs).
+CUCA_API int cuca_moe_sparse_act(const void* h, const void* w_up, const void* w_down, const int* idx, const float* wts,
+                                 void* a, int lda, float* y, int store, int dtype, int T, int entries, int E, int F,
+                                 int Fs, int K, int N, int act, int C, float limit, float limit_s, float alpha,
+                                 cudaStream_t stream) {
   if (T == 0) return 0;
-  CUCA_REQUIRE(T * top <= 65535 && T <= 65535, "moe_sparse: %d tokens exceed the launch limit", T);
-  const int ld = glu ? C : E * F;
-  CUCA_REQUIRE(ld >= E * F, "moe_sparse: %d columns do not hold %d experts of %d", ld, E, F);
+  CUCA_REQUIRE(T * entries <= 65535 && T <= 65535, "moe_sparse: %d tokens exceed the launch limit", T);
+  const int ld = act ? C : E * F, wide = F > Fs ? F : Fs;
+  CUCA_REQUIRE(ld >= E * F + Fs, "moe_sparse: %d columns do not hold %d experts of %d and a shared one of %d", ld, E, F, Fs);
+  CUCA_REQUIRE(lda >= wide, "moe_sparse: rows of %d values do not hold %d", lda, wide);
+  CUCA_REQUIRE(act >= 0 && act <= 2, "moe_sparse: unknown activation %d", act);
+  const SparseUnit unit = {limit, limit_s, alpha};
+#define UP(TT, ACT)                                                                                                 \
+  cuca_launch(moe_up_sparse_kernel<TT, ACT>, dim3((wide + 7) / 8, T * entries), dim3(256), 0, stream, true,         \
+              (const TT*)h, (const TT*)w_up, idx, wts, (TT*)a, lda, entries, F, Fs, K, E, (size_t)C, unit)
 #define SPARSE(TT)                                                                                                  \
   do {                                                                                                              \
-    if (glu)                                                                                                        \
-      cuca_launch(moe_up_sparse_kernel<TT, true>, dim3((F + 7) / 8, T * top), dim3(256), 0, stream, true,           \
-                  (const TT*)h, (const TT*)w_up, idx, wts, (TT*)a, top, F, K, E, (size_t)C);                        \
-    else                                                                                                            \
-      cuca_launch(moe_up_sparse_kernel<TT, false>, dim3((F + 7) / 8, T * top), dim3(256), 0, stream, true,          \
-                  (const TT*)h, (const TT*)w_up, idx, wts, (TT*)a, top, F, K, E, (size_t)0);                        \
+    if (act == 0) UP(TT, 0);                                                                                        \
+    else if (act == 1) UP(TT, 1);                                                                                   \
+    else UP(TT, 2);                                                                                                 \
     CUCA_CHECK_LAUNCH("moe_up_sparse");                                                                             \
-    cuca_launch(moe_down_sparse_kernel<TT>, dim3((N + 7) / 8, T), dim3(256), 0, stream, true, (const TT*)a,         \
-                (const TT*)w_down, idx, y, store, top, F, ld, N, E);                                                \
+    cuca_launch(moe_down_sparse_kernel<TT>, dim3((N + 7) / 8, T), dim3(256), 0, stream, true, (const TT*)a, lda,    \
+                (const TT*)w_down, idx, y, store, entries, F, Fs, ld, N, E);                                        \
   } while (0)
   if (dtype == CUCA_F32) SPARSE(float);
   else if (dtype == CUCA_BF16) SPARSE(__nv_bfloat16);
   else CUCA_REQUIRE(false, "moe_sparse: unknown dtype %d", dtype);
 #undef SPARSE
+#undef UP
   CUCA_CHECK_LAUNCH("moe_down_sparse");
+  return 0;
+}
+
+// The same without a shared expert: glu 0: relu(up)^2 experts, 1: silu-gated ones.
+CUCA_API int cuca_moe_sparse(const void* h, const void* w_up, const void* w_down, const int* idx, const float* wts,
+                             void* a, float* y, int store, int dtype, int T, int top, int E, int F, int K, int N,
+                             int glu, int C, cudaStream_t stream) {
+  return cuca_moe_sparse_act(h, w_up, w_down, idx, wts, a, F, y, store, dtype, T, top, E, F, 0, K, N, glu ? 1 : 0, C, 0.f,
+                             0.f, 0.f, stream);
+}
+
+// logits: [T, E + 1] with has_shared (the last column the shared expert's), else [T, E]; idx, wts: [T, top + 1] or
+// [T, top]; dense (or null): as wide as the logits.
+CUCA_API int cuca_moe_route_grouped(const float* logits, int T, int E, int groups, int keep, int top, float scale,
+                                    int has_shared, int* idx, float* wts, float* dense, cudaStream_t stream) {
+  if (T == 0) return 0;
+  CUCA_REQUIRE(E >= 1 && E <= MAX_EXPERTS && top >= 1 && top <= MAX_TOP,
+               "moe_route: %d of %d experts is outside what the kernel takes (experts <= %d, chosen <= %d)", top, E,
+               MAX_EXPERTS, MAX_TOP);
+  CUCA_REQUIRE(groups >= 1 && E % groups == 0 && keep >= 1 && keep <= groups && top <= keep * (E / groups),
+               "moe_route: %d of the %d experts in %d of %d groups cannot be chosen", top, E, keep, groups);
+  cuca_launch(moe_route_grouped_kernel, dim3((T + 3) / 4), dim3(128), 0, stream, true, logits, T, E, groups, keep, top,
+              scale, has_shared, idx, wts, dense);
+  CUCA_CHECK_LAUNCH("moe_route_grouped");
+  return 0;
+}
+
+CUCA_API int cuca_moe_glu_capped_dense(const void* gu, const float* dense, int ld_dense, void* a, int dtype, int T, int C,
+                                       int EF, int F, float limit, float limit_s, float alpha, cudaStream_t stream) {
+  if (T == 0) return 0;
+  CUCA_REQUIRE(F >= 1 && EF % F == 0 && EF <= C && EF / F + (C > EF ? 1 : 0) <= ld_dense,
+               "moe_glu_capped_dense: bad sizes C=%d EF=%d F=%d", C, EF, F);
+  const int V = dtype == CUCA_BF16 ? 8 : 4;
+  const bool vec = F % V == 0 && C % V == 0 && ((uintptr_t)gu & 15) == 0 && ((uintptr_t)a & 15) == 0;
+  const size_t work = (size_t)T * C / (vec ? V : 1);
+  size_t blocks = (work + 255) / 256;
+  blocks = blocks > 16384 ? 16384 : blocks;
+#define CD(TT, VV)                                                                                                     \
+  cuca_launch(moe_glu_capped_dense_kernel<TT, VV>, dim3((unsigned)blocks), dim3(256), 0, stream, true, (const TT*)gu,  \
+              dense, ld_dense, (TT*)a, work, C, EF, F, limit, limit_s, alpha)
+  if (dtype == CUCA_F32) { if (vec) CD(float, 4); else CD(float, 1); }
+  else if (dtype == CUCA_BF16) { if (vec) CD(__nv_bfloat16, 8); else CD(__nv_bfloat16, 1); }
+  else CUCA_REQUIRE(false, "moe_glu_capped_dense: unknown dtype %d", dtype);
+#undef CD
+  CUCA_CHECK_LAUNCH("moe_glu_capped_dense");
   return 0;
 }
 

@@ -1044,6 +1044,25 @@ def retention_scan(proj, q_col, k_col, v_col, decay, cos, sin, rot_dims, k_scale
     library.launches += 1
 
 
+def lightning_scan(proj, decay, state, out, step, H, d, dv) -> None:
+    """Lightning attention along every request's rows: the recurrence of retention on silu(q), silu(k), silu(v) (see
+    `parts/recurrent.py:Lightning`). The first H (2 d + dv) columns of the 32-bit `proj` hold q, k, v before their
+    activation and are rewritten in place; two launches."""
+    _cuda(proj, decay, state, out)
+    library.check(library.load().cuca_lightning_scan(
+        _p(proj), proj.stride(0), 0, _p(decay), _p(state), _p(out), _p(step.seq_of_row), _p(step.req_row0),
+        _p(step.req_count), _p(step.slots), proj.shape[0], step.n_seqs, H, d, dv, _stream()), "lightning_scan")
+    library.launches += 1
+
+
+def row_norm_gate(o, weight, gate, out, eps: float) -> None:
+    """out[r] = o[r] / rms(o[r]) * weight * sigmoid(gate[r]) over whole rows; gate: 32-bit rows of any stride."""
+    _cuda(o, weight, gate, out)
+    library.check(library.load().cuca_row_norm_gate(_p(o), _p(weight), _p(gate), gate.stride(0), _p(out),
+                                                    dtype_code(out.dtype), o.shape[0], o.shape[1], float(eps), _stream()),
+                  "row_norm_gate")
+
+
 def head_norm_gate(o, weight, per_head: bool, gate, out, H, dv, eps, gate_act: str = "sigmoid") -> None:
     """out[r, h] = o[r, h] / rms(o[r, h]) * weight * act(gate[r, h]); weight [dv] for every head or [H dv], or None;
     act the sigmoid or, `gate_act` "silu", g sigmoid(g)."""
@@ -1105,3 +1124,95 @@ def moe_identity_add(y, h, ident, store: bool) -> None:
     _cuda(y, h, ident)
     library.check(library.load().cuca_moe_identity_add(_p(y), _p(h), dtype_code(h.dtype), _p(ident), int(bool(store)),
                                                        h.shape[0], h.shape[1], _stream()), "moe_identity_add")
+
+
+def moe_route_grouped(logits, experts: int, groups: int, keep: int, top: int, scale: float, shared: bool, idx, wts,
+                      dense=None) -> None:
+    """Scores sigmoid(logits); of `groups` equal groups of neighbouring experts the `keep` with the largest sums of their
+    two largest scores are open, the `top` largest scores among those are chosen, weights score * scale. `shared`: the
+    logits' last column is a shared expert's; it becomes the last entry (number `experts`) with weight sigmoid."""
+    _cuda(logits, idx, wts, dense)
+    library.check(library.load().cuca_moe_route_grouped(
+        _p(logits), logits.shape[0], int(experts), int(groups), int(keep), int(top), float(scale), int(bool(shared)),
+        _p(idx), _p(wts), _p(dense), _stream()), "moe_route_grouped")
+
+
+def moe_sparse_capped(h, w_gu, w_down, idx, wts, a, y, store, E: int, F: int, Fs: int, limit: float, limit_s: float,
+                      alpha: float) -> None:
+    """`moe_sparse` for experts that are capped gated units (`glu_capped`): `w_gu` [2 C, K] all gates then all ups,
+    `w_down` [N, C], C = E F + Fs. Entry number E is the shared expert of Fs rows with cap `limit_s`."""
+    _cuda(h, w_gu, w_down, idx, wts, a, y)
+    library.check(library.load().cuca_moe_sparse_act(
+        _p(h), _p(w_gu), _p(w_down), _p(idx), _p(wts), _p(a), a.stride(0), _p(y), int(bool(store)), dtype_code(h.dtype),
+        h.shape[0], idx.shape[1], E, F, Fs, h.shape[1], y.shape[1], 2, w_down.shape[1], float(limit), float(limit_s),
+        float(alpha), _stream()), "moe_sparse")
+    library.launches += 1
+
+
+def moe_glu_capped_dense(gu, dense, a, EF: int, F: int, limit: float, limit_s: float, alpha: float) -> None:
+    """a[t, c] = capped unit of (gu[t, c], gu[t, C + c]) * w: c < EF: w = dense[t, c // F] and cap `limit`; behind (a
+    shared expert): w = dense[t, EF // F] and cap `limit_s`."""
+    _cuda(gu, dense, a)
+    library.check(library.load().cuca_moe_glu_capped_dense(
+        _p(gu), _p(dense), dense.shape[1], _p(a), dtype_code(gu.dtype), gu.shape[0], a.shape[1], int(EF), int(F),
+        float(limit), float(limit_s), float(alpha), _stream()), "moe_glu_capped_dense")
+
+
+# ------------------------------------------------------------------ a sublayer's output on its way to the stream
+MAX_TERMS = 8  # `cuca_max_terms` says the same
+
+
+class _Terms(ctypes.Structure):
+    """The kernels' description of a weighted sum of terms (`csrc/sublayer_output.cu:CucaTerms`)."""
+
+    _fields_ = [("n", ctypes.c_int), ("data", ctypes.c_void_p * MAX_TERMS), ("slices", ctypes.c_int * MAX_TERMS),
+                ("stride", ctypes.c_size_t * MAX_TERMS), ("scale", ctypes.c_float * MAX_TERMS)]
+
+
+def _terms(terms) -> _Terms:
+    """`terms`: (32-bit tensor [rows, E] or `PartialSums`, factor) pairs."""
+    t = _Terms()
+    if len(terms) > MAX_TERMS:
+        raise library.KernelError(f"{len(terms)} terms exceed {MAX_TERMS}")
+    t.n = len(terms)
+    for i, (x, scale) in enumerate(terms):
+        if isinstance(x, PartialSums):
+            t.data[i], t.slices[i], t.stride[i] = x.data.data_ptr(), x.slices, x.slice_stride
+        else:
+            if x.dtype != torch.float32 or not x.is_contiguous():
+                raise library.KernelError("a term is a contiguous 32-bit tensor or a contraction's K slices")
+            t.data[i], t.slices[i], t.stride[i] = x.data_ptr(), 1, 0
+        t.scale[i] = float(scale)
+    return t
+
+
+def norm_add(x, terms, weight, eps: float, out=None, center: bool = True) -> None:
+    """x += N(y) * weight with y the weighted sum of `terms`; `out` (or None) = the new x in out's dtype. N is the
+    layer norm, or the RMS norm with `center` False."""
+    _cuda(x, weight, out)
+    t = _terms(terms)
+    library.check(library.load().cuca_norm_add(_p(x), ctypes.addressof(t), _p(weight), _p(out),
+                                               dtype_code(out.dtype) if out is not None else 0, x.shape[0], x.shape[1],
+                                               float(eps), int(bool(center)), _stream()), "norm_add")
+
+
+def layer_norm(x, weight, out, eps: float, rows=None) -> None:
+    """out[r] = (x - mean) / sqrt(mean((x - mean)^2) + eps) * weight of row r (or rows[r]) of x."""
+    _cuda(x, weight, out, rows)
+    library.check(library.load().cuca_layer_norm(_p(x), _p(weight), _p(out), dtype_code(out.dtype), _p(rows), out.shape[0],
+                                                 x.shape[1], float(eps), _stream()), "layer_norm")
+
+
+def add_terms(x, terms, store: bool) -> None:
+    """x (+)= the weighted sum of `terms`."""
+    _cuda(x)
+    t = _terms(terms)
+    library.check(library.load().cuca_add_terms(_p(x), ctypes.addressof(t), int(bool(store)), x.numel(), _stream()),
+                  "add_terms")
+
+
+def round_rows(x, out) -> None:
+    """out = x in out's dtype."""
+    _cuda(x, out)
+    library.check(library.load().cuca_round_rows(_p(x), _p(out), dtype_code(out.dtype), x.numel(), _stream()),
+                  "round_rows")

@@ -3,11 +3,12 @@
 `sandwich_shift`: a norm before and after each sublayer, and the mixer reads its input mixed with the previous
 token's: x += n1b(mixer(shift(n1(x)))); x += n2b(ffn(n2(x))).
 `hyper_connections`: several copies of the stream; a sublayer reads a weighted sum of them and writes into all.
-`parallel_residual`: one norm, both sublayers read its output: x += mixer(h) + ffn(h) with h = norm(x)."""
+`parallel_residual`: one norm, both sublayers read its output: x += mixer(h) + ffn(h) with h = norm(x).
+`post_norm`: the sublayers read the stream as it is, their outputs are normed: x += norm(mixer(x)); x += norm(ffn(x))."""
 from __future__ import annotations
 
 from ..kernels import ops
-from ..runtime import ResidualStream
+from ..runtime import ResidualStream, SublayerOutput
 from .base import Block, CacheNeeds, StateNeeds, TensorNeed, register_block
 
 
@@ -31,6 +32,27 @@ class ParallelResidualBlock(Block):
         self.mixer.forward(h, stream, step, cache)
         if self.feed_forward is not None:
             self.feed_forward.forward(h, stream, step)
+
+
+@register_block("post_norm")
+class PostNormBlock(Block):
+    """x += mixer_norm(mixer(x)); x += ffn_norm(ffn(x)): the norms stand on the sublayers' outputs only. A sublayer reads
+    the stream rounded to the compute dtype and its output is gathered as terms (`SublayerOutput`); one kernel then adds
+    the terms up (a contraction's K slices over few tokens among them), norms, adds into the stream and leaves the
+    rounded stream for the next sublayer.
+
+    params: width."""
+
+    def forward(self, stream, step, cache) -> None:
+        rt, width = self.rt, int(self.spec.params["width"])
+        stream = rt.stream(stream)
+        y = SublayerOutput(rt, step.n_rows, width)
+        self.mixer.forward(stream.rounded(), y, step, cache)
+        stream.add_normed(y, self.mixer_norm)
+        if self.feed_forward is not None:
+            y = SublayerOutput(rt, step.n_rows, width)
+            self.feed_forward.forward(stream.rounded(), y, step)
+            stream.add_normed(y, self.ffn_norm)
 
 
 @register_block("sandwich_shift")

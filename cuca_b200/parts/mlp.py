@@ -355,3 +355,102 @@ class ScoredExperts(FeedForward):
         a = rt.empty(T, self.w_down.shape[1])
         ops.moe_glu_dense(gu, spread, a, self.experts * self.inner, self.inner)
         stream.add_linear(a, self.w_down)
+
+
+@register_feed_forward("routed_grouped")
+class GroupedExperts(FeedForward):
+    """Routed experts with sigmoid scores s = sigmoid(W_r f) (32-bit) and a choice restricted to groups: the experts
+    form `groups` equal groups of neighbours, a group's score is the sum of its two largest scores, and the `top`
+    largest scores among the experts of the `keep` best groups are chosen. Their weights are s * scale, not
+    renormalised. The experts are capped gated units (see `glu_capped`, cap `limit`, slope `alpha`). With `shared` > 0
+    one more such unit of that inner size (cap `shared_limit`) runs for every token, weighted by sigmoid(w_s . f).
+
+    The router's rows and the shared expert's weight row are one contraction. The experts' weights are stacked at load as
+    the scored experts' are: `w_gu` [2 C, width] (every expert's gate rows, the shared expert's behind them, then the up
+    rows in the same order; C = experts * inner + shared), `w_down` [width, C]. Many tokens: one contraction gives all
+    gates and ups, the units are weighted per expert (0 for the ones a token did not choose), one contraction over C
+    goes down. Few tokens: only the chosen experts' rows and the shared one's are read, a warp per output: the shared
+    expert is one more entry of a token's choice. Both sum a token's experts in a fixed order.
+
+    params: width, inner, limit, alpha (default 1.702), experts, top, groups, keep (default 1, 1: no restriction), scale
+    (default 1), shared (0: none), shared_limit. tensors: router [experts, width], `gate{e}`, `up{e}` [inner, width],
+    `down{e}` [width, inner] per expert e, and shared_gate, shared_up [shared, width], shared_down [width, shared],
+    shared_weight [1, width]."""
+
+    graph_safe = True
+    SPARSE_MAX_TOKENS = 32  # up to this many tokens only the chosen experts are read
+
+    def __init__(self, spec, runtime):
+        super().__init__(spec, runtime)
+        p = spec.params
+        self.width, self.inner = int(p["width"]), int(p["inner"])
+        self.limit, self.alpha = float(p["limit"]), float(p.get("alpha", 1.702))
+        self.experts, self.top = int(p["experts"]), int(p["top"])
+        self.groups, self.keep = int(p.get("groups") or 1), int(p.get("keep") or 1)
+        self.scale = float(p.get("scale", 1.0))
+        self.shared = int(p.get("shared") or 0)
+        self.shared_limit = float(p["shared_limit"]) if self.shared else 1.0
+        if not (self.limit > 0 and self.shared_limit > 0):
+            raise ValueError("routed feed-forward: the caps must be positive")
+        if self.experts % self.groups or not 1 <= self.keep <= self.groups:
+            raise ValueError(f"routed feed-forward: {self.keep} of {self.groups} groups of {self.experts} experts do not fit")
+        if (self.experts > ops.MOE_MAX_EXPERTS
+                or not 1 <= self.top <= min(self.keep * (self.experts // self.groups), ops.MOE_MAX_TOP)):
+            raise ValueError(f"routed feed-forward: {self.top} of {self.experts} experts is outside what the kernels "
+                             f"take (experts <= {ops.MOE_MAX_EXPERTS}, chosen <= {ops.MOE_MAX_TOP})")
+        self.w_router = self.w_gu = self.w_down = None
+
+    def tensors(self):
+        t = self.spec.tensors
+        out = {t["router"]: TensorNeed((self.experts, self.width))}
+        for e in range(self.experts):
+            out[t[f"gate{e}"]] = TensorNeed((self.inner, self.width))
+            out[t[f"up{e}"]] = TensorNeed((self.inner, self.width))
+            out[t[f"down{e}"]] = TensorNeed((self.width, self.inner))
+        if self.shared:
+            out[t["shared_gate"]] = TensorNeed((self.shared, self.width))
+            out[t["shared_up"]] = TensorNeed((self.shared, self.width))
+            out[t["shared_down"]] = TensorNeed((self.width, self.shared))
+            out[t["shared_weight"]] = TensorNeed((1, self.width))
+        return out
+
+    def load(self, get):
+        t = self.spec.tensors
+        names = [str(e) for e in range(self.experts)]
+        gates, ups = [get(t["gate" + e]) for e in names], [get(t["up" + e]) for e in names]
+        downs, router = [get(t["down" + e]) for e in names], [get(t["router"])]
+        if self.shared:
+            gates.append(get(t["shared_gate"]))
+            ups.append(get(t["shared_up"]))
+            downs.append(get(t["shared_down"]))
+            router.append(get(t["shared_weight"]))
+        self.w_router = torch.cat(router, dim=0).contiguous()
+        self.w_gu = torch.cat(gates + ups, dim=0).contiguous()
+        self.w_down = torch.cat(downs, dim=1).contiguous()
+
+    def weight_bytes(self):
+        """What a step of several tokens reads at most: the router and every expert once."""
+        return sum(w.numel() * w.element_size() for w in (self.w_router, self.w_gu, self.w_down))
+
+    def forward(self, h, stream, step) -> None:
+        rt, T = self.rt, h.shape[0]
+        stream = rt.stream(stream)
+        logits = rt.linear(h, self.w_router, out_dtype=torch.float32)  # [experts | the shared one's weight]
+        entries = self.top + (1 if self.shared else 0)
+        idx = torch.empty(T, entries, dtype=torch.int32, device=rt.device)
+        wts = torch.empty(T, entries, dtype=torch.float32, device=rt.device)
+        few = T <= self.SPARSE_MAX_TOKENS
+        spread = None if few else torch.empty(T, logits.shape[1], dtype=torch.float32, device=rt.device)
+        ops.moe_route_grouped(logits, self.experts, self.groups, self.keep, self.top, self.scale, self.shared > 0, idx,
+                              wts, spread)
+        if few:
+            a = rt.empty(T * entries, max(self.inner, self.shared))
+            y, fresh = stream.claim()
+            ops.moe_sparse_capped(h, self.w_gu, self.w_down, idx, wts, a, y, fresh, self.experts, self.inner, self.shared,
+                                  self.limit, self.shared_limit, self.alpha)
+            return
+        gu = rt.linear(h, self.w_gu)
+        a = rt.empty(T, self.w_down.shape[1])
+        ops.moe_glu_capped_dense(gu, spread, a, self.experts * self.inner, self.inner, self.limit, self.shared_limit,
+                                 self.alpha)
+        stream.add_linear(a, self.w_down)

@@ -1,5 +1,6 @@
 """RMSNorm: h = x * rsqrt(mean(x^2) + eps) * w, the weight multiplies directly
-(src/provider/local/model/cpu.rs:3651-3654; formula in model/gpu.rs:5883-5896)."""
+(src/provider/local/model/cpu.rs:3651-3654; formula in model/gpu.rs:5883-5896). Beside it the layer norm and the forms
+other arrangements of a layer want."""
 from __future__ import annotations
 
 from ..kernels import ops
@@ -40,6 +41,44 @@ class RMSNorm(Norm):
         else:
             ops.rmsnorm(x, self.weight, out, self.eps, rows, groups=self.groups)
         return out
+
+
+    def add_normed(self, x, terms, out) -> None:
+        """x += this norm of the terms' weighted sum; `out` (or None): the new x in the compute dtype."""
+        if self.groups != 1:
+            raise ValueError("rmsnorm: a norm in parts is not applied to a sublayer's output")
+        ops.norm_add(x, terms, self.weight, self.eps, out, center=False)
+
+
+@register_norm("layernorm")
+class LayerNorm(Norm):
+    """h = (x - mean) / sqrt(mean((x - mean)^2) + eps) * w, a weight and no bias.
+    params: width, eps. tensors: weight [width]."""
+
+    def __init__(self, spec, runtime):
+        super().__init__(spec, runtime)
+        self.width = int(spec.params["width"])
+        self.eps = float(spec.params["eps"])
+        self.weight = None
+
+    def tensors(self):
+        return {self.spec.tensors["weight"]: TensorNeed((self.width,), keep_fp32=True, init="ones")}
+
+    def load(self, get):
+        self.weight = get(self.spec.tensors["weight"])
+
+    def weight_bytes(self):
+        return self.weight.numel() * self.weight.element_size()
+
+    def forward(self, stream, rows=None):
+        x = self.rt.stream(stream).data
+        out = self.rt.empty(x.shape[0] if rows is None else rows.shape[0], self.width)
+        ops.layer_norm(x, self.weight, out, self.eps, rows)
+        return out
+
+    def add_normed(self, x, terms, out) -> None:
+        """x += this norm of the terms' weighted sum; `out` (or None): the new x in the compute dtype."""
+        ops.norm_add(x, terms, self.weight, self.eps, out)
 
 
 @register_norm("rmsnorm_scalar")

@@ -1,11 +1,12 @@
 """Two mixers side by side on the same input: out = c (n(left(h)) * w_l + n(right(h)) * w_r), each output
-RMS-normed over the model's width with a weight of its own before they are joined."""
+RMS-normed over the model's width with a weight of its own before they are joined; or, without norms,
+out = c_l left(h) + c_r right(h)."""
 from __future__ import annotations
 
 import dataclasses
 
 from ..kernels import ops
-from ..runtime import ResidualStream
+from ..runtime import ResidualStream, SublayerOutput
 from .base import MIXERS, CacheNeeds, Mixer, StateNeeds, TensorNeed, register_mixer
 
 
@@ -19,15 +20,19 @@ def _named(state, prefix: str) -> dict:
 
 @register_mixer("parallel")
 class ParallelMixers(Mixer):
-    """params: width, eps, scale (c, default 1/2), left, right (the `PartSpec`s of the two mixers).
-    tensors: left_out [width], right_out [width]. At most one of the two may keep paged keys and values; their
+    """params: width, left, right (the `PartSpec`s of the two mixers), norms (default True), with norms eps and scale (c,
+    default 1/2), without left_scale and right_scale (default 1).
+    tensors: with norms left_out [width], right_out [width]. At most one of the two may keep paged keys and values; their
     per-request states live side by side in the layer run's slot, named `left.*` and `right.*`."""
 
     def __init__(self, spec, runtime):
         super().__init__(spec, runtime)
         p = spec.params
-        self.width, self.eps = int(p["width"]), float(p["eps"])
-        self.scale = float(p.get("scale", 0.5))
+        self.width = int(p["width"])
+        self.norms = bool(p.get("norms", True))
+        if self.norms:
+            self.eps, self.scale = float(p["eps"]), float(p.get("scale", 0.5))
+        self.factors = {name: float(p.get(name + "_scale", 1.0)) for name in ("left", "right")}
         self.sides = {name: MIXERS.get(p[name].kind)(p[name], runtime) for name in ("left", "right")}
         self.w_left = self.w_right = None
 
@@ -47,15 +52,16 @@ class ParallelMixers(Mixer):
 
     def tensors(self):
         t = self.spec.tensors
-        out = {t["left_out"]: TensorNeed((self.width,), keep_fp32=True, init="ones"),
-               t["right_out"]: TensorNeed((self.width,), keep_fp32=True, init="ones")}
+        out = {t[name]: TensorNeed((self.width,), keep_fp32=True, init="ones") for name in ("left_out", "right_out")} \
+            if self.norms else {}
         for m in self.sides.values():
             out.update(m.tensors())
         return out
 
     def load(self, get):
         t = self.spec.tensors
-        self.w_left, self.w_right = get(t["left_out"]), get(t["right_out"])
+        if self.norms:
+            self.w_left, self.w_right = get(t["left_out"]), get(t["right_out"])
         for m in self.sides.values():
             m.load(get)
 
@@ -64,7 +70,8 @@ class ParallelMixers(Mixer):
             m.prepare(context_length)
 
     def weight_bytes(self):
-        return (self.w_left.numel() + self.w_right.numel()) * 4 + sum(m.weight_bytes() for m in self.sides.values())
+        norms = (self.w_left.numel() + self.w_right.numel()) * 4 if self.norms else 0
+        return norms + sum(m.weight_bytes() for m in self.sides.values())
 
     def _view(self, cache, name: str):
         """The side's share of the layer run's cache: the pages if it is the one that keeps them, its own states."""
@@ -80,6 +87,16 @@ class ParallelMixers(Mixer):
 
     def forward(self, h, stream, step, cache) -> None:
         rt, rows = self.rt, h.shape[0]
+        if not self.norms:
+            # the two outputs stay terms of one weighted sum: whoever adds the sum up reads each once
+            target = rt.stream(stream)
+            out = target if isinstance(target, SublayerOutput) else SublayerOutput(rt, rows, self.width)
+            for name, m in self.sides.items():
+                m.forward(h, out.scaled(self.factors[name]), step, self._view(cache, name))
+            if out is not target:
+                x, fresh = target.claim()
+                ops.add_terms(x, out.terms, store=fresh)
+            return
         outs = {}
         for name, m in self.sides.items():
             y = ResidualStream.unwritten(rt, rows, self.width)

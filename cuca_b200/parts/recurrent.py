@@ -389,3 +389,57 @@ class Retention(Mixer):
         out = rt.empty(rows, H * dv)
         ops.head_norm_gate(o, None, False, proj[:, 2 * H * d + H * dv:], out, H, dv, self.eps, gate_act="silu")
         rt.stream(stream).add_linear(out, self.w_o)
+
+
+@register_mixer("lightning")
+class Lightning(Mixer):
+    """Lightning attention: linear attention with one fixed decay per head behind silu, no softmax, no denominator, no
+    rotation and no scale. q = silu(W_q h), k = silu(W_k h) (heads x dim), v = silu(W_v h) (heads x vdim); per head, S
+    of dim x vdim (zero at the start):
+        S <- decay_a S + k v^T;   o = S^T q;
+    the concatenated heads are divided by their common root mean square, times `norm` [heads * vdim], times
+    sigmoid(W_g h), then W_o. State: S in 32-bit.
+    params: width, heads, dim, vdim, decay (one number per head), eps. tensors: q, k, v, g, norm, o."""
+
+    graph_safe = True
+
+    def __init__(self, spec, runtime):
+        super().__init__(spec, runtime)
+        p = spec.params
+        self.width, self.heads = int(p["width"]), int(p["heads"])
+        self.dim, self.vdim, self.eps = int(p["dim"]), int(p["vdim"]), float(p["eps"])
+        self.decay_values = [float(v) for v in p["decay"]]
+        if len(self.decay_values) != self.heads:
+            raise ValueError(f"lightning: {len(self.decay_values)} decays for {self.heads} heads")
+        if self.dim > ops.MATRIX_STATE_MAX_DIM:
+            raise ValueError(f"lightning: {self.dim} key channels exceed {ops.MATRIX_STATE_MAX_DIM}")
+        self.w_in = self.w_o = self.norm_w = self.decay = None
+
+    def cache_needs(self):
+        return CacheNeeds(state={"memory": StateNeeds((self.heads, self.vdim, self.dim))})
+
+    def tensors(self):
+        t, E, H = self.spec.tensors, self.width, self.heads
+        inner = H * self.vdim
+        return {t["q"]: TensorNeed((H * self.dim, E)), t["k"]: TensorNeed((H * self.dim, E)),
+                t["v"]: TensorNeed((inner, E)), t["g"]: TensorNeed((inner, E)),
+                t["norm"]: TensorNeed((inner,), keep_fp32=True, init="ones"), t["o"]: TensorNeed((E, inner))}
+
+    def load(self, get):
+        t = self.spec.tensors
+        self.w_in = torch.cat([get(t[r]) for r in ("q", "k", "v", "g")], dim=0).contiguous()
+        self.norm_w, self.w_o = get(t["norm"]), get(t["o"])
+        self.decay = torch.tensor(self.decay_values, dtype=torch.float32, device=self.rt.device)
+
+    def weight_bytes(self):
+        return sum(w.numel() * w.element_size() for w in (self.w_in, self.norm_w, self.w_o))
+
+    def forward(self, h, stream, step, cache) -> None:
+        rt, rows = self.rt, h.shape[0]
+        H, d, dv = self.heads, self.dim, self.vdim
+        proj = rt.linear(h, self.w_in, out_dtype=torch.float32)  # [q | k | v | g]
+        o = rt.empty(rows, H * dv, dtype=torch.float32)
+        ops.lightning_scan(proj, self.decay, cache.state["memory"], o, step, H, d, dv)
+        out = rt.empty(rows, H * dv)
+        ops.row_norm_gate(o, self.norm_w, proj[:, H * (2 * d + dv):], out, self.eps)
+        rt.stream(stream).add_linear(out, self.w_o)

@@ -19,7 +19,7 @@ import torch
 from .base import PositionEncoding, register_position
 
 
-def llama3_factors(n_dims: int, base: float, factor: float, low: float, high: float, original: int) -> np.ndarray:
+def llama3_factors(n_dims: int, base: float, factor: float, low: float, high: float, original: float) -> np.ndarray:
     out = np.empty(n_dims // 2, dtype=np.float32)
     low_wavelen, high_wavelen = original / low, original / high
     for i in range(n_dims // 2):
@@ -95,7 +95,7 @@ class RotaryEncoding(PositionEncoding):
         elif kind == "llama3":
             factors = llama3_factors(self.rotary_dim, self.theta, float(self.scaling["factor"]),
                                      float(self.scaling["low_freq_factor"]), float(self.scaling["high_freq_factor"]),
-                                     int(self.scaling["original_max_position_embeddings"]))
+                                     float(self.scaling["original_max_position_embeddings"]))
         elif kind == "linear":
             freq_scale = 1.0 / float(self.scaling["factor"])
         elif kind != "default":

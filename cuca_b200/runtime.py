@@ -81,6 +81,7 @@ class ResidualStream:
         self._tensor = tensor
         self._pending = None
         self._unwritten = False
+        self._rounded = None  # the stream in the compute dtype, while nothing has touched the stream since it was made
 
     @classmethod
     def unwritten(cls, runtime: "Runtime", rows: int, width: int) -> "ResidualStream":
@@ -94,7 +95,7 @@ class ResidualStream:
         """The stream is `tensor` from now on (an operation that rewrote the whole stream out of place)."""
         if tensor.dtype != torch.float32 or tensor.shape != self._tensor.shape:
             raise ValueError("a residual stream is replaced by a 32-bit tensor of its own shape")
-        self._pending = None
+        self._pending = self._rounded = None
         self._tensor = tensor
 
     @property
@@ -104,6 +105,7 @@ class ResidualStream:
     @property
     def data(self) -> torch.Tensor:
         """The stream's tensor with everything added; it may be read and updated in place."""
+        self._rounded = None
         if self._unwritten:
             self._tensor.zero_()
             self._unwritten = False
@@ -115,6 +117,7 @@ class ResidualStream:
     def take(self):
         """(tensor, pending slices or None) for a reader that adds the slices itself, in the stream too: after
         the reader's kernel the tensor must hold the sum."""
+        self._rounded = None
         if self._unwritten:
             self._tensor.zero_()
             self._unwritten = False
@@ -132,6 +135,7 @@ class ResidualStream:
     def add_linear(self, a, w, bias=None) -> None:
         """stream += a @ w.T (+ bias). Over few tokens the slices may stay pending until the next reader."""
         rt = self.rt
+        self._rounded = None
         if self._unwritten:
             self._unwritten = False
             ops.gemm(a, w, self._tensor, ops.EPI_STORE, bias, rt.err)
@@ -150,3 +154,94 @@ class ResidualStream:
     def drop_pending(self) -> None:
         """Forget unadded slices: the stream will not be read again (no logits are wanted)."""
         self._pending = None
+
+    # ------------------------------------------------ arrangements whose sublayers read the stream as it is
+    def rounded(self) -> torch.Tensor:
+        """The stream in the compute dtype, to be read only: what `add_normed` left, else made now. In the 32-bit mode
+        the stream itself."""
+        if self._rounded is None:
+            x = self.data
+            if x.dtype == self.rt.dtype:
+                return x
+            out = self.rt.empty(*x.shape)
+            ops.round_rows(x, out)
+            self._rounded = out
+        return self._rounded
+
+    def add_normed(self, output: "SublayerOutput", norm) -> None:
+        """stream += norm(output), `norm` a part with `add_normed`; the rounded copy for the next sublayer's reader
+        comes from the same pass."""
+        x = self.data
+        out = None if x.dtype == self.rt.dtype else self.rt.empty(*x.shape)
+        norm.add_normed(x, output.terms, out)
+        self._rounded = out
+
+
+class SublayerOutput(ResidualStream):
+    """A sublayer's output gathered apart from the stream, for an arrangement that norms it before it is added: a
+    weighted sum of terms, each a 32-bit tensor or the unadded K slices of a contraction. Nothing adds them up until
+    a reader that takes terms does (`ResidualStream.add_normed`, `ops.add_terms`). A part writes to it as to a stream;
+    `scaled(c)` is the same output with everything written through it multiplied by c."""
+
+    def __init__(self, runtime: Runtime, rows: int, width: int):
+        self.rt = runtime
+        self._shape = (rows, width)
+        self.factor = 1.0
+        self.terms: list = []  # (tensor or PartialSums, factor)
+
+    def scaled(self, factor: float) -> "SublayerOutput":
+        view = SublayerOutput(self.rt, *self._shape)
+        view.factor = self.factor * float(factor)
+        view.terms = self.terms
+        return view
+
+    @property
+    def shape(self):
+        return torch.Size(self._shape)
+
+    def claim(self):
+        for t, c in self.terms:
+            if isinstance(t, torch.Tensor) and c == self.factor:
+                return t, False
+        if len(self.terms) >= ops.MAX_TERMS:
+            self._merge()
+            return self.claim() if self.factor == 1.0 else self._fresh()
+        return self._fresh()
+
+    def _fresh(self):
+        t = torch.empty(*self._shape, dtype=torch.float32, device=self.rt.device)
+        self.terms.append((t, self.factor))
+        return t, True
+
+    def _merge(self) -> torch.Tensor:
+        """One term with factor 1 in the place of all."""
+        t = torch.empty(*self._shape, dtype=torch.float32, device=self.rt.device)
+        ops.add_terms(t, self.terms, store=True)
+        self.terms[:] = [(t, 1.0)]
+        return t
+
+    @property
+    def data(self) -> torch.Tensor:
+        if self.factor != 1.0:
+            raise ValueError("a scaled view of a sublayer's output is only written to")
+        if len(self.terms) == 1 and isinstance(self.terms[0][0], torch.Tensor) and self.terms[0][1] == 1.0:
+            return self.terms[0][0]
+        return self._merge()
+
+    def take(self):
+        return self.data, None
+
+    def add_linear(self, a, w, bias=None) -> None:
+        rt = self.rt
+        if (rt.use_partials and bias is None and len(self.terms) < ops.MAX_TERMS - 1
+                and ops.gemm_partial_supported(a, w)):
+            self.terms.append((ops.gemm_partial(a, w, rt.err), self.factor))
+            return
+        t, fresh = self.claim()
+        ops.gemm(a, w, t, ops.EPI_STORE if fresh else ops.EPI_RESIDUAL, bias, rt.err)
+
+    def replace(self, tensor: torch.Tensor) -> None:
+        raise ValueError("a sublayer's output is written to, not replaced")
+
+    def drop_pending(self) -> None:
+        pass
