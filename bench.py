@@ -273,6 +273,24 @@ def _sutosun_config(width, ff, heads, layers, vocab, window):
                        for i in range(layers)]}
 
 
+def _nudorax_config(width, ff, heads, layers, vocab, window):
+    """`layers` layers alike: sliding-window attention (half as many heads of 128 as the width holds, a quarter as many key
+    heads, rotation of a whole head with frequencies scaled by wavelength, a norm over the whole q and k projections, a
+    sink per head) beside lightning attention (as many heads of 128 x 128), and routed capped units (eight experts of
+    ff / 4 in four groups of which two are kept, two chosen, and a shared expert of ff / 4)."""
+    H = max(1, width // 256)
+    left = {"heads": H, "kv_heads": max(1, H // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": window},
+            "rot": {"base": 500000.0, "dims": 128,
+                    "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    right = {"heads": H, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** -(5 + a % 8) for a in range(H)]}
+    layer = {"type": "parallel",
+             "mixer": {"left": left, "right": right, "left_scale": 0.7, "right_scale": 0.9},
+             "mlp": {"kind": "moe", "expert": {"ff": ff // 4, "limit": 7.0}, "shared": {"ff": ff // 4, "limit": 7.0},
+                     "router": {"experts": 8, "top": 2, "scale": 1.5, "groups": {"count": 4, "keep": 2}}}}
+    return {"architecture": "Nudorax", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "logit_softcap": 30.0,
+            "embedding": {"scale": width ** 0.5}, "layers": [layer] * layers}
+
+
 def _llama_config(width, ff, heads, layers, vocab):
     return {"architectures": ["LlamaForCausalLM"], "model_type": "llama", "num_hidden_layers": layers,
             "hidden_size": width, "num_attention_heads": heads, "num_key_value_heads": max(1, heads // 4),
@@ -287,8 +305,8 @@ DESIGN_SIZES = {  # name -> (width, feed-forward, heads, layers, vocabulary)
 
 def design_table(args) -> int:
     """Prefill of one prompt and decode steps of `--batch` requests for the chosen design and for a Llama of the
-    same width, feed-forward size and number of layer runs (for Sutosun: a Pudinex, the closest of the other designs,
-    and the Llama), one JSON line per size and model: tokens/s of both phases, the decode step's bytes (weights once,
+    same width, feed-forward size and number of layer runs (for Sutosun also a Pudinex and for Nudorax also a Sutosun,
+    the closest of the other designs), one JSON line per size and model: tokens/s of both phases, the decode step's bytes (weights once,
     what a request keeps) over the measured copy bandwidth."""
     import numpy as np
     import torch
@@ -303,12 +321,14 @@ def design_table(args) -> int:
     ctx = max(T, P + steps + warmup + 64) + 64
     for size in (args.sizes.split(",") if args.sizes else list(DESIGN_SIZES)):
         width, ff, heads, layers, vocab = DESIGN_SIZES[size]
-        runs = layers if args.design in ("pudinex", "sutosun") else layers + layers // 2  # (a looped half runs twice)
+        runs = layers if args.design in ("pudinex", "sutosun", "nudorax") else layers + layers // 2  # (a looped half runs twice)
         make = {"bananex": _bananex_config, "dupenex": _dupenex_config, "pudinex": _pudinex_config,
-                "sutosun": _sutosun_config}[args.design]
+                "sutosun": _sutosun_config, "nudorax": _nudorax_config}[args.design]
         pair = [(args.design, make(width, ff, heads, layers, vocab, window=1024))]
         if args.design == "sutosun":
             pair.append(("pudinex", _pudinex_config(width, ff, heads, layers, vocab, window=1024)))
+        if args.design == "nudorax":
+            pair.append(("sutosun", _sutosun_config(width, ff, heads, layers, vocab, window=1024)))
         pair.append(("llama", _llama_config(width, ff, heads, runs, vocab)))
         for name, cfg in pair:
             if args.only_model and name != args.only_model:
@@ -397,7 +417,7 @@ def main() -> int:
     ap.add_argument("--decode-only", action="store_true",
                     help="with --shape llama-3.2-1b: the plain decode line at --batch instead of the mixed workload")
     ap.add_argument("--only-model", default=None, help="with --design: run only this model of the pair (the design's name or llama)")
-    ap.add_argument("--design", default=None, choices=["bananex", "dupenex", "pudinex", "sutosun"],
+    ap.add_argument("--design", default=None, choices=["bananex", "dupenex", "nudorax", "pudinex", "sutosun"],
                     help="instead of the bench: prefill and decode of this design beside a Llama of equal width, "
                          "feed-forward size and layer runs, at --sizes (1b,3b,8b layer sizes; a few layers each)")
     ap.add_argument("--sizes", default=None, help="with --design: which of 1b,3b,8b (all else)")

@@ -213,17 +213,34 @@ round_rows_kernel(const float* __restrict__ x, TO* __restrict__ out, size_t n) {
     st<V>(out + i, ld<V>(x + i));
 }
 
-// o: [rows, n] 32-bit; gate: 32-bit rows of stride ldg. One block per row.
-template <typename TO, int V>
+template <int V> __device__ __forceinline__ Pack<V> ld_as_f32(const float* p) { return ld<V>(p); }
+template <int V> __device__ __forceinline__ Pack<V> ld_as_f32(const __nv_bfloat16* p) {
+  Pack<V> r;
+  if (V == 4) {
+    const uint2 w = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w.y));
+    r.v[0] = a.x;
+    if (V > 1) r.v[V > 1 ? 1 : 0] = a.y;
+    if (V > 2) r.v[V > 2 ? 2 : 0] = b.x;
+    if (V > 3) r.v[V > 3 ? 3 : 0] = b.y;
+  } else {
+    r.v[0] = __bfloat162float(p[0]);
+  }
+  return r;
+}
+
+// o: [rows, n] 32-bit; gate: rows of stride ldg. One block per row.
+template <typename TG, typename TO, int V>
 __global__ void __launch_bounds__(512)
-row_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ w, const float* __restrict__ gate, int ldg,
+row_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ w, const TG* __restrict__ gate, int ldg,
                      TO* __restrict__ out, int n, float eps) {
   __shared__ float red[32];
   pdl_trigger();
   pdl_wait();
   const size_t row = blockIdx.x;
   const float* orow = o + row * n;
-  const float* grow = gate + row * ldg;
+  const TG* grow = gate + row * ldg;
   TO* dst = out + row * n;
   float q = 0.f;
   for (int i = threadIdx.x * V; i < n; i += blockDim.x * V) {
@@ -234,7 +251,7 @@ row_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ w, c
   const float inv = 1.f / sqrtf(block_sum(q, red) / (float)n + eps);
   for (int i = threadIdx.x * V; i < n; i += blockDim.x * V) {
     Pack<V> v = ld<V>(orow + i);
-    const Pack<V> g = ld<V>(grow + i), wv = ld<V>(w + i);
+    const Pack<V> g = ld_as_f32<V>(grow + i), wv = ld<V>(w + i);
 #pragma unroll
     for (int k = 0; k < V; ++k) v.v[k] = v.v[k] * inv * wv.v[k] / (1.f + expf(-g.v[k]));
     st<V>(dst + i, v);
@@ -350,26 +367,28 @@ CUCA_API int cuca_round_rows(const float* x, void* out, int out_dtype, size_t n,
   return 0;
 }
 
-// out[r] = o[r] / sqrt(mean(o[r]^2) + eps) * w * sigmoid(gate[r]); o: [n_rows, n], gate: rows of stride ldg, both 32-bit
-CUCA_API int cuca_row_norm_gate(const float* o, const float* w, const float* gate, int ldg, void* out, int out_dtype,
-                                int n_rows, int n, float eps, cudaStream_t stream) {
+// out[r] = o[r] / sqrt(mean(o[r]^2) + eps) * w * sigmoid(gate[r]); o: [n_rows, n] 32-bit, gate: rows of stride ldg
+CUCA_API int cuca_row_norm_gate(const float* o, const float* w, const void* gate, int gate_dtype, int ldg, void* out,
+                                int out_dtype, int n_rows, int n, float eps, cudaStream_t stream) {
   if (n_rows == 0) return 0;
   CUCA_REQUIRE(n > 0, "row_norm_gate: bad width %d", n);
-  const bool wide = n % 4 == 0 && ldg % 4 == 0 && aligned(o, 16) && aligned(w, 16) && aligned(gate, 16) && aligned(out, 16);
+  const bool wide = n % 4 == 0 && ldg % 4 == 0 && aligned(o, 16) && aligned(w, 16) && aligned(gate, gate_dtype == CUCA_F32 ? 16 : 8) &&
+                    aligned(out, 16);
   const int packs = wide ? n / 4 : n;
   int threads = (packs + 31) / 32 * 32;
   threads = threads > 512 ? 512 : threads;
   if (n_rows >= 512 && threads > 256) threads = 256;
-#define RNG(TO)                                                                                                        \
+#define RNG(TG, TO)                                                                                                    \
   do {                                                                                                                 \
-    if (wide) cuca_launch(row_norm_gate_kernel<TO, 4>, dim3(n_rows), dim3(threads), 0, stream, true, o, w, gate, ldg,   \
-                          (TO*)out, n, eps);                                                                           \
-    else cuca_launch(row_norm_gate_kernel<TO, 1>, dim3(n_rows), dim3(threads), 0, stream, true, o, w, gate, ldg,        \
-                     (TO*)out, n, eps);                                                                                \
+    if (wide) cuca_launch(row_norm_gate_kernel<TG, TO, 4>, dim3(n_rows), dim3(threads), 0, stream, true, o, w,          \
+                          (const TG*)gate, ldg, (TO*)out, n, eps);                                                     \
+    else cuca_launch(row_norm_gate_kernel<TG, TO, 1>, dim3(n_rows), dim3(threads), 0, stream, true, o, w,               \
+                     (const TG*)gate, ldg, (TO*)out, n, eps);                                                          \
   } while (0)
-  if (out_dtype == CUCA_F32) RNG(float);
-  else if (out_dtype == CUCA_BF16) RNG(__nv_bfloat16);
-  else CUCA_REQUIRE(false, "row_norm_gate: unknown dtype %d", out_dtype);
+  if (gate_dtype == CUCA_F32 && out_dtype == CUCA_F32) RNG(float, float);
+  else if (gate_dtype == CUCA_F32 && out_dtype == CUCA_BF16) RNG(float, __nv_bfloat16);
+  else if (gate_dtype == CUCA_BF16 && out_dtype == CUCA_BF16) RNG(__nv_bfloat16, __nv_bfloat16);
+  else CUCA_REQUIRE(false, "row_norm_gate: unsupported dtypes %d/%d", gate_dtype, out_dtype);
 #undef RNG
   CUCA_CHECK_LAUNCH("row_norm_gate");
   return 0;

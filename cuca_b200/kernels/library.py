@@ -150,7 +150,10 @@ _SIGNATURES = {
     "cuca_layer_norm": [_P, _P, _P, _I, _P, _I, _I, _F, _P],
     "cuca_add_terms": [_P, _P, _I, c_size_t, _P],
     "cuca_round_rows": [_P, _P, _I, c_size_t, _P],
-    "cuca_row_norm_gate": [_P, _P, _P, _I, _P, _I, _I, _I, _F, _P],
+    "cuca_row_norm_gate": [_P, _P, _P, _I, _I, _P, _I, _I, _I, _F, _P],
+    "cuca_lightning_chunk_tokens": [],
+    "cuca_lightning_chunk_max_dim": [],
+    "cuca_lightning_chunked": [_P, _I, _I, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P],
     "cuca_moe_sparse_act": [_P, _P, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _P],
     "cuca_moe_route_grouped": [_P, _I, _I, _I, _I, _I, _F, _I, _P, _P, _P, _P],
     "cuca_moe_glu_capped_dense": [_P, _P, _I, _P, _I, _I, _I, _I, _I, _F, _F, _F, _P],

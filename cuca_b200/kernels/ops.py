@@ -1056,11 +1056,36 @@ def lightning_scan(proj, decay, state, out, step, H, d, dv) -> None:
 
 
 def row_norm_gate(o, weight, gate, out, eps: float) -> None:
-    """out[r] = o[r] / rms(o[r]) * weight * sigmoid(gate[r]) over whole rows; gate: 32-bit rows of any stride."""
+    """out[r] = o[r] / rms(o[r]) * weight * sigmoid(gate[r]) over whole rows; gate: rows of any stride."""
     _cuda(o, weight, gate, out)
-    library.check(library.load().cuca_row_norm_gate(_p(o), _p(weight), _p(gate), gate.stride(0), _p(out),
-                                                    dtype_code(out.dtype), o.shape[0], o.shape[1], float(eps), _stream()),
-                  "row_norm_gate")
+    library.check(library.load().cuca_row_norm_gate(_p(o), _p(weight), _p(gate), dtype_code(gate.dtype), gate.stride(0),
+                                                    _p(out), dtype_code(out.dtype), o.shape[0], o.shape[1], float(eps),
+                                                    _stream()), "row_norm_gate")
+
+
+LIGHTNING_CHUNK, LIGHTNING_CHUNK_MAX_DIM = 64, 256  # `cuca_lightning_chunk_tokens` / `_max_dim` say the same
+LIGHTNING_CHUNKED_FROM = 32  # steps with a portion at least this long, in the serving precision only
+
+
+def lightning_chunks(step, dtype, d: int) -> int:
+    """Chunks of this step's portions if it should run chunk by chunk on the tensor cores, else 0 (token by token: single
+    tokens, short portions, the 32-bit path always)."""
+    counts = step.host.get("counts") if step.static_max_len is None else None
+    if dtype != torch.bfloat16 or d > LIGHTNING_CHUNK_MAX_DIM or not counts or max(counts) < LIGHTNING_CHUNKED_FROM:
+        return 0
+    return sum(-(-c // LIGHTNING_CHUNK) for c in counts)
+
+
+def lightning_chunked(proj, decay, state, out, step, n_chunks: int, H, d, dv) -> None:
+    """`lightning_scan` chunk by chunk from a bfloat16 `proj` (read only); three launches."""
+    _cuda(proj, decay, state, out)
+    if proj.dtype != torch.bfloat16:
+        raise library.KernelError("lightning_chunked takes a bfloat16 projection")
+    chunks = torch.empty(n_chunks, H, dv, d, dtype=torch.float32, device=out.device)
+    library.check(library.load().cuca_lightning_chunked(
+        _p(proj), proj.stride(0), 0, _p(decay), _p(state), _p(chunks), _p(out), _p(step.req_row0), _p(step.req_count),
+        _p(step.slots), step.n_seqs, n_chunks, H, d, dv, _stream()), "lightning_chunked")
+    library.launches += 2
 
 
 def head_norm_gate(o, weight, per_head: bool, gate, out, H, dv, eps, gate_act: str = "sigmoid") -> None:

@@ -398,7 +398,8 @@ class Lightning(Mixer):
     of dim x vdim (zero at the start):
         S <- decay_a S + k v^T;   o = S^T q;
     the concatenated heads are divided by their common root mean square, times `norm` [heads * vdim], times
-    sigmoid(W_g h), then W_o. State: S in 32-bit.
+    sigmoid(W_g h), then W_o. State: S in 32-bit. Single tokens and short portions walk the recurrence token by token;
+    in bfloat16 a step with a long portion runs chunk by chunk on the tensor cores (`csrc/lightning_chunk.cu`).
     params: width, heads, dim, vdim, decay (one number per head), eps. tensors: q, k, v, g, norm, o."""
 
     graph_safe = True
@@ -437,9 +438,13 @@ class Lightning(Mixer):
     def forward(self, h, stream, step, cache) -> None:
         rt, rows = self.rt, h.shape[0]
         H, d, dv = self.heads, self.dim, self.vdim
-        proj = rt.linear(h, self.w_in, out_dtype=torch.float32)  # [q | k | v | g]
         o = rt.empty(rows, H * dv, dtype=torch.float32)
-        ops.lightning_scan(proj, self.decay, cache.state["memory"], o, step, H, d, dv)
+        n_chunks = ops.lightning_chunks(step, rt.dtype, d)
+        proj = rt.linear(h, self.w_in, out_dtype=None if n_chunks else torch.float32)  # [q | k | v | g]
+        if n_chunks:
+            ops.lightning_chunked(proj, self.decay, cache.state["memory"], o, step, n_chunks, H, d, dv)
+        else:
+            ops.lightning_scan(proj, self.decay, cache.state["memory"], o, step, H, d, dv)
         out = rt.empty(rows, H * dv)
         ops.row_norm_gate(o, self.norm_w, proj[:, H * (2 * d + dv):], out, self.eps)
         rt.stream(stream).add_linear(out, self.w_o)

@@ -119,6 +119,8 @@ def lightning(h, w, p, m, eps):
     q = silu(mm(h, w[p + "q"])).reshape(T, H, d)
     k = silu(mm(h, w[p + "k"])).reshape(T, H, d)
     v = silu(mm(h, w[p + "v"])).reshape(T, H, dv)
+    if ROUND is not None:
+        q, k, v = ROUND(q), ROUND(k), ROUND(v)
     out = np.zeros((T, H, dv))
     for a in range(H):
         S = np.zeros((d, dv))
