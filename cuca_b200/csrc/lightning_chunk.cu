@@ -40,7 +40,8 @@ __device__ __forceinline__ uint32_t pack2(float a, float b) {
   return *reinterpret_cast<const uint32_t*>(&t);
 }
 __device__ __forceinline__ float rounded(float v) { return __bfloat162float(__float2bfloat16_rn(v)); }
-__device__ __forceinline__ float silu_(float v) { return v / (1.f + expf(-v)); }
+// (rounded to bfloat16 right after: the fast quotient and exponential are exact enough)
+__device__ __forceinline__ float silu_(float v) { return __fdividef(v, 1.f + __expf(-v)); }
 
 // Which chunk of which request the gid-th chunk of the step is, worked out by one warp.
 struct Where { int req, chunk; };
@@ -72,37 +73,50 @@ __device__ Where find_chunk(int gid, const int* __restrict__ req_count, int n_se
 template <typename W>
 __device__ __forceinline__ void stage_silu(const __nv_bfloat16* __restrict__ src, int ld, int n, int n_cols, int pad,
                                            __nv_bfloat16* hi, __nv_bfloat16* lo, int pitch, bool wide, W weight) {
-  const int groups = pad / 8;
-  for (int e = threadIdx.x; e < C * groups; e += blockDim.x) {
-    const int j = e / groups, c = (e % groups) * 8;
-    float v[8];
-    const __nv_bfloat16* at = src + (size_t)j * ld + c;
-    if (j < n && wide && c + 8 <= n_cols) {
-      const uint4 w = *reinterpret_cast<const uint4*>(at);
-      const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&w);
+  const int groups = pad / 8, total = C * groups;
+  constexpr int U = 4;  // pieces a thread asks for before it works on the first
+  for (int e0 = threadIdx.x; e0 < total; e0 += U * blockDim.x) {
+    uint4 raw[U];
 #pragma unroll
-      for (int k = 0; k < 4; ++k) { const float2 f = __bfloat1622float2(h[k]); v[2 * k] = f.x; v[2 * k + 1] = f.y; }
-    } else {
+    for (int u = 0; u < U; ++u) {
+      const int e = e0 + u * blockDim.x, j = e / groups, c = (e % groups) * 8;
+      raw[u] = make_uint4(0u, 0u, 0u, 0u);
+      if (e >= total || j >= n) continue;
+      const __nv_bfloat16* at = src + (size_t)j * ld + c;
+      if (wide && c + 8 <= n_cols) {
+        raw[u] = *reinterpret_cast<const uint4*>(at);
+      } else {
+        uint32_t q[4] = {0u, 0u, 0u, 0u};
 #pragma unroll
-      for (int k = 0; k < 8; ++k) v[k] = (j < n && c + k < n_cols) ? __bfloat162float(at[k]) : 0.f;
-    }
-    const float wt = weight(j);
-    uint4 h4, l4;
-    uint32_t* hp = reinterpret_cast<uint32_t*>(&h4);
-    uint32_t* lp = reinterpret_cast<uint32_t*>(&l4);
-#pragma unroll
-    for (int k = 0; k < 4; ++k) {
-      float a = rounded(silu_(v[2 * k])), b = rounded(silu_(v[2 * k + 1]));
-      if (lo) {
-        a *= wt; b *= wt;
-        const float ah = rounded(a), bh = rounded(b);
-        lp[k] = pack2(a - ah, b - bh);
-        a = ah; b = bh;
+        for (int k = 0; k < 8; ++k)
+          if (c + k < n_cols) q[k >> 1] |= (uint32_t)__bfloat16_as_ushort(at[k]) << (16 * (k & 1));
+        raw[u] = make_uint4(q[0], q[1], q[2], q[3]);
       }
-      hp[k] = pack2(a, b);
     }
-    *reinterpret_cast<uint4*>(hi + (size_t)j * pitch + c) = h4;
-    if (lo) *reinterpret_cast<uint4*>(lo + (size_t)j * pitch + c) = l4;
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int e = e0 + u * blockDim.x, j = e / groups, c = (e % groups) * 8;
+      if (e >= total) break;
+      const __nv_bfloat162* v2 = reinterpret_cast<const __nv_bfloat162*>(&raw[u]);
+      const float wt = weight(j);
+      uint4 h4, l4;
+      uint32_t* hp = reinterpret_cast<uint32_t*>(&h4);
+      uint32_t* lp = reinterpret_cast<uint32_t*>(&l4);
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        const float2 f = __bfloat1622float2(v2[k]);
+        float a = rounded(silu_(f.x)), b = rounded(silu_(f.y));
+        if (lo) {
+          a *= wt; b *= wt;
+          const float ah = rounded(a), bh = rounded(b);
+          lp[k] = pack2(a - ah, b - bh);
+          a = ah; b = bh;
+        }
+        hp[k] = pack2(a, b);
+      }
+      *reinterpret_cast<uint4*>(hi + (size_t)j * pitch + c) = h4;
+      if (lo) *reinterpret_cast<uint4*>(lo + (size_t)j * pitch + c) = l4;
+    }
   }
 }
 
@@ -192,7 +206,7 @@ chunk_state_kernel(const Args p) {
 // Per (request, head) and element of the state: chunks[.] becomes the state before each chunk, state the one behind the
 // last. V elements a thread.
 template <int V>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(128)
 chunk_carry_kernel(const Args p) {
   struct alignas(4 * V) Pack { float v[V]; };
   pdl_trigger();
@@ -216,7 +230,7 @@ chunk_carry_kernel(const Args p) {
   float* ch = p.chunks + ((size_t)first * p.H + h) * per + e;
   const size_t step = (size_t)p.H * per;
   Pack s = *reinterpret_cast<const Pack*>(st);
-  constexpr int AHEAD = 8;  // chunks whose sums are asked for together
+  constexpr int AHEAD = 16;  // chunks whose sums are asked for together
   for (int c0 = 0; c0 < nc; c0 += AHEAD) {
     Pack kv[AHEAD];
 #pragma unroll
@@ -261,23 +275,32 @@ chunk_output_kernel(const Args p, int dp) {
     const float* st = p.chunks + (((size_t)gid * p.H + h) * p.dv + c0) * p.d;
     const int groups = dp / 4;
     const bool wide = (p.d & 3) == 0;
-    for (int e = threadIdx.x; e < CW * groups; e += blockDim.x) {
-      const int c = e / groups, r = (e % groups) * 4;
-      float v[4] = {0.f, 0.f, 0.f, 0.f};
-      const float* at = st + (size_t)c * p.d + r;
-      if (c < nc) {
-        if (wide && r + 4 <= p.d) *reinterpret_cast<float4*>(v) = *reinterpret_cast<const float4*>(at);
-        else {
+    constexpr int U = 8;  // pieces a thread asks for before it splits the first
+    for (int e0 = threadIdx.x; e0 < CW * groups; e0 += U * blockDim.x) {
+      float4 v4[U];
 #pragma unroll
-          for (int k = 0; k < 4; ++k) if (r + k < p.d) v[k] = at[k];
+      for (int u = 0; u < U; ++u) {
+        const int e = e0 + u * blockDim.x, c = e / groups, r = (e % groups) * 4;
+        v4[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (c >= nc) continue;
+        const float* at = st + (size_t)c * p.d + r;
+        if (wide && r + 4 <= p.d) v4[u] = *reinterpret_cast<const float4*>(at);
+        else {
+          if (r < p.d) v4[u].x = at[0];
+          if (r + 1 < p.d) v4[u].y = at[1];
+          if (r + 2 < p.d) v4[u].z = at[2];
+          if (r + 3 < p.d) v4[u].w = at[3];
         }
       }
-      float hi[4];
 #pragma unroll
-      for (int k = 0; k < 4; ++k) hi[k] = rounded(v[k]);
-      *reinterpret_cast<uint2*>(ss_hi + (size_t)c * pitch + r) = make_uint2(pack2(hi[0], hi[1]), pack2(hi[2], hi[3]));
-      *reinterpret_cast<uint2*>(ss_lo + (size_t)c * pitch + r) =
-          make_uint2(pack2(v[0] - hi[0], v[1] - hi[1]), pack2(v[2] - hi[2], v[3] - hi[3]));
+      for (int u = 0; u < U; ++u) {
+        const int e = e0 + u * blockDim.x, c = e / groups, r = (e % groups) * 4;
+        if (c >= CW) break;
+        const float4 v = v4[u];
+        const float h0 = rounded(v.x), h1 = rounded(v.y), h2 = rounded(v.z), h3 = rounded(v.w);
+        *reinterpret_cast<uint2*>(ss_hi + (size_t)c * pitch + r) = make_uint2(pack2(h0, h1), pack2(h2, h3));
+        *reinterpret_cast<uint2*>(ss_lo + (size_t)c * pitch + r) = make_uint2(pack2(v.x - h0, v.y - h1), pack2(v.z - h2, v.w - h3));
+      }
     }
   }
   stage_powers(pw, p.decay[h]);
@@ -382,9 +405,9 @@ CUCA_API int cuca_lightning_chunked(const void* proj, int ld, int col0, const fl
   CUCA_CHECK_LAUNCH("lightning_chunk_state");
   const int per = dv * d;
   if (per % 4 == 0 && ((uintptr_t)chunks & 15) == 0 && ((uintptr_t)state & 15) == 0)
-    cuca_launch(chunk_carry_kernel<4>, dim3((per / 4 + 255) / 256, H, n_seqs), dim3(256), 0, stream, true, p);
+    cuca_launch(chunk_carry_kernel<4>, dim3((per / 4 + 127) / 128, H, n_seqs), dim3(128), 0, stream, true, p);
   else
-    cuca_launch(chunk_carry_kernel<1>, dim3((per + 255) / 256, H, n_seqs), dim3(256), 0, stream, true, p);
+    cuca_launch(chunk_carry_kernel<1>, dim3((per + 127) / 128, H, n_seqs), dim3(128), 0, stream, true, p);
   CUCA_CHECK_LAUNCH("lightning_chunk_carry");
   const int dp = (d + 15) / 16 * 16;
   const size_t smem = output_smem(dp);

@@ -4,6 +4,8 @@
 //   moe_act_dense    a[t, e, f] = relu(u[t, e, f])^2 * weight[t, e]: all experts' up-projections at once, the ones a
 //                    token did not choose weighted 0, so that one contraction over (e, f) is the weighted sum
 //   moe_up_sparse / moe_down_sparse   few tokens: only the chosen experts' weights are read, a warp per output
+//   moe_up_shared / moe_down_shared   the same by expert on the tensor cores, for bfloat16 tokens that share experts:
+//                    each weight row is read once
 //   moe_route_scored scores are a softmax over ALL router outputs; the choice goes by score + a correction per output,
 //                    the weights are the chosen scores over their sum; the last outputs may stand for experts that
 //                    return their input (their weights are summed per token for `moe_identity_add`)
@@ -424,6 +426,169 @@ moe_down_sparse_kernel(const T* __restrict__ a, int lda, const T* __restrict__ w
   if (lane == 0) y[(size_t)t * N + o] = store ? acc : y[(size_t)t * N + o] + acc;
 }
 
+// ---- the same for a few bfloat16 tokens that share experts: an expert's rows are read once, straight into tensor-core
+// operands, for up to sixteen tokens that chose it. The order of k within a product is free as long as both operands
+// agree: a lane takes eight consecutive values (16 bytes) of its weight row and of its token, and they serve as its
+// operands of two 16-wide steps.
+constexpr int SHARED_MAX_TOKENS = 32, SHARED_MAX_EXPERTS = 64, SHARED_TILE = 16, SHARED_K = 32;
+
+__device__ __forceinline__ void mma_tokens(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0,
+                                           uint32_t b1) {
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+               : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+// d[token, row] += 32 values of tokens (lo: tokens 0..7, hi: 8..15) times 32 values of weight rows
+__device__ __forceinline__ void mma_k32(float (&d)[4], const uint4& lo, const uint4& hi, const uint4& w) {
+  mma_tokens(d, lo.x, hi.x, lo.y, hi.y, w.x, w.y);
+  mma_tokens(d, lo.z, hi.z, lo.w, hi.w, w.z, w.w);
+}
+__device__ __forceinline__ uint4 load16(const __nv_bfloat16* p, bool on) {
+  return on ? *reinterpret_cast<const uint4*>(p) : make_uint4(0u, 0u, 0u, 0u);
+}
+
+// Block (x, e, z): eight rows f of expert e for the sixteen of its tokens from number 16 z on; the eight warps take K's runs
+// of 32 in turn and their sums are added in order. Arguments as in `moe_up_sparse_kernel`; K, F and Fs are multiples of
+// 32. (Tokens of a batch may all choose the same two experts: what is in flight must not hang on their number.)
+template <int ACT>
+__global__ void __launch_bounds__(256)
+moe_up_shared_kernel(const __nv_bfloat16* __restrict__ h, const __nv_bfloat16* __restrict__ w_up, const int* __restrict__ idx,
+                     const float* __restrict__ wts, __nv_bfloat16* __restrict__ a, int lda, int n_tokens, int entries, int F,
+                     int Fs, int K, int n_real, size_t up_rows, const SparseUnit unit) {
+  __shared__ int pair_of[SHARED_MAX_TOKENS];
+  __shared__ int members[SHARED_MAX_TOKENS];
+  __shared__ int n_members;
+  __shared__ float sums[ACT == 0 ? 1 : 2][8][SHARED_TILE * 8];
+  pdl_trigger();
+  pdl_wait();
+  const int e = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (threadIdx.x < SHARED_MAX_TOKENS) pair_of[threadIdx.x] = -1;
+  __syncthreads();
+  for (int i = threadIdx.x; i < n_tokens * entries; i += blockDim.x)
+    if (idx[i] == e) pair_of[i / entries] = i;
+  __syncthreads();
+  if (warp == 0) {
+    const int mine = pair_of[lane];
+    const unsigned who = __ballot_sync(0xffffffffu, mine >= 0);
+    if (mine >= 0) members[__popc(who & ((1u << lane) - 1u))] = mine;
+    if (lane == 0) n_members = __popc(who);
+  }
+  __syncthreads();
+  const int count = n_members - (int)blockIdx.z * SHARED_TILE, f0 = blockIdx.x * 8;
+  if (count <= 0 || f0 >= (e < n_real ? F : Fs)) return;
+  const int* mem = members + blockIdx.z * SHARED_TILE;
+  const int g = lane >> 2, q = lane & 3;
+  const __nv_bfloat16* wg = w_up + ((size_t)e * F + f0 + g) * K + q * 8;
+  const __nv_bfloat16* wu = wg + up_rows * K;
+  const bool on0 = g < count, on1 = g + 8 < count;
+  const __nv_bfloat16* h0 = h + (size_t)(on0 ? mem[g] / entries : 0) * K + q * 8;
+  const __nv_bfloat16* h1 = h + (size_t)(on1 ? mem[g + 8] / entries : 0) * K + q * 8;
+  float dg[4] = {0.f, 0.f, 0.f, 0.f}, du[4] = {0.f, 0.f, 0.f, 0.f};
+  constexpr int U = 4;  // runs asked for together
+  for (int k0 = warp * SHARED_K; k0 < K; k0 += U * 8 * SHARED_K) {
+    uint4 xg[U], xu[U], lo[U];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int k = k0 + u * 8 * SHARED_K;
+      xg[u] = load16(wg + k, k < K);
+      if (ACT != 0) xu[u] = load16(wu + k, k < K);
+      lo[u] = load16(h0 + k, k < K && on0);
+    }
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int k = k0 + u * 8 * SHARED_K;
+      const uint4 hi = load16(h1 + k, k < K && on1);
+      mma_k32(dg, lo[u], hi, xg[u]);
+      if (ACT != 0) mma_k32(du, lo[u], hi, xu[u]);
+    }
+  }
+#pragma unroll
+  for (int c = 0; c < 4; ++c) {
+    const int at = (g + (c >> 1) * 8) * 8 + q * 2 + (c & 1);
+    sums[0][warp][at] = dg[c];
+    if (ACT != 0) sums[ACT == 0 ? 0 : 1][warp][at] = du[c];
+  }
+  __syncthreads();
+  const int m = threadIdx.x >> 3;
+  if (m >= SHARED_TILE || m >= count) return;
+  float x = 0.f, y = 0.f;
+#pragma unroll
+  for (int k = 0; k < 8; ++k) {
+    x += sums[0][k][threadIdx.x];
+    if (ACT != 0) y += sums[ACT == 0 ? 0 : 1][k][threadIdx.x];
+  }
+  float v;
+  if (ACT == 0) { v = fmaxf(x, 0.f); v = v * v; }
+  else if (ACT == 1) v = x / (1.f + expf(-x)) * y;
+  else v = capped_unit(x, y, e == n_real ? unit.limit_s : unit.limit, unit.alpha);
+  const int pair = mem[m];
+  a[(size_t)pair * lda + f0 + (threadIdx.x & 7)] = __float2bfloat16_rn(v * wts[pair]);
+}
+
+// Block (x, y): eight output columns for the sixteen tokens from 16 y on. W_down's columns are dealt to the eight warps in
+// runs of 32 by their place in the row (so a token's sum does not depend on which experts others chose); a chosen
+// expert's columns are read once. The warps' sums are added in order.
+__global__ void __launch_bounds__(256)
+moe_down_shared_kernel(const __nv_bfloat16* __restrict__ a, int lda, const __nv_bfloat16* __restrict__ w_down,
+                       const int* __restrict__ idx, float* __restrict__ y, int store, int n_tokens, int entries, int F, int Fs,
+                       int ld, int N, int n_real) {
+  __shared__ short pair_of[SHARED_MAX_EXPERTS][SHARED_TILE];
+  __shared__ int chosen[SHARED_MAX_EXPERTS];
+  __shared__ float sums[8][SHARED_TILE * 8];
+  pdl_trigger();
+  pdl_wait();
+  const int t0 = blockIdx.y * SHARED_TILE, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int nt = n_tokens - t0 < SHARED_TILE ? n_tokens - t0 : SHARED_TILE;
+  const int n_experts = n_real + (Fs > 0 ? 1 : 0);
+  for (int i = threadIdx.x; i < n_experts * SHARED_TILE; i += blockDim.x) pair_of[i / SHARED_TILE][i % SHARED_TILE] = -1;
+  for (int i = threadIdx.x; i < n_experts; i += blockDim.x) chosen[i] = 0;
+  __syncthreads();
+  for (int i = threadIdx.x; i < nt * entries; i += blockDim.x) {
+    const int e = idx[t0 * entries + i];
+    if (e < n_experts) { pair_of[e][i / entries] = (short)(t0 * entries + i); chosen[e] = 1; }
+  }
+  __syncthreads();
+  const int g = lane >> 2, q = lane & 3, o0 = blockIdx.x * 8;
+  const int row = o0 + g < N ? o0 + g : N - 1;  // (rows past the last are not stored)
+  float d[4] = {0.f, 0.f, 0.f, 0.f};
+  for (int e = 0; e < n_experts; ++e) {
+    if (!chosen[e]) continue;
+    const int n = e < n_real ? F : Fs, first = (e * F / SHARED_K) & 7;  // the warp that has the expert's first run
+    const __nv_bfloat16* wr = w_down + (size_t)row * ld + (size_t)e * F + q * 8;
+    const int p0 = pair_of[e][g], p1 = pair_of[e][g + 8];
+    const __nv_bfloat16* a0 = a + (size_t)(p0 < 0 ? 0 : p0) * lda + q * 8;
+    const __nv_bfloat16* a1 = a + (size_t)(p1 < 0 ? 0 : p1) * lda + q * 8;
+    constexpr int U = 8;  // runs asked for together
+    for (int k0 = ((warp - first) & 7) * SHARED_K; k0 < n; k0 += U * 8 * SHARED_K) {
+      uint4 x[U], lo[U];
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const int k = k0 + u * 8 * SHARED_K;
+        x[u] = load16(wr + k, k < n);
+        lo[u] = load16(a0 + k, k < n && p0 >= 0);
+      }
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const int k = k0 + u * 8 * SHARED_K;
+        mma_k32(d, lo[u], load16(a1 + k, k < n && p1 >= 0), x[u]);
+      }
+    }
+  }
+#pragma unroll
+  for (int c = 0; c < 4; ++c) sums[warp][(g + (c >> 1) * 8) * 8 + q * 2 + (c & 1)] = d[c];
+  __syncthreads();
+  if (threadIdx.x < SHARED_TILE * 8) {
+    const int t = threadIdx.x >> 3, o = o0 + (threadIdx.x & 7);
+    float v = 0.f;
+#pragma unroll
+    for (int k = 0; k < 8; ++k) v += sums[k][threadIdx.x];
+    if (t < nt && o < N) {
+      float* at = y + (size_t)(t0 + t) * N + o;
+      *at = store ? v : *at + v;
+    }
+  }
+}
+
 }  // namespace
 
 CUCA_API int cuca_moe_max_experts() { return MAX_EXPERTS; }
@@ -472,6 +637,26 @@ CUCA_API int cuca_moe_sparse_act(const void* h, const void* w_up, const void* w_
   CUCA_REQUIRE(lda >= wide, "moe_sparse: rows of %d values do not hold %d", lda, wide);
   CUCA_REQUIRE(act >= 0 && act <= 2, "moe_sparse: unknown activation %d", act);
   const SparseUnit unit = {limit, limit_s, alpha};
+  const int n_experts = E + (Fs > 0 ? 1 : 0);
+  // bfloat16 tokens that may share experts, and sizes the tensor cores take: by expert, each weight row read once
+  auto even = [&](const void* p) { return ((uintptr_t)p & 15) == 0; };
+  if (dtype == CUCA_BF16 && T >= 2 && T <= SHARED_MAX_TOKENS && n_experts <= SHARED_MAX_EXPERTS && even(h) && even(w_up) &&
+      even(w_down) && even(a) && K % SHARED_K == 0 && F % SHARED_K == 0 && Fs % SHARED_K == 0 && lda % 8 == 0 && ld % 8 == 0) {
+    const int tiles = (T + SHARED_TILE - 1) / SHARED_TILE;
+    const dim3 grid(wide / 8, n_experts, tiles);
+#define UPS(ACT)                                                                                                    \
+  cuca_launch(moe_up_shared_kernel<ACT>, grid, dim3(256), 0, stream, true, (const __nv_bfloat16*)h,                 \
+              (const __nv_bfloat16*)w_up, idx, wts, (__nv_bfloat16*)a, lda, T, entries, F, Fs, K, E, (size_t)C, unit)
+    if (act == 0) UPS(0);
+    else if (act == 1) UPS(1);
+    else UPS(2);
+#undef UPS
+    CUCA_CHECK_LAUNCH("moe_up_shared");
+    cuca_launch(moe_down_shared_kernel, dim3((N + 7) / 8, tiles), dim3(256), 0, stream, true, (const __nv_bfloat16*)a, lda,
+                (const __nv_bfloat16*)w_down, idx, y, store, T, entries, F, Fs, ld, N, E);
+    CUCA_CHECK_LAUNCH("moe_down_shared");
+    return 0;
+  }
 #define UP(TT, ACT)                                                                                                 \
   cuca_launch(moe_up_sparse_kernel<TT, ACT>, dim3((wide + 7) / 8, T * entries), dim3(256), 0, stream, true,         \
               (const TT*)h, (const TT*)w_up, idx, wts, (TT*)a, lda, entries, F, Fs, K, E, (size_t)C, unit)

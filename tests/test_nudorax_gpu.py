@@ -221,9 +221,11 @@ def test_lightning_in_chunks_keeps_32_bit_precision(rt32, H, d, dv, offset):
     assert n_chunks == 1 + 1 + 2 + 1 + 4 + 1
     ops.lightning_chunked(proj, _f32(decay, dev), st, out, step, n_chunks, H, d, dv)
     got, new = out.cpu().numpy().reshape(want.shape), st.cpu().numpy()
+    def close(x, y):  # in the mean to 32-bit precision; a silu that falls between two 16-bit numbers may go either way
+        d = np.abs(x - y)
+        return np.sqrt(np.mean(d * d)) < 1e-4 * np.sqrt(np.mean(y * y)) and d.max() < 1e-3 * np.abs(y).max()
     for a in range(H):  # (every head by its own size: the one that never decays grows)
-        assert np.abs(got[:, a] - want[:, a]).max() < 3e-5 * np.abs(want[:, a]).max(), a
-        assert np.abs(new[:, a] - after[:, a]).max() < 3e-5 * np.abs(after[:, a]).max(), a
+        assert close(got[:, a], want[:, a]) and close(new[:, a], after[:, a]), a
     assert np.array_equal(new[[1, 7]], state[[1, 7]])  # slots of no request of the step
 
 
@@ -521,6 +523,10 @@ def test_grouped_experts_alone(rt32, mlp, E):
 
 
 @pytest.mark.parametrize("mlp, E", [(nu.moe(), 48), (nu.moe(ff=64, experts=33, top=5, groups=(11, 4)), 64), (nu.moe(ff=40, shared=None), 56),
+                                    # (sizes in steps of 32: few tokens go through the tensor-core form)
+                                    (nu.moe(ff=96, experts=8, groups=(4, 2), shared=(160, 2.0)), 96),
+                                    (nu.moe(ff=32, experts=20, top=5, groups=(5, 3), shared=None), 64),
+                                    (nu.moe(ff=64, experts=4, top=4, groups=(2, 2), shared=(32, 1.0)), 100 * 32),
                                     (nu.moe(ff=200, experts=8, top=2, groups=(4, 2), shared=(136, 2.0)), 512)])
 def test_grouped_experts_in_bfloat16(mlp, E):
     """Both forms in the serving precision, on the tokens whose choice is clear (rounding cannot change it): the last
@@ -534,7 +540,7 @@ def test_grouped_experts_in_bfloat16(mlp, E):
     r = mlp["router"]
     top, g = r["top"], r["groups"]
     rs = np.random.default_rng(E + 1)
-    for T in (7, 13, part.SPARSE_MAX_TOKENS, 200):
+    for T in (1, 2, 7, 13, 17, part.SPARSE_MAX_TOKENS, 200):
         f = nu.bf16_round(rs.normal(0, 1.5, (T, E)))
         want = pn.routed_ff(f, ws, "l0.mlp.", mlp)
         clear = np.zeros(T, dtype=bool)
@@ -544,10 +550,12 @@ def test_grouped_experts_in_bfloat16(mlp, E):
             sums = np.sort([sum(sorted(s[i * size:(i + 1) * size])[-2:]) for i in range(g["count"])])[::-1]
             chosen = pn.chosen_experts(s, r)
             rest = [s[e] for e in pn.chosen_experts(s, dict(r, top=g["keep"] * size)) if e not in chosen]
-            clear[t] = (sums[g["keep"] - 1] - sums[g["keep"]] > 0.01) and (not rest or s[chosen[-1]] - max(rest) > 0.01)
+            clear[t] = (g["keep"] == g["count"] or sums[g["keep"] - 1] - sums[g["keep"]] > 0.01) and (not rest or s[chosen[-1]] - max(rest) > 0.01)
         assert clear.sum() >= T // 4
         stream = rt.stream(torch.zeros(T, E, device=dev))  # few rows may leave slices pending on it
         part.forward(torch.tensor(f, dtype=torch.bfloat16, device=dev), stream, None)
+        if not clear.any():
+            continue
         assert np.abs(stream.data.cpu().numpy() - want)[clear].max() < 3e-2 * np.abs(want).max()
 
 
