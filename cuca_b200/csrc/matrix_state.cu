@@ -8,7 +8,7 @@
 //                     S <- f * S (rows) + (1 - f) v^T;  o = S^T q
 //   retention_scan  linear attention with one fixed decay per head and no denominator:
 //                     S <- decay S + k v^T;  o = S^T q
-//   lightning_scan  the same recurrence on q = silu(.), k = silu(.), v = silu(.)
+//   lightning_scan  the same recurrence on q = silu(.), k = silu(.), v = silu(.); lightning_step: for single tokens
 //   head_norm_gate  out = o / rms(o) per head, times a weight (or none), times sigmoid(gate) or silu(gate)
 // What does not depend on the state (unit vectors, decays, gates) is computed for all rows at once by a preparing
 // kernel, in place. A scan block then takes one (head, request, run of value columns) and walks the request's rows of
@@ -266,6 +266,69 @@ silu_columns_kernel(float* __restrict__ proj, int ld, int col0, int n, const int
     } else {
       *at *= sigmoidf_(*at);
     }
+  }
+}
+
+// A step in which every request brings one token: S <- decay[h] S + silu(k) silu(v)^T, o = S^T silu(q), with q, k, v the
+// columns of the request's row from col0 on. A warp takes COLS value columns; a lane holds R packs of V consecutive key
+// channels of each (32 V R >= d).
+template <int V, int R, int COLS>
+__global__ void __launch_bounds__(256)
+lightning_step_kernel(const float* __restrict__ proj, int ld, int col0, const float* __restrict__ decay,
+                      float* __restrict__ state, float* __restrict__ out, const int* __restrict__ req_row0,
+                      const int* __restrict__ req_count, const int* __restrict__ slots, int H, int d, int dv) {
+  struct alignas(4 * V) Pack { float v[V]; };
+  pdl_trigger();
+  pdl_wait();
+  const int h = blockIdx.x, rq = blockIdx.y;
+  const int slot = slots[rq];
+  if (slot < 0 || req_count[rq] <= 0) return;
+  const size_t row = req_row0[rq];
+  const int c0 = (blockIdx.z * 8 + (threadIdx.x >> 5)) * COLS, lane = threadIdx.x & 31;
+  if (c0 >= dv) return;
+  const float* pr = proj + row * ld + col0;
+  const float* qp = pr + (size_t)h * d;
+  const float* kp = qp + (size_t)H * d;
+  const float* vp = pr + (size_t)2 * H * d + (size_t)h * dv;
+  float* st = state + ((size_t)slot * H + h) * dv * d;
+  const float dec = decay[h];
+  Pack S[COLS][R], q[R], k[R];
+#pragma unroll
+  for (int c = 0; c < COLS; ++c)
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+      const int r = (lane + 32 * i) * V;
+      if (c0 + c < dv && r < d) S[c][i] = *reinterpret_cast<const Pack*>(st + (size_t)(c0 + c) * d + r);
+    }
+#pragma unroll
+  for (int i = 0; i < R; ++i) {
+    const int r = (lane + 32 * i) * V;
+    if (r < d) { q[i] = *reinterpret_cast<const Pack*>(qp + r); k[i] = *reinterpret_cast<const Pack*>(kp + r); }
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      q[i].v[j] = r < d ? q[i].v[j] * sigmoidf_(q[i].v[j]) : 0.f;
+      k[i].v[j] = r < d ? k[i].v[j] * sigmoidf_(k[i].v[j]) : 0.f;
+    }
+  }
+#pragma unroll
+  for (int c = 0; c < COLS; ++c) {
+    if (c0 + c >= dv) break;
+    const float x = vp[c0 + c], v = x * sigmoidf_(x);
+    float sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+      const int r = (lane + 32 * i) * V;
+      if (r < d) {
+#pragma unroll
+        for (int j = 0; j < V; ++j) {
+          S[c][i].v[j] = fmaf(dec, S[c][i].v[j], k[i].v[j] * v);
+          sum = fmaf(S[c][i].v[j], q[i].v[j], sum);
+        }
+        *reinterpret_cast<Pack*>(st + (size_t)(c0 + c) * d + r) = S[c][i];
+      }
+    }
+    sum = warp_sum(sum);
+    if (lane == 0) out[row * H * dv + (size_t)h * dv + c0 + c] = sum;
   }
 }
 
@@ -812,6 +875,27 @@ CUCA_API int cuca_lightning_scan(float* proj, int ld, int col0, const float* dec
   CUCA_CHECK_LAUNCH("silu_columns");
   return launch_decay_scan("lightning_scan", proj, ld, col0, col0 + H * d, col0 + 2 * H * d, decay, state, out, req_row0,
                            req_count, slots, n_seqs, H, d, dv, stream);
+}
+
+// The same for a step in which every request brings one token, in one launch; proj is only read.
+CUCA_API int cuca_lightning_step(const float* proj, int ld, int col0, const float* decay, float* state, float* out,
+                                 const int* req_row0, const int* req_count, const int* slots, int n_seqs, int H, int d,
+                                 int dv, cudaStream_t stream) {
+  if (n_seqs == 0) return 0;
+  CUCA_REQUIRE(H > 0 && d > 0 && dv > 0 && d <= 32 * MAXR, "lightning_step: bad sizes heads=%d dim=%d vdim=%d", H, d, dv);
+  CUCA_REQUIRE(n_seqs <= 65535, "lightning_step: %d requests exceed the launch limit", n_seqs);
+  const bool wide = d % 4 == 0 && ld % 4 == 0 && col0 % 4 == 0 && ((uintptr_t)proj & 15) == 0 && ((uintptr_t)state & 15) == 0;
+#define LS(V, R, COLS)                                                                                              \
+  cuca_launch(lightning_step_kernel<V, R, COLS>, dim3(H, n_seqs, (dv + 8 * COLS - 1) / (8 * COLS)), dim3(256), 0,   \
+              stream, true, proj, ld, col0, decay, state, out, req_row0, req_count, slots, H, d, dv)
+  if (wide && d <= 128) LS(4, 1, 4);
+  else if (wide && d <= 256) LS(4, 2, 4);
+  else if (wide) LS(4, 8, 1);
+  else if (d <= 128) LS(1, 4, 4);
+  else LS(1, 32, 1);
+#undef LS
+  CUCA_CHECK_LAUNCH("lightning_step");
+  return 0;
 }
 
 // gate_act 0: the gate's factor is sigmoid(gate); 1: silu(gate). w null: no weight.

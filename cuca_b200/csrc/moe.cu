@@ -155,17 +155,10 @@ __device__ __forceinline__ float capped_unit(float gate, float up, float limit, 
 // largest (of its one, where it has one); the `keep` best groups' experts can be chosen, the `top` largest of them are
 // (the lower number on a tie), with weights s * scale. Column E of a row of logits, where has_shared, belongs to a shared
 // expert that every token uses, with weight sigmoid(z): it becomes entry `top` of idx / wts (number E) and column E of
-// dense. A warp per token; lane l holds experts l, l + 32, ...
-__global__ void __launch_bounds__(128)
-moe_route_grouped_kernel(const float* __restrict__ logits, int T, int E, int groups, int keep, int top, float scale,
-                         int has_shared, int* __restrict__ idx, float* __restrict__ wts, float* __restrict__ dense) {
-  __shared__ float group_score[4][MAX_EXPERTS];
-  pdl_trigger();
-  pdl_wait();
-  const int warp = threadIdx.x >> 5, t = blockIdx.x * 4 + warp, lane = threadIdx.x & 31;
-  if (t >= T) return;
+// dense. One warp; lane l holds experts l, l + 32, ...; z: the token's logits, gs: shared memory for a score per group.
+__device__ void route_grouped(const float* z, float* gs, int t, int lane, int E, int groups, int keep, int top, float scale,
+                              int has_shared, int* __restrict__ idx, float* __restrict__ wts, float* __restrict__ dense) {
   const int n_out = E + (has_shared ? 1 : 0), entries = top + (has_shared ? 1 : 0);
-  const float* z = logits + (size_t)t * n_out;
   auto score = [&](int e) {  // (a row of padding may hold anything: every lane must still see one order)
     const float v = z[e];
     return v == v ? 1.f / (1.f + expf(-v)) : -1.f;
@@ -173,7 +166,6 @@ moe_route_grouped_kernel(const float* __restrict__ logits, int T, int E, int gro
   unsigned open = 0xffffffffu;  // bit k: this lane's expert lane + 32 k can be chosen
   if (groups > 1 && keep < groups) {
     const int size = E / groups;
-    float* gs = group_score[warp];
     if (size <= 32) {  // a lane per group
       for (int g = lane; g < groups; g += 32) {
         float a = -INFINITY, b = -INFINITY;
@@ -245,6 +237,18 @@ moe_route_grouped_kernel(const float* __restrict__ logits, int T, int E, int gro
     wts[(size_t)t * entries + top] = sw;
     if (dense) dense[(size_t)t * n_out + E] = sw;
   }
+}
+
+__global__ void __launch_bounds__(128)
+moe_route_grouped_kernel(const float* __restrict__ logits, int T, int E, int groups, int keep, int top, float scale,
+                         int has_shared, int* __restrict__ idx, float* __restrict__ wts, float* __restrict__ dense) {
+  __shared__ float group_score[4][MAX_EXPERTS];
+  pdl_trigger();
+  pdl_wait();
+  const int warp = threadIdx.x >> 5, t = blockIdx.x * 4 + warp;
+  if (t >= T) return;
+  route_grouped(logits + (size_t)t * (E + (has_shared ? 1 : 0)), group_score[warp], t, threadIdx.x & 31, E, groups, keep, top,
+                scale, has_shared, idx, wts, dense);
 }
 
 // gu: [T, 2 C] (gates, then ups); a[t, c] = capped_unit(g, u) w; c < EF: expert c / F's columns, w = dense[t, c / F] and
@@ -377,6 +381,24 @@ __device__ __forceinline__ float warp_dot(const __nv_bfloat16* w, const __nv_bfl
 struct SparseUnit {
   float limit, limit_s, alpha;  // ACT 2: the caps of the experts and of the shared expert
 };
+
+// Few tokens and few experts: the router's logits (32-bit sums) and the choice in one launch, a block per token.
+constexpr int ROUTER_MAX_OUTPUTS = 64;
+template <typename T>
+__global__ void __launch_bounds__(512)
+moe_router_grouped_kernel(const T* __restrict__ h, const T* __restrict__ w, int K, int E, int groups, int keep, int top,
+                          float scale, int has_shared, int* __restrict__ idx, float* __restrict__ wts) {
+  __shared__ float z[ROUTER_MAX_OUTPUTS], group_score[ROUTER_MAX_OUTPUTS];
+  pdl_trigger();
+  pdl_wait();
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_out = E + (has_shared ? 1 : 0);
+  for (int e = warp; e < n_out; e += 16) {
+    const float v = warp_dot(w + (size_t)e * K, h + (size_t)t * K, K, lane);
+    if (lane == 0) z[e] = v;
+  }
+  __syncthreads();
+  if (warp == 0) route_grouped(z, group_score, t, lane, E, groups, keep, top, scale, has_shared, idx, wts, nullptr);
+}
 
 // a[pair, f] = act(W[e(pair)] . h[t]) * weight(pair); pair = t * entries + j. ACT 0: W_up [E F, K]. ACT 1 and 2: w_up
 // holds every expert's gate rows and, `up_rows` rows further on, its up rows. Entry number n_real is the shared expert
@@ -699,6 +721,27 @@ CUCA_API int cuca_moe_route_grouped(const float* logits, int T, int E, int group
   cuca_launch(moe_route_grouped_kernel, dim3((T + 3) / 4), dim3(128), 0, stream, true, logits, T, E, groups, keep, top,
               scale, has_shared, idx, wts, dense);
   CUCA_CHECK_LAUNCH("moe_route_grouped");
+  return 0;
+}
+
+// The same from the activations: h [T, K], router weights w [E (+ 1), K] of one dtype; up to 64 outputs.
+CUCA_API int cuca_moe_router_grouped(const void* h, const void* w, int dtype, int T, int K, int E, int groups, int keep,
+                                     int top, float scale, int has_shared, int* idx, float* wts, cudaStream_t stream) {
+  if (T == 0) return 0;
+  CUCA_REQUIRE(E >= 1 && E + (has_shared ? 1 : 0) <= ROUTER_MAX_OUTPUTS && top >= 1 && top <= MAX_TOP,
+               "moe_router: %d of %d experts is outside what the kernel takes (outputs <= %d, chosen <= %d)", top, E,
+               ROUTER_MAX_OUTPUTS, MAX_TOP);
+  CUCA_REQUIRE(groups >= 1 && E % groups == 0 && keep >= 1 && keep <= groups && top <= keep * (E / groups),
+               "moe_router: %d of the %d experts in %d of %d groups cannot be chosen", top, E, keep, groups);
+  if (dtype == CUCA_F32)
+    cuca_launch(moe_router_grouped_kernel<float>, dim3(T), dim3(512), 0, stream, true, (const float*)h, (const float*)w, K, E,
+                groups, keep, top, scale, has_shared, idx, wts);
+  else if (dtype == CUCA_BF16)
+    cuca_launch(moe_router_grouped_kernel<__nv_bfloat16>, dim3(T), dim3(512), 0, stream, true, (const __nv_bfloat16*)h,
+                (const __nv_bfloat16*)w, K, E, groups, keep, top, scale, has_shared, idx, wts);
+  else
+    CUCA_REQUIRE(false, "moe_router: unknown dtype %d", dtype);
+  CUCA_CHECK_LAUNCH("moe_router_grouped");
   return 0;
 }
 

@@ -145,6 +145,7 @@ _SIGNATURES = {
                             _P, _P],
     "cuca_head_norm_gate_act": [_P, _P, _I, _P, _I, _I, _I, _P, _I, _I, _I, _I, _F, _P],
     "cuca_lightning_scan": [_P, _I, _I, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P],
+    "cuca_lightning_step": [_P, _I, _I, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _P],
     "cuca_max_terms": [],
     "cuca_norm_add": [_P, _P, _P, _P, _I, _I, _I, _F, _I, _P],
     "cuca_layer_norm": [_P, _P, _P, _I, _P, _I, _I, _F, _P],
@@ -156,6 +157,7 @@ _SIGNATURES = {
     "cuca_lightning_chunked": [_P, _I, _I, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P],
     "cuca_moe_sparse_act": [_P, _P, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _P],
     "cuca_moe_route_grouped": [_P, _I, _I, _I, _I, _I, _F, _I, _P, _P, _P, _P],
+    "cuca_moe_router_grouped": [_P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P, _P, _P],
     "cuca_moe_glu_capped_dense": [_P, _P, _I, _P, _I, _I, _I, _I, _I, _F, _F, _F, _P],
 }
 

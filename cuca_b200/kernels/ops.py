@@ -1047,8 +1047,13 @@ def retention_scan(proj, q_col, k_col, v_col, decay, cos, sin, rot_dims, k_scale
 def lightning_scan(proj, decay, state, out, step, H, d, dv) -> None:
     """Lightning attention along every request's rows: the recurrence of retention on silu(q), silu(k), silu(v) (see
     `parts/recurrent.py:Lightning`). The first H (2 d + dv) columns of the 32-bit `proj` hold q, k, v before their
-    activation and are rewritten in place; two launches."""
+    activation and may be rewritten in place; two launches, or one where every request brings a single token."""
     _cuda(proj, decay, state, out)
+    if step.all_single():
+        library.check(library.load().cuca_lightning_step(
+            _p(proj), proj.stride(0), 0, _p(decay), _p(state), _p(out), _p(step.req_row0), _p(step.req_count),
+            _p(step.slots), step.n_seqs, H, d, dv, _stream()), "lightning_step")
+        return
     library.check(library.load().cuca_lightning_scan(
         _p(proj), proj.stride(0), 0, _p(decay), _p(state), _p(out), _p(step.seq_of_row), _p(step.req_row0),
         _p(step.req_count), _p(step.slots), proj.shape[0], step.n_seqs, H, d, dv, _stream()), "lightning_scan")
@@ -1160,6 +1165,17 @@ def moe_route_grouped(logits, experts: int, groups: int, keep: int, top: int, sc
     library.check(library.load().cuca_moe_route_grouped(
         _p(logits), logits.shape[0], int(experts), int(groups), int(keep), int(top), float(scale), int(bool(shared)),
         _p(idx), _p(wts), _p(dense), _stream()), "moe_route_grouped")
+
+
+MOE_ROUTER_MAX_OUTPUTS = 64
+
+
+def moe_router_grouped(h, w, experts: int, groups: int, keep: int, top: int, scale: float, shared: bool, idx, wts) -> None:
+    """`moe_route_grouped` from the activations h and the router's rows w (up to `MOE_ROUTER_MAX_OUTPUTS`), one launch."""
+    _cuda(h, w, idx, wts)
+    library.check(library.load().cuca_moe_router_grouped(
+        _p(h), _p(w), dtype_code(h.dtype), h.shape[0], h.shape[1], int(experts), int(groups), int(keep), int(top),
+        float(scale), int(bool(shared)), _p(idx), _p(wts), _stream()), "moe_router_grouped")
 
 
 def moe_sparse_capped(h, w_gu, w_down, idx, wts, a, y, store, E: int, F: int, Fs: int, limit: float, limit_s: float,

@@ -435,14 +435,17 @@ class GroupedExperts(FeedForward):
     def forward(self, h, stream, step) -> None:
         rt, T = self.rt, h.shape[0]
         stream = rt.stream(stream)
-        logits = rt.linear(h, self.w_router, out_dtype=torch.float32)  # [experts | the shared one's weight]
         entries = self.top + (1 if self.shared else 0)
         idx = torch.empty(T, entries, dtype=torch.int32, device=rt.device)
         wts = torch.empty(T, entries, dtype=torch.float32, device=rt.device)
         few = T <= self.SPARSE_MAX_TOKENS
-        spread = None if few else torch.empty(T, logits.shape[1], dtype=torch.float32, device=rt.device)
-        ops.moe_route_grouped(logits, self.experts, self.groups, self.keep, self.top, self.scale, self.shared > 0, idx,
-                              wts, spread)
+        choice = (self.experts, self.groups, self.keep, self.top, self.scale, self.shared > 0)
+        if few and self.w_router.shape[0] <= ops.MOE_ROUTER_MAX_OUTPUTS:
+            ops.moe_router_grouped(h, self.w_router, *choice, idx, wts)
+        else:
+            logits = rt.linear(h, self.w_router, out_dtype=torch.float32)  # [experts | the shared one's weight]
+            spread = None if few else torch.empty_like(logits)
+            ops.moe_route_grouped(logits, *choice, idx, wts, spread)
         if few:
             a = rt.empty(T * entries, max(self.inner, self.shared))
             y, fresh = stream.claim()

@@ -570,14 +570,19 @@ def test_rows_of_padding_may_hold_anything(rt32):
     z[2], z[5, 3], z[7] = np.nan, np.nan, np.inf
     bad = torch.tensor(z, device=dev)
     outs = []
-    for logits in (clean, bad):
+    eye = torch.eye(E + 1, device=dev)  # (the form that makes the logits itself: they are the activations' own entries)
+    for few, logits in ((False, clean), (False, bad), (True, clean)):
         idx = torch.empty(T, 4, dtype=torch.int32, device=dev)
         wts = torch.empty(T, 4, dtype=torch.float32, device=dev)
-        ops.moe_route_grouped(logits, E, 3, 2, 3, 2.0, True, idx, wts)
+        if few:
+            ops.moe_router_grouped(logits, eye, E, 3, 2, 3, 2.0, True, idx, wts)
+        else:
+            ops.moe_route_grouped(logits, E, 3, 2, 3, 2.0, True, idx, wts)
         outs.append((idx.cpu().numpy(), wts.cpu().numpy()))
     assert ((outs[1][0] >= 0) & (outs[1][0] <= E)).all() and (outs[1][0][:, 3] == E).all()
     for t in (0, 1, 3, 4, 6, 8):
         assert (outs[0][0][t] == outs[1][0][t]).all() and (outs[0][1][t] == outs[1][1][t]).all()
+    assert (outs[0][0] == outs[2][0]).all() and (outs[0][1] == outs[2][1]).all()
     for t in range(T):  # no expert twice
         assert len(set(outs[1][0][t].tolist())) == 4
 
