@@ -72,6 +72,12 @@ struct Params {
   // the gated epilogue: limit = 0: silu(g) u; limit > 0: g' sigmoid(alpha g') (u' + 1), g' = min(g, limit),
   // u' = clamp(u, -limit, limit); limit < 0: gelu(g) u with the tanh form of gelu
   float glu_limit, glu_alpha;
+  // with col_w (32-bit [M, ld_w]): output column n of token m is multiplied by col_w[m, n / w_run] (n < w_cols), or, behind
+  // w_cols, by col_w[m, w_cols / w_run] with cap glu_limit_s: experts of w_run columns each and a shared one. w_run and
+  // w_cols are multiples of 16
+  const float* col_w;
+  int ld_w, w_run, w_cols;
+  float glu_limit_s;
 };
 
 constexpr int STAGING_BUF = 32 * 128;  // 32 rows of 128 bytes
@@ -197,13 +203,25 @@ struct SegmentWalk {
 // for a numerator of zero, which is what every padded row or column of a tile holds, and a warp then pays the slow
 // path for all its lanes (measured: SwiGLU over 255 tokens took 76.7 us, over 256 tokens 63.1).
 __device__ __forceinline__ float silu_mul(float g, float u) { return __fdividef(g, 1.f + __expf(-g)) * u; }
-__device__ __forceinline__ float glu_act(const Params& p, float g, float u) {
-  if (p.glu_limit > 0.f) {
-    g = fminf(g, p.glu_limit);
-    u = fminf(fmaxf(u, -p.glu_limit), p.glu_limit);
-    return __fdividef(g, 1.f + __expf(-p.glu_alpha * g)) * (u + 1.f);
+// What the gated epilogue needs of an output column (or of sixteen from a multiple of 16 on) of one token: the cap and the
+// factor on the result.
+struct GluAt { float limit, weight; };
+__device__ __forceinline__ GluAt glu_at(const Params& p, int m, int n) {
+  GluAt at = {p.glu_limit, 1.f};
+  if (p.col_w && m < p.M && n < p.N) {
+    const bool shared = n >= p.w_cols;
+    if (shared) at.limit = p.glu_limit_s;
+    at.weight = __ldg(p.col_w + (size_t)m * p.ld_w + (shared ? p.w_cols : n) / p.w_run);
   }
-  if (p.glu_limit < 0.f) {
+  return at;
+}
+__device__ __forceinline__ float glu_act(const Params& p, const GluAt& at, float g, float u) {
+  if (at.limit > 0.f) {
+    g = fminf(g, at.limit);
+    u = fminf(fmaxf(u, -at.limit), at.limit);
+    return __fdividef(g, 1.f + __expf(-p.glu_alpha * g)) * (u + 1.f) * at.weight;
+  }
+  if (at.limit < 0.f) {
     // 0.5 g (1 + tanh(y)) = g sigmoid(2 y) with y = sqrt(2/pi) (g + 0.044715 g^3)
     const float y2 = 1.5957691216057308f * (g + 0.044715f * g * g * g);
     return __fdividef(g, 1.f + __expf(-y2)) * u;
@@ -225,7 +243,7 @@ __device__ __forceinline__ void store16(const Params& p, int a0, int b0, int lan
       const int m = b0 + c + j;
       if (m >= p.M) break;
       const size_t o = (size_t)m * p.ldo + n;
-      if (DUAL) ((__nv_bfloat16*)p.out)[o] = __float2bfloat16_rn(glu_act(p, v[j], u[j]));
+      if (DUAL) ((__nv_bfloat16*)p.out)[o] = __float2bfloat16_rn(glu_act(p, glu_at(p, m, n), v[j], u[j]));
       else if (p.epilogue == EPI_RESIDUAL) atomicAdd((float*)p.out + o, v[j] + bias);  // result unused: a fire-and-forget
                                                                                        // add; one thread owns the element
       else if (p.out_f32) ((float*)p.out)[o] = v[j] + bias;
@@ -238,8 +256,10 @@ __device__ __forceinline__ void store16(const Params& p, int a0, int b0, int lan
     const int n = b0 + c;
     if (n >= p.N) return;
     float r[16];
+    GluAt at = {0.f, 1.f};
+    if (DUAL) at = glu_at(p, m, n);
 #pragma unroll
-    for (int j = 0; j < 16; ++j) r[j] = DUAL ? glu_act(p, v[j], u[j]) : v[j];
+    for (int j = 0; j < 16; ++j) r[j] = DUAL ? glu_act(p, at, v[j], u[j]) : v[j];
     const size_t o = (size_t)m * p.ldo + n;
     const bool full = n + 16 <= p.N;
     if (!DUAL && p.bias) {
@@ -313,8 +333,9 @@ __device__ __forceinline__ void tma_epilogue(const Params& p, const CUtensorMap*
       if (DUAL) {
         float u[16];
         tmem_ld16(acc + 128 + c + h, u);
+        const GluAt at = glu_at(p, y0 + lane, b0 + c + h);
 #pragma unroll
-        for (int j = 0; j < 16; ++j) v[j] = glu_act(p, v[j], u[j]);
+        for (int j = 0; j < 16; ++j) v[j] = glu_act(p, at, v[j], u[j]);
       } else if (p.bias && with_bias) {
 #pragma unroll
         for (int j = 0; j < 16; ++j)
@@ -1084,7 +1105,8 @@ CUCA_API void cuca_gemm_pair_mode(int mode) { allow_pair = mode; }
 static int gemm_tc_impl(const void* A, const void* W, const void* bias, void* out, int out_dtype, int M, int N,
                         int K, int lda, int ldo, int epilogue, void* workspace, size_t ws_bytes, int* counters,
                         int n_counters, int max_splits, int* n_slices_out, int* err, cudaStream_t stream,
-                        float glu_limit = 0.f, float glu_alpha = 1.f) {
+                        float glu_limit = 0.f, float glu_alpha = 1.f, const float* col_w = nullptr, int ld_w = 0,
+                        int w_run = 16, int w_cols = 0, float glu_limit_s = 0.f) {
   if (M == 0 || N == 0) return 0;
   if (!cuca_gemm_tc_supported(A, W, M, N, K, lda)) return 1;
   CUCA_REQUIRE(epilogue != EPI_RESIDUAL || out_dtype == CUCA_F32, "gemm_tc: the residual stream is 32-bit");
@@ -1103,6 +1125,7 @@ static int gemm_tc_impl(const void* A, const void* W, const void* bias, void* ou
     p.out = out; p.bias = nullptr; p.workspace = nullptr; p.counters = nullptr; p.err = err;
     p.M = M; p.N = N; p.K = K; p.ldo = N; p.epilogue = EPI_PARTIAL; p.out_f32 = 1;
     p.glu_limit = 0.f; p.glu_alpha = 1.f;
+    p.col_w = nullptr; p.ld_w = p.w_cols = 0; p.w_run = 16; p.glu_limit_s = 0.f;
     p.tile_rows = 2 * TILE_A;
     p.tiles_a = (M + 255) / 256;
     p.tiles = p.tiles_a * ((N + 255) / 256);
@@ -1134,6 +1157,7 @@ static int gemm_tc_impl(const void* A, const void* W, const void* bias, void* ou
   if (!tma_out) tmO = tmA;  // unused
   Params p;
   p.glu_limit = glu_limit; p.glu_alpha = glu_alpha;
+  p.col_w = col_w; p.ld_w = ld_w; p.w_run = w_run; p.w_cols = w_cols; p.glu_limit_s = glu_limit_s;
   p.out = out; p.bias = (const __nv_bfloat16*)bias; p.workspace = (float*)workspace; p.counters = counters;
   p.err = err; p.M = M; p.N = N; p.K = K; p.ldo = ldo; p.epilogue = epilogue; p.out_f32 = out_dtype == CUCA_F32;
   const int out_cols = swap ? bn : (dual ? 128 : 256);
@@ -1311,6 +1335,19 @@ CUCA_API int cuca_gemm_tc_glu(const void* A, const void* W, void* out, int M, in
                       n_counters, max_splits, nullptr, err, stream, limit, alpha);
 }
 
+// The capped epilogue for routed experts, w_run output columns each (w_cols in all), and behind them a shared expert's
+// columns: column n of token m times weights[m, n / w_run], the shared one's times weights[m, w_cols / w_run] with its own
+// cap. weights: 32-bit rows of ld_w values.
+CUCA_API int cuca_gemm_tc_glu_experts(const void* A, const void* W, void* out, int M, int N, int K, int lda, int ldo,
+                                      float limit, float limit_s, float alpha, const float* weights, int ld_w, int w_run,
+                                      int w_cols, void* workspace, size_t ws_bytes, int* counters, int n_counters,
+                                      int max_splits, int* err, cudaStream_t stream) {
+  CUCA_REQUIRE(limit > 0.f && limit_s > 0.f, "gemm_tc_glu_experts: the caps %g and %g must be positive", (double)limit, (double)limit_s);
+  CUCA_REQUIRE(weights && w_run >= 16 && w_run % 16 == 0 && w_cols % w_run == 0 && w_cols <= N &&
+               w_cols / w_run + (N > w_cols ? 1 : 0) <= ld_w, "gemm_tc_glu_experts: %d columns in runs of %d, %d in all, %d weights", w_cols, w_run, N, ld_w);
+  return gemm_tc_impl(A, W, nullptr, out, CUCA_BF16, M, N, K, lda, ldo, EPI_SWIGLU, workspace, ws_bytes, counters,
+                      n_counters, max_splits, nullptr, err, stream, limit, alpha, weights, ld_w, w_run, w_cols, limit_s);
+}
 
 // The gated epilogue with a chosen activation: act 0: silu(g) u, 1: gelu(g) u with the tanh form of gelu,
 // 0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3))).

@@ -269,7 +269,7 @@ bool terms_wide(const CucaTerms& t) {
 // threads and held packs for rows of `packs` packs: few rows get as many threads as a row has packs, many rows a
 // quarter of that with four packs each
 void norm_shape(int packs, int n_rows, int* threads, int* held) {
-  int r = n_rows >= 512 && packs > 128 ? 4 : 1;
+  int r = n_rows >= 512 && packs > 1024 ? 2 : 1;
   while (r < 8 && (packs + r - 1) / r > 1024) r *= 2;
   if ((packs + r - 1) / r > 1024) { *threads = 1024; *held = 0; return; }
   *threads = ((packs + r - 1) / r + 31) / 32 * 32;

@@ -158,6 +158,8 @@ _SIGNATURES = {
     "cuca_moe_sparse_act": [_P, _P, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _P],
     "cuca_moe_route_grouped": [_P, _I, _I, _I, _I, _I, _F, _I, _P, _P, _P, _P],
     "cuca_moe_router_grouped": [_P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P, _P, _P],
+    "cuca_gemm_tc_glu_experts": [_P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _F, _P, _I, _I, _I, _P, c_size_t, _P, _I, _I, _P,
+                                 _P],
     "cuca_moe_glu_capped_dense": [_P, _P, _I, _P, _I, _I, _I, _I, _I, _F, _F, _F, _P],
 }
 

@@ -238,6 +238,20 @@ def gemm_tc_glu_act(a, w, out, act: int, err=None, max_splits=16) -> None:
                                            int(max_splits), _p(err), _stream()), "gemm_tc_glu_act")
 
 
+def gemm_tc_glu_experts(a, w, out, weights, run: int, cols: int, limit: float, limit_s: float, alpha: float, err=None,
+                        max_splits=16) -> None:
+    """`gemm_tc_glu` for routed experts of `run` output columns each (`cols` in all, `run` a multiple of 16) and a shared
+    expert behind them: column n of row m times weights[m, n // run]; the shared one's times weights[m, cols // run], with
+    cap `limit_s`."""
+    _cuda(a, w, out, weights)
+    M, K = a.shape
+    ws, counters = gemm_scratch(a.device)
+    library.check(library.load().cuca_gemm_tc_glu_experts(
+        _p(a), _p(w), _p(out), M, out.shape[1], K, a.stride(0), out.stride(0), float(limit), float(limit_s), float(alpha),
+        _p(weights), weights.stride(0), int(run), int(cols), _p(ws), ws.numel() * 4, _p(counters), counters.numel(),
+        int(max_splits), _p(err), _stream()), "gemm_tc_glu_experts")
+
+
 def gemm_pair_mode(mode: int) -> None:
     """When contractions over many tokens run as pairs of CTAs on one tile (`tcgen05.mma.cta_group::2`): 1 where
     the library's rule expects them to be faster, 0 never, 2 wherever they can (tests and measurements), -1 as the

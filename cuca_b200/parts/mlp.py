@@ -378,6 +378,10 @@ class GroupedExperts(FeedForward):
     shared_weight [1, width]."""
 
     graph_safe = True
+    # From this width on the units and their weights are the gate/up contraction's epilogue. Measured on prompts of 2,048
+    # tokens, six layers: width 2048 5.00 ms with a pass of its own against 5.11 (a tile's main loop is too short to hide
+    # the epilogue's exponentials), 3072 6.41 against 6.35, 4096 11.4 against 10.97.
+    FUSED_FROM_WIDTH = 2560
     SPARSE_MAX_TOKENS = 32  # up to this many tokens only the chosen experts are read
 
     def __init__(self, spec, runtime):
@@ -452,8 +456,14 @@ class GroupedExperts(FeedForward):
             ops.moe_sparse_capped(h, self.w_gu, self.w_down, idx, wts, a, y, fresh, self.experts, self.inner, self.shared,
                                   self.limit, self.shared_limit, self.alpha)
             return
-        gu = rt.linear(h, self.w_gu)
         a = rt.empty(T, self.w_down.shape[1])
-        ops.moe_glu_capped_dense(gu, spread, a, self.experts * self.inner, self.inner, self.limit, self.shared_limit,
-                                 self.alpha)
+        EF = self.experts * self.inner
+        if (h.dtype == torch.bfloat16 and self.inner % 16 == 0 and self.width >= self.FUSED_FROM_WIDTH
+                and ops.gemm_tc_supported(h, self.w_gu)):
+            # the units and their weights are the contraction's epilogue, from the 32-bit sums
+            ops.gemm_tc_glu_experts(h, self.w_gu, a, spread, self.inner, EF, self.limit, self.shared_limit, self.alpha,
+                                    rt.err)
+        else:
+            gu = rt.linear(h, self.w_gu)
+            ops.moe_glu_capped_dense(gu, spread, a, EF, self.inner, self.limit, self.shared_limit, self.alpha)
         stream.add_linear(a, self.w_down)

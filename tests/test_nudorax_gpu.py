@@ -528,19 +528,21 @@ def test_grouped_experts_alone(rt32, mlp, E):
                                     (nu.moe(ff=32, experts=20, top=5, groups=(5, 3), shared=None), 64),
                                     (nu.moe(ff=64, experts=4, top=4, groups=(2, 2), shared=(32, 1.0)), 100 * 32),
                                     (nu.moe(ff=200, experts=8, top=2, groups=(4, 2), shared=(136, 2.0)), 512)])
-def test_grouped_experts_in_bfloat16(mlp, E):
-    """Both forms in the serving precision, on the tokens whose choice is clear (rounding cannot change it): the last
+@pytest.mark.parametrize("fused", [False, True])
+def test_grouped_experts_in_bfloat16(monkeypatch, mlp, E, fused):
+    """Few tokens and many (the units in a pass of their own and as the contraction's epilogue) in the serving precision, on the tokens whose choice is clear (rounding cannot change it): the last
     chosen score well above the first open one left, the last kept group's sum well above the next one's."""
     from cuca_b200.runtime import Runtime
     rt = Runtime("cuda:0", torch.bfloat16)
     dev = rt.device
     part = _grouped(mlp, E, rt)
+    monkeypatch.setattr(type(part), "FUSED_FROM_WIDTH", 0 if fused else 1 << 30)
     ws = _weights_for(part, E, rounded=True)
     _load_as(part, ws, rt)
     r = mlp["router"]
     top, g = r["top"], r["groups"]
     rs = np.random.default_rng(E + 1)
-    for T in (1, 2, 7, 13, 17, part.SPARSE_MAX_TOKENS, 200):
+    for T in ((40, 200, 300) if fused else (1, 2, 7, 13, 17, part.SPARSE_MAX_TOKENS, 40, 200)):
         f = nu.bf16_round(rs.normal(0, 1.5, (T, E)))
         want = pn.routed_ff(f, ws, "l0.mlp.", mlp)
         clear = np.zeros(T, dtype=bool)
