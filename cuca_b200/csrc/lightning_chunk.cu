@@ -248,8 +248,9 @@ chunk_carry_kernel(const Args p) {
   *reinterpret_cast<Pack*>(st) = s;
 }
 
-// out rows of the chunk, CW value columns of head h. Four warps of 16 tokens each. dp: d rounded up to 16.
-__global__ void __launch_bounds__(128)
+// out rows of the chunk, CW value columns of head h. Eight warps: 16 tokens and half of the columns each (both halves work
+// the scores of their tokens out: the blocks are bound by latency, not by products). dp: d rounded up to 16.
+__global__ void __launch_bounds__(256)
 chunk_output_kernel(const Args p, int dp) {
   extern __shared__ __align__(16) unsigned char raw[];
   __shared__ float pw[C + 1];
@@ -305,14 +306,14 @@ chunk_output_kernel(const Args p, int dp) {
   }
   stage_powers(pw, p.decay[h]);
   __syncthreads();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, mi = lane >> 3, li = lane & 7;
+  const int warp = (threadIdx.x >> 5) & 3, half_no = threadIdx.x >> 7, lane = threadIdx.x & 31, mi = lane >> 3, li = lane & 7;
   const int i0 = warp * 16 + (lane >> 2);  // this thread's rows: i0 and i0 + 8
   if (warp * 16 >= n) return;
-  float o[8][4], s[8][4];
+  float o[4][4], s[8][4];
 #pragma unroll
   for (int t = 0; t < 8; ++t)
 #pragma unroll
-    for (int k = 0; k < 4; ++k) { o[t][k] = 0.f; s[t][k] = 0.f; }
+    for (int k = 0; k < 4; ++k) { o[t & 3][k] = 0.f; s[t][k] = 0.f; }
   for (int kk = 0; kk < dp / 16; ++kk) {
     uint32_t a[4];
     ldsm4(a, sq + (warp * 16 + (mi & 1) * 8 + li) * pitch + kk * 16 + (mi >> 1) * 8);
@@ -320,12 +321,15 @@ chunk_output_kernel(const Args p, int dp) {
     for (int np = 0; np < 4; ++np) {
       uint32_t b[4];
       const int at = (np * 16 + (mi >> 1) * 8 + li) * pitch + kk * 16 + (mi & 1) * 8;
-      ldsm4(b, ss_hi + at);
-      mma16816(o[2 * np], a, b[0], b[1]);
-      mma16816(o[2 * np + 1], a, b[2], b[3]);
-      ldsm4(b, ss_lo + at);
-      mma16816(o[2 * np], a, b[0], b[1]);
-      mma16816(o[2 * np + 1], a, b[2], b[3]);
+      if (np < 2) {
+        const int col = at + half_no * 32 * pitch;
+        ldsm4(b, ss_hi + col);
+        mma16816(o[(2 * np) & 3], a, b[0], b[1]);
+        mma16816(o[(2 * np + 1) & 3], a, b[2], b[3]);
+        ldsm4(b, ss_lo + col);
+        mma16816(o[(2 * np) & 3], a, b[0], b[1]);
+        mma16816(o[(2 * np + 1) & 3], a, b[2], b[3]);
+      }
       if (np <= warp) {  // keys of this warp's own tokens and those before them
         ldsm4(b, sk + at);
         mma16816(s[2 * np], a, b[0], b[1]);
@@ -335,7 +339,7 @@ chunk_output_kernel(const Args p, int dp) {
   }
   const float f0 = pw[i0 + 1], f1 = pw[i0 + 9];
 #pragma unroll
-  for (int t = 0; t < 8; ++t) { o[t][0] *= f0; o[t][1] *= f0; o[t][2] *= f1; o[t][3] *= f1; }
+  for (int t = 0; t < 4; ++t) { o[t][0] *= f0; o[t][1] *= f0; o[t][2] *= f1; o[t][3] *= f1; }
 #pragma unroll
   for (int kk = 0; kk < 4; ++kk) {  // 16 keys at a time
     if (kk > warp) break;
@@ -350,9 +354,9 @@ chunk_output_kernel(const Args p, int dp) {
       lo[q] = pack2(x - xh, y - yh);
     }
 #pragma unroll
-    for (int np = 0; np < 4; ++np) {
+    for (int np = 0; np < 2; ++np) {
       uint32_t b[4];
-      ldsm4_t(b, sv + (kk * 16 + (mi & 1) * 8 + li) * PITCH + np * 16 + (mi >> 1) * 8);
+      ldsm4_t(b, sv + (kk * 16 + (mi & 1) * 8 + li) * PITCH + half_no * 32 + np * 16 + (mi >> 1) * 8);
       mma16816(o[2 * np], hi, b[0], b[1]);
       mma16816(o[2 * np + 1], hi, b[2], b[3]);
       mma16816(o[2 * np], lo, b[0], b[1]);
@@ -366,8 +370,8 @@ chunk_output_kernel(const Args p, int dp) {
     if (i >= n) continue;
     float* dst = p.out + (row0 + i) * p.H * p.dv + (size_t)h * p.dv;
 #pragma unroll
-    for (int t = 0; t < 8; ++t) {
-      const int c = c0 + t * 8 + (lane & 3) * 2;
+    for (int t = 0; t < 4; ++t) {
+      const int c = c0 + half_no * 32 + t * 8 + (lane & 3) * 2;
       if (pairs && c + 1 < p.dv) *reinterpret_cast<float2*>(dst + c) = make_float2(o[t][2 * half], o[t][2 * half + 1]);
       else {
         if (c < p.dv) dst[c] = o[t][2 * half];
@@ -417,7 +421,7 @@ CUCA_API int cuca_lightning_chunked(const void* proj, int ld, int col0, const fl
     CUCA_REQUIRE(e == cudaSuccess, "lightning_chunked: %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
     allowed = smem;
   }
-  cuca_launch(chunk_output_kernel, dim3(n_chunks, H, c_tiles), dim3(128), smem, stream, true, p, dp);
+  cuca_launch(chunk_output_kernel, dim3(n_chunks, H, c_tiles), dim3(256), smem, stream, true, p, dp);
   CUCA_CHECK_LAUNCH("lightning_chunk_output");
   return 0;
 }
