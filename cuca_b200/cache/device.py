@@ -20,26 +20,27 @@ _STATE_DTYPES = {"float32": torch.float32, "bfloat16": torch.bfloat16, "int32": 
 
 def plan_groups(cache_needs: dict, kv_tokens: int, block_size: int, max_sequences: int,
                 max_step_tokens: int, window_pools: str = "sized") -> list:
-    """Group caches by (key heads, head size, window) and size each group's pool.
+    """Group caches by (key heads, head size, window, kept first positions) and size each group's pool.
 
     A group that keeps all keys gets ceil(kv_tokens / block) pages. A windowed
     group needs at most `max_sequences * (ceil((w - 1 + max_step_tokens) / block) + 2)`
-    pages (src/provider/local/model/paged.rs:175-220); `window_pools="full"` sizes
-    it like a full group instead.
+    pages (src/provider/local/model/paged.rs:175-220), and those of the first positions it keeps;
+    `window_pools="full"` sizes it like a full group instead.
     """
     by_key: dict = {}
     for cid in sorted(cache_needs):
         kv = cache_needs[cid].kv
         if kv is None:
             continue
-        by_key.setdefault((kv.n_kv_heads, kv.head_dim, kv.window, kv.v_head_dim), []).append(cid)
+        keep = kv.keep_first if kv.window is not None else 0
+        by_key.setdefault((kv.n_kv_heads, kv.head_dim, kv.window, kv.v_head_dim, keep), []).append(cid)
     full = -(-kv_tokens // block_size)
     groups = []
-    for (nkv, d, window, vd), ids in by_key.items():
+    for (nkv, d, window, vd, keep), ids in by_key.items():
         n = full
         if window is not None and window_pools == "sized":
-            n = min(full, max_sequences * (-(-(window - 1 + max_step_tokens) // block_size) + 2))
-        groups.append(GroupLayout(nkv, d, window, tuple(ids), max(1, n), vd))
+            n = min(full, max_sequences * (-(-(window - 1 + max_step_tokens) // block_size) + 2 + -(-keep // block_size)))
+        groups.append(GroupLayout(nkv, d, window, tuple(ids), max(1, n), vd, keep))
     return groups
 
 

@@ -6,7 +6,7 @@ window) share a group, each group has a pool of its own, and each request has
 one block table per group (src/provider/local/model/paged.rs:6-16,52-103,
 344-489 of the reference). Pages go back to the pool when a request ends and,
 in a windowed group, as soon as the window has passed them
-(model/paged.rs:736-761). No tensors live here; `cache/device.py` owns the
+(model/paged.rs:736-761), except those of the first positions a group keeps. No tensors live here; `cache/device.py` owns the
 memory the page ids index.
 
 The books themselves are kept by the C++ host core (`csrc/host/kv_pools.cpp`);
@@ -45,6 +45,7 @@ class GroupLayout:
     cache_ids: tuple  # caches (run-order cache numbers) that live in this group
     n_blocks: int
     v_head_dim: Optional[int] = None  # None: values as wide as keys; 0: the group has no value slab
+    keep_first: int = 0  # positions at a request's start that stay visible beside the window
 
 
 def _raise(code: int) -> None:
@@ -219,7 +220,8 @@ class KvPools:
         self._lib = host.load()
         self._h = self._lib.cuca_host_pools_new(
             self.n_groups, host.ints(g.n_blocks for g in self.groups),
-            host.ints(-1 if g.window is None else int(g.window) for g in self.groups), block_size)
+            host.ints(-1 if g.window is None else int(g.window) for g in self.groups),
+            host.ints(0 if g.window is None else int(g.keep_first) for g in self.groups), block_size)
         if not self._h:
             raise ValueError("the page pools could not be made")
         self.pools = [_GroupPool(self, gi) for gi in range(self.n_groups)]

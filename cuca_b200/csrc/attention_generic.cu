@@ -4,6 +4,7 @@
 // head sizes its tensor-core kernels refuse. A row's arithmetic depends only
 // on its own position and keys: tiles start at multiples of 32 key positions,
 // so cutting a prompt or batching it differently gives the same bits.
+#include "attention_options.cuh"
 #include "common.cuh"
 #include <math.h>
 
@@ -16,8 +17,9 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ 
                          const T* __restrict__ kpool, const T* __restrict__ vpool, int n_blocks, int bs,
                          const int* __restrict__ positions, const int* __restrict__ seq_of_row,
                          const int* __restrict__ tables, int table_stride, int nh, int nkv, int d, int dv,
-                         float scale, int window, float softcap, int sink, const float* __restrict__ sink_val,
-                         int* err) {
+                         const CucaAttnOptions opt, int* err) {
+  const float scale = opt.scale, softcap = opt.softcap;
+  const int window = opt.window;
   extern __shared__ float qs[];  // [4][d]
   pdl_trigger();
   pdl_wait();
@@ -35,15 +37,19 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ 
 
   int lo = 0;
   if (window > 0 && P - (window - 1) > 0) lo = P - (window - 1);
+  const int first = (lo / 32) * 32;             // the window's first tile
+  const int keep = window > 0 ? opt.keep : 0;
+  const int kept_end = min((keep + 31) / 32 * 32, first);  // the tiles of the kept first keys that lie before it
+  const float slope = opt.slopes ? opt.slopes[head] : 0.f;
   float m = -INFINITY, l = 0.f;
   float acc[VC];
 #pragma unroll
   for (int c = 0; c < VC; ++c) acc[c] = 0.f;
   const int* table = tables + (size_t)seq * table_stride;
 
-  for (int t0 = (lo / 32) * 32; t0 <= P; t0 += 32) {
+  for (int t0 = kept_end > 0 ? 0 : first; t0 <= P; t0 = t0 + 32 == kept_end ? first : t0 + 32) {
     int kp = t0 + lane;
-    bool valid = kp >= lo && kp <= P;
+    bool valid = (kp >= lo || kp < keep) && kp <= P;
     long long base = -1;  // this key's row number in the pools (key rows of d values, value rows of dv)
     if (valid) {
       int blk = table[kp / bs];
@@ -61,6 +67,7 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ 
       for (int i = 0; i < d; ++i) dot = fmaf(qv[i], to_f32(kr[i]), dot);
       s = dot * scale;
       if (softcap > 0.f) s = softcap * tanhf(s / softcap);  // a smooth cap on the score
+      if (opt.slopes) s -= slope * (float)(P - kp);
     }
     float m_new = fmaxf(m, warp_max(s));
     if (m_new == -INFINITY) continue;  // a tile with no readable key
@@ -82,8 +89,8 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ 
     }
     m = m_new;
   }
-  if (sink) {  // one more term in the denominator: a key of score 0 (or of the head's stored score) that has no value
-    const float s0 = sink_val ? sink_val[head] : 0.f;
+  if (opt.sink) {  // one more term in the denominator: a key of score 0 (or of the head's stored score) that has no value
+    const float s0 = opt.sink_val ? opt.sink_val[head] : 0.f;
     const float m_new = fmaxf(m, s0);
     const float corr = expf(m - m_new);
     l = l * corr + expf(s0 - m_new);
@@ -92,10 +99,14 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ 
   }
   float inv = l > 0.f ? 1.f / l : 0.f;
   T* o = out + (size_t)row * out_stride + (size_t)head * dv;
+  const T* gate = opt.gate ? (const T*)opt.gate + (size_t)row * opt.gate_stride + (size_t)head * dv : nullptr;
 #pragma unroll
   for (int c = 0; c < VC; ++c) {
     int dim = c * 32 + lane;
-    if (dim < dv) o[dim] = from_f32<T>(acc[c] * inv);
+    if (dim >= dv) continue;
+    float r = acc[c] * inv;
+    if (gate) r /= 1.f + expf(-to_f32(gate[dim]));
+    o[dim] = from_f32<T>(r);
   }
 }
 
@@ -108,17 +119,14 @@ CUCA_API int cuca_attention_max_head_dim() { return 256; }
 
 // q: rows of `q_stride` elements whose first nh*d hold the (rotated) query
 // heads; out: [n_rows, out_stride] with nh heads of dv values; key pool [n_blocks][nkv][bs][d], value pool
-// [n_blocks][nkv][bs][dv]. Row r is at position positions[r] of sequence seq_of_row[r] (< 0: padding, skipped) and
-// sees keys max(0, P - window + 1)..P of that sequence (window 0: all). softcap c > 0: a score s becomes
-// c tanh(s / c). sink: the softmax's denominator holds one more term, exp(0), or with sink_val (32-bit, one number per
-// query head) exp(sink_val[head]): a score that is neither scaled nor capped.
-CUCA_API int cuca_attention_generic_sv(const void* q, int q_stride, void* out, int out_stride, int dtype,
+// [n_blocks][nkv][bs][dv]. Row r is at position positions[r] of sequence seq_of_row[r] (< 0: padding, skipped).
+CUCA_API int cuca_attention_generic_o(const void* q, int q_stride, void* out, int out_stride, int dtype,
                                       const void* kpool, const void* vpool, int n_blocks, int bs,
                                       const int* positions, const int* seq_of_row, const int* tables,
-                                      int table_stride, int n_rows, int nh, int nkv, int d, int dv, float scale,
-                                      int window, float softcap, int sink, const float* sink_val, int* err,
-                                      cudaStream_t stream) {
+                                      int table_stride, int n_rows, int nh, int nkv, int d, int dv,
+                                      const CucaAttnOptions* opt, int* err, cudaStream_t stream) {
   if (n_rows == 0) return 0;
+  CUCA_REQUIRE(opt != nullptr && opt->window >= 0 && opt->keep >= 0, "attention: bad options");
   CUCA_REQUIRE(d > 0 && d <= cuca_attention_max_head_dim(), "attention: head size %d is outside 1..%d", d, cuca_attention_max_head_dim());
   CUCA_REQUIRE(dv > 0 && dv <= 2 * cuca_attention_max_head_dim(), "attention: value size %d is outside 1..%d", dv,
                2 * cuca_attention_max_head_dim());
@@ -129,7 +137,7 @@ CUCA_API int cuca_attention_generic_sv(const void* q, int q_stride, void* out, i
 #define AG(T, VC)                                                                                                  \
   cuca_launch(attention_generic_kernel<T, VC>, grid, dim3(128), smem, stream, true, (const T*)q, q_stride, (T*)out, \
               out_stride, (const T*)kpool, (const T*)vpool, n_blocks, bs, positions, seq_of_row, tables,            \
-              table_stride, nh, nkv, d, dv, scale, window, softcap, sink, sink_val, err)
+              table_stride, nh, nkv, d, dv, *opt, err)
   if (dtype == CUCA_F32) {
     if (dv <= 256) AG(float, 8); else AG(float, 16);
   } else if (dtype == CUCA_BF16) {
@@ -140,6 +148,18 @@ CUCA_API int cuca_attention_generic_sv(const void* q, int q_stride, void* out, i
 #undef AG
   CUCA_CHECK_LAUNCH("attention_generic");
   return 0;
+}
+
+// softcap, sink and sink_val: see CucaAttnOptions
+CUCA_API int cuca_attention_generic_sv(const void* q, int q_stride, void* out, int out_stride, int dtype,
+                                       const void* kpool, const void* vpool, int n_blocks, int bs,
+                                       const int* positions, const int* seq_of_row, const int* tables,
+                                       int table_stride, int n_rows, int nh, int nkv, int d, int dv, float scale,
+                                       int window, float softcap, int sink, const float* sink_val, int* err,
+                                       cudaStream_t stream) {
+  const CucaAttnOptions opt{scale, window, 0, softcap, sink, 0, sink_val, nullptr, nullptr};
+  return cuca_attention_generic_o(q, q_stride, out, out_stride, dtype, kpool, vpool, n_blocks, bs, positions, seq_of_row,
+                                  tables, table_stride, n_rows, nh, nkv, d, dv, &opt, err, stream);
 }
 
 CUCA_API int cuca_attention_generic_s(const void* q, int q_stride, void* out, int out_stride, int dtype,
@@ -275,6 +295,8 @@ CUCA_API int cuca_rope_store_general(void* qkv, int dtype, int ld, int k_col, in
 // q_norm [nh d], k alike over its nkv d values with k_norm [nkv d] (v_norm is not combined with it).
 // qt_every > 0: the query of a row at position p is multiplied by 1 + qt_coef ln(floor((p + 1) / qt_every) + 1), after
 // norm and rotation.
+// unit != 0: the norms per head without a weight (q_norm and k_norm null). q_mul [nh]: a factor on every query of a head,
+// after the norm. v_col may be k_col: the values are then the keys as projected.
 namespace {
 template <typename T, typename TP>
 __global__ void __launch_bounds__(256)
@@ -284,7 +306,8 @@ norm_rope_store_kernel(T* __restrict__ qkv, int ld, int k_col, int v_col, TP* __
                        const float* __restrict__ sin_t, int table_rows, int rot, int pairs,
                        const float* __restrict__ q_norm, const float* __restrict__ k_norm, int v_norm, float eps,
                        TP* __restrict__ kpool, TP* __restrict__ vpool, int n_blocks, int bs, int nh, int nkv, int d, int dv,
-                       int v_split, int dv_src, int whole, float qt_coef, int qt_every, int* err) {
+                       int v_split, int dv_src, int whole, float qt_coef, int qt_every, int unit,
+                       const float* __restrict__ q_mul_head, int* err) {
   __shared__ float red[2][8];
   pdl_trigger();
   pdl_wait();
@@ -332,9 +355,9 @@ norm_rope_store_kernel(T* __restrict__ qkv, int ld, int k_col, int v_col, TP* __
     const T* src = base + (kind == 0 ? 0 : (kind == 1 ? k_col : v_col)) + (size_t)hh * n;
     const float* w = kind == 0 ? q_norm : (kind == 1 ? k_norm : nullptr);
     if (whole && w) w += (size_t)hh * d;  // the weight covers the whole projection
-    const bool normed = kind == 2 ? v_norm != 0 : (w != nullptr && !whole);
+    const bool normed = kind == 2 ? v_norm != 0 : ((w != nullptr || unit) && !whole);
     float inv = (whole && kind != 2) ? inv_whole[kind] : 1.f;
-    const float mul = kind == 0 ? q_mul : 1.f;
+    const float mul = kind == 0 ? q_mul * (q_mul_head ? q_mul_head[hh] : 1.f) : 1.f;
     if (normed) {
       float ss = 0.f;
       for (int i = lane; i < n; i += 32) { const float v = to_f32(src[i]); ss = fmaf(v, v, ss); }
@@ -369,18 +392,83 @@ norm_rope_store_kernel(T* __restrict__ qkv, int ld, int k_col, int v_col, TP* __
     }
   }
 }
+
+// The same without rotation for bfloat16 rows with heads of a multiple of eight values and value heads as wide as keys:
+// `group` lanes (a power of two) take one head of one row, 16 bytes a lane. Values that are the keys as projected
+// (v_col == k_col) are written by the lanes that have them.
+__global__ void __launch_bounds__(256)
+norm_store_kernel(__nv_bfloat16* __restrict__ qkv, int ld, int k_col, int v_col, const int* __restrict__ positions,
+                  const int* __restrict__ seq_of_row, const int* __restrict__ tables, int table_stride,
+                  const float* __restrict__ q_norm, const float* __restrict__ k_norm, int v_norm, float eps,
+                  __nv_bfloat16* __restrict__ kpool, __nv_bfloat16* __restrict__ vpool, int n_blocks, int bs, int n_rows,
+                  int nh, int nkv, int d, int group, float qt_coef, int qt_every, int unit,
+                  const float* __restrict__ q_mul_head, int* err) {
+  pdl_trigger();
+  pdl_wait();
+  const int heads = nh + nkv * (v_col == k_col ? 1 : 2);
+  const long long item = ((long long)blockIdx.x * blockDim.x + threadIdx.x) / group;
+  const int row = (int)(item / heads), head = (int)(item % heads), c = (threadIdx.x % group) * 8;
+  const int seq = row < n_rows ? seq_of_row[row] : -1;
+  const bool active = seq >= 0 && c < d;  // (the shuffles below are the whole warp's)
+  const int kind = head < nh ? 0 : (head < nh + nkv ? 1 : 2);  // q, k, v
+  const int hh = kind == 0 ? head : (kind == 1 ? head - nh : head - nh - nkv);
+  __nv_bfloat16* src = qkv + (size_t)(row < n_rows ? row : 0) * ld + (kind == 0 ? 0 : (kind == 1 ? k_col : v_col)) + (size_t)hh * d + c;
+  const int pos = seq >= 0 ? positions[row] : 0;
+  uint4 raw = make_uint4(0, 0, 0, 0);
+  if (active) raw = *reinterpret_cast<const uint4*>(src);
+  const __nv_bfloat16* rv = reinterpret_cast<const __nv_bfloat16*>(&raw);
+  float v[8], ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) { v[i] = __bfloat162float(rv[i]); ss = fmaf(v[i], v[i], ss); }
+  for (int o = group / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  if (!active) return;
+  const float* w = kind == 0 ? q_norm : (kind == 1 ? k_norm : nullptr);
+  const bool normed = kind == 2 ? v_norm != 0 : (w != nullptr || unit);
+  float mul = normed ? 1.f / sqrtf(ss / (float)d + eps) : 1.f;
+  if (kind == 0) {
+    if (qt_every > 0 && pos >= 0) mul *= 1.f + qt_coef * logf((float)((pos + 1) / qt_every + 1));
+    if (q_mul_head) mul *= q_mul_head[hh];
+  }
+  uint4 res;
+  __nv_bfloat162* r2 = reinterpret_cast<__nv_bfloat162*>(&res);
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+    r2[i] = __floats2bfloat162_rn(v[2 * i] * mul * (w ? w[c + 2 * i] : 1.f), v[2 * i + 1] * mul * (w ? w[c + 2 * i + 1] : 1.f));
+  if (kind == 0) {
+    *reinterpret_cast<uint4*>(src) = res;
+    return;
+  }
+  const int blk = pos >= 0 ? tables[(size_t)seq * table_stride + pos / bs] : -1;
+  if (blk < 0 || blk >= n_blocks) {
+    if (err) atomicExch(err, CUCA_ERR_BLOCK_RANGE);
+    return;
+  }
+  const size_t at = (((size_t)blk * nkv + hh) * bs + pos % bs) * d + c;
+  if (kind == 1) *reinterpret_cast<uint4*>(kpool + at) = res;
+  if (kind == 2) *reinterpret_cast<uint4*>(vpool + at) = res;
+  if (kind == 1 && v_col == k_col) {
+    if (v_norm) {  // (the norm has no weight here, whatever the key's is)
+      const float inv = 1.f / sqrtf(ss / (float)d + eps);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) r2[i] = __floats2bfloat162_rn(v[2 * i] * inv, v[2 * i + 1] * inv);
+      raw = res;
+    }
+    *reinterpret_cast<uint4*>(vpool + at) = raw;
+  }
+}
 }  // namespace
 
 // dtype: of the rows; pool_dtype: of the pools and of q_out (null: q in place, in the rows' type).
-// whole, qt_coef, qt_every: see the kernel (0, 0, 0: norms per head, no query temperature).
-CUCA_API int cuca_norm_rope_store_w(void* qkv, int dtype, int ld, int k_col, int v_col, void* q_out, int pool_dtype,
+// whole, qt_coef, qt_every, unit, q_mul: see the kernel (0, 0, 0, 0, null: norms per head, no factor on the queries).
+CUCA_API int cuca_norm_rope_store_u(void* qkv, int dtype, int ld, int k_col, int v_col, void* q_out, int pool_dtype,
                                     const int* positions, const int* seq_of_row, const int* tables, int table_stride,
                                     const float* cos_t, const float* sin_t, int table_rows, int rot, int pairs,
                                     const float* q_norm, const float* k_norm, int v_norm, float eps, void* kpool,
                                     void* vpool, int n_blocks, int bs, int n_rows, int nh, int nkv, int d, int dv,
-                                    int v_split, int dv_src, int whole, float qt_coef, int qt_every, int* err,
-                                    cudaStream_t stream) {
+                                    int v_split, int dv_src, int whole, float qt_coef, int qt_every, int unit,
+                                    const float* q_mul, int* err, cudaStream_t stream) {
   if (n_rows == 0) return 0;
+  CUCA_REQUIRE(!unit || (!whole && !q_norm && !k_norm), "norm_rope_store: a norm without a weight is given none");
   CUCA_REQUIRE(!whole || (q_norm && (nkv == 0 || k_norm) && !v_norm),
                "norm_rope_store: a norm over the whole projection needs both weights and takes no value norm");
   if (dv_src <= 0) dv_src = dv;
@@ -388,11 +476,24 @@ CUCA_API int cuca_norm_rope_store_w(void* qkv, int dtype, int ld, int k_col, int
   CUCA_REQUIRE(rot >= 0 && rot <= d && rot % 2 == 0, "norm_rope_store: rotary size %d does not fit head size %d", rot, d);
   CUCA_REQUIRE(bs > 0 && nh > 0 && nkv >= 0 && d > 0 && dv > 0, "norm_rope_store: bad sizes");
   CUCA_REQUIRE(v_split >= 1 && dv % v_split == 0, "norm_rope_store: %d slabs do not divide value size %d", v_split, dv);
+  const bool aligned = (((uintptr_t)qkv | (uintptr_t)kpool | (uintptr_t)vpool) & 15) == 0;
+  if (rot == 0 && !whole && dtype == CUCA_BF16 && pool_dtype == CUCA_BF16 && !q_out && nkv > 0 && d % 8 == 0 && d <= 256 &&
+      dv == d && dv_src == d && v_split == 1 && ld % 8 == 0 && k_col % 8 == 0 && v_col % 8 == 0 && aligned) {
+    int group = 1;
+    while (group * 8 < d) group *= 2;
+    const long long lanes = (long long)n_rows * (nh + nkv * (v_col == k_col ? 1 : 2)) * group;
+    cuca_launch(norm_store_kernel, dim3((unsigned)((lanes + 255) / 256)), dim3(256), 0, stream, true, (__nv_bfloat16*)qkv, ld,
+                k_col, v_col, positions, seq_of_row, tables, table_stride, q_norm, k_norm, v_norm, eps,
+                (__nv_bfloat16*)kpool, (__nv_bfloat16*)vpool, n_blocks, bs, n_rows, nh, nkv, d, group, qt_coef, qt_every,
+                unit, q_mul, err);
+    CUCA_CHECK_LAUNCH("norm_store");
+    return 0;
+  }
 #define NRS(T, TP)                                                                                                    \
   cuca_launch(norm_rope_store_kernel<T, TP>, dim3(n_rows), dim3(256), 0, stream, true, (T*)qkv, ld, k_col, v_col,      \
               (TP*)q_out, positions, seq_of_row, tables, table_stride, cos_t, sin_t, table_rows, rot, pairs, q_norm,   \
               k_norm, v_norm, eps, (TP*)kpool, (TP*)vpool, n_blocks, bs, nh, nkv, d, dv, v_split, dv_src, whole,       \
-              qt_coef, qt_every, err)
+              qt_coef, qt_every, unit, q_mul, err)
   if (dtype == CUCA_F32 && pool_dtype == CUCA_F32) NRS(float, float);
   else if (dtype == CUCA_BF16 && pool_dtype == CUCA_BF16) NRS(__nv_bfloat16, __nv_bfloat16);
   else if (dtype == CUCA_F32 && pool_dtype == CUCA_BF16) {
@@ -402,6 +503,19 @@ CUCA_API int cuca_norm_rope_store_w(void* qkv, int dtype, int ld, int k_col, int
 #undef NRS
   CUCA_CHECK_LAUNCH("norm_rope_store");
   return 0;
+}
+
+CUCA_API int cuca_norm_rope_store_w(void* qkv, int dtype, int ld, int k_col, int v_col, void* q_out, int pool_dtype,
+                                    const int* positions, const int* seq_of_row, const int* tables, int table_stride,
+                                    const float* cos_t, const float* sin_t, int table_rows, int rot, int pairs,
+                                    const float* q_norm, const float* k_norm, int v_norm, float eps, void* kpool,
+                                    void* vpool, int n_blocks, int bs, int n_rows, int nh, int nkv, int d, int dv,
+                                    int v_split, int dv_src, int whole, float qt_coef, int qt_every, int* err,
+                                    cudaStream_t stream) {
+  return cuca_norm_rope_store_u(qkv, dtype, ld, k_col, v_col, q_out, pool_dtype, positions, seq_of_row, tables,
+                                table_stride, cos_t, sin_t, table_rows, rot, pairs, q_norm, k_norm, v_norm, eps, kpool,
+                                vpool, n_blocks, bs, n_rows, nh, nkv, d, dv, v_split, dv_src, whole, qt_coef, qt_every, 0,
+                                nullptr, err, stream);
 }
 
 CUCA_API int cuca_norm_rope_store(void* qkv, int dtype, int ld, int k_col, int v_col, void* q_out, int pool_dtype,

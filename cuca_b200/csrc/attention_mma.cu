@@ -17,6 +17,7 @@
 //    128-byte swizzle, one thread, mbarrier hand-over) through a ring of its own, so the loop has no block-wide
 //    barrier and no per-thread address arithmetic (batch 64: 69 -> 55 us per layer at Llama-3.1-8B sizes).
 // Positions outside a row's range (causal, window) are masked after scaling.
+#include "attention_options.cuh"
 #include "tcgen05.cuh"
 #include <math.h>
 #include <stdlib.h>
@@ -50,6 +51,10 @@ struct AttnParams {
   int sink;              // 1: the softmax's denominator holds one more exp(0) ...
   const float* sink_val; // ... or, when given, exp(sink_val[query head]) (32-bit; neither scaled nor capped)
   int window;
+  int keep;              // beside the window, the first `keep` keys of a request are seen (0 without a window)
+  const float* slopes;   // distance bias per query head (null: none): slopes[head] (P - key) is taken off a score
+  const __nv_bfloat16* gate;  // with it the result is multiplied by sigmoid(gate[row][head D + dim])
+  int gate_stride;
   int chunk;             // decode: key positions per split (multiple of 64); 0: each row divides its own length
   int slots;             // decode, chunk 0: CTAs the GPU holds at once (for the choice of chunks per row)
   float* part;           // decode: [rows][nh][splits][D + 2] partial (acc, m, l)
@@ -147,6 +152,7 @@ __device__ __forceinline__ float score_log2(float raw, const AttnParams& p) {
   if (p.cap_log2e > 0.f) return p.cap_log2e - __fdividef(2.f * p.cap_log2e, exp2f(raw * p.cap_arg) + 1.f);
   return raw * p.scale_log2e;
 }
+__device__ __forceinline__ float sigmoid_of(__nv_bfloat16 g) { return 1.f / (1.f + __expf(-__bfloat162float(g))); }
 // What a sink (score 0 or the head's stored score, no value) adds to a row sum kept relative to the maximum m (log2 units)
 __device__ __forceinline__ float sink_term(float m, const AttnParams& p, int head) {
   if (m == -INFINITY) return 1.f;  // a row without keys: its sums are 0 and so is its output
@@ -174,7 +180,12 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
   if (!EARLY) pdl_wait();
 
   // ---------------------------------------------------------------- what this CTA and warp own
-  int seq, kvh, range_lo, range_hi;   // keys [range_lo, range_hi) of request `seq`
+  // Keys of request `seq` that some row of the CTA may see: [range_lo, range_hi) and, below range_lo, the first p.keep.
+  // They are walked in tiles of 64 positions, counted without the gap between: the n_kept tiles that hold the first keys,
+  // then the window's from tile number window_tile on. The CTA takes n_tiles of them from first_tile on.
+  int seq, kvh, range_lo, range_hi;
+  int window_tile, n_kept, first_tile = 0, n_tiles;
+  bool has_own = false;  // decode: the row's own position is among the CTA's keys
   int row_token[2], row_head[2], row_pos[2];  // per owned MMA row (g, g + 8): token row, query head, position
   bool row_ok[2];
   int dec_row = 0, P = 0, warp_pmax = 0;
@@ -185,13 +196,16 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
     if (seq < 0) return;
     P = p.positions[dec_row];
     kvh = blockIdx.y;
-    int lo = (p.window > 0 && P - (p.window - 1) > 0) ? P - (p.window - 1) : 0;
+    range_lo = (p.window > 0 && P - (p.window - 1) > 0) ? P - (p.window - 1) : 0;
+    range_hi = P + 1;
+    window_tile = range_lo / TILE;
+    n_kept = min((p.keep + TILE - 1) / TILE, window_tile);
+    const int tiles = n_kept + P / TILE - window_tile + 1;
     // chunk 0: every row picks how many of the gridDim.x chunks it uses from its own length, so that the tiles
     // of 64 keys on the critical path (rounds of CTAs the GPU needs, times tiles per chunk) are fewest, and
     // spreads its keys evenly over them; the other chunks of the row are empty
     int chunk = p.chunk;
     if (chunk == 0) {
-      const int tiles = (P + TILE) / TILE;
       const int pairs = (int)(gridDim.y * gridDim.z);
       const int nmax = min((int)gridDim.x, tiles);
       int best = 1, best_cost = 0x7fffffff;
@@ -213,8 +227,9 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
       }
       return;
     }
-    range_lo = max(lo, (int)blockIdx.x * chunk);
-    range_hi = min(P + 1, ((int)blockIdx.x + 1) * chunk);
+    first_tile = (int)blockIdx.x * (chunk / TILE);
+    n_tiles = max(0, min(tiles - first_tile, chunk / TILE));
+    has_own = n_tiles > 0 && first_tile + n_tiles == tiles;
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
       int item = g + 8 * h;
@@ -233,6 +248,9 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
     kvh = head / G;
     range_lo = (p.window > 0 && pos0 - (p.window - 1) > 0) ? pos0 - (p.window - 1) : 0;
     range_hi = pos0 + n;
+    window_tile = range_lo / TILE;
+    n_kept = min((p.keep + TILE - 1) / TILE, window_tile);
+    n_tiles = n_kept + (range_hi - 1) / TILE - window_tile + 1;
     warp_pmax = pos0 + warp * 16 + 15;
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
@@ -271,18 +289,23 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
   st.l[0] = st.l[1] = 0.f;
 
   // ---------------------------------------------------------------- tile loop
-  const int first_tile = range_lo < range_hi ? (range_lo / TILE) : 0;
-  const int n_tiles = range_lo < range_hi ? ((range_hi - 1) / TILE - first_tile + 1) : 0;
+  auto tile_key0 = [&](int ti) {  // first key of the CTA's tile ti
+    const int v = first_tile + ti;
+    return (v < n_kept ? v : window_tile + v - n_kept) * TILE;
+  };
+  float slope2[2];  // the distance bias of the owned rows, in log2 units
+#pragma unroll
+  for (int h = 0; h < 2; ++h) slope2[h] = (p.slopes && row_ok[h]) ? p.slopes[row_head[h]] * CUCA_LOG2E : 0.f;
 
   // Row offsets of a tile's 64 keys in the pools (-1: masked or without a page), one tile ahead of the copies:
   // the page-table lookups of tile i + 2 are in flight while tile i is computed, so no copy waits on one.
   __shared__ long long s_rowoff[STAGES][TILE];
   const int bs_shift = __ffs(p.bs) - 1, bs_mask = p.bs - 1;
   // fused form: the CTA whose keys include the row's own position makes that key and value itself
-  const bool owner = FUSED && p.has_kv && P >= range_lo && P < range_hi;
+  const bool owner = FUSED && p.has_kv && has_own;
   auto row_offset = [&](int tile_index) -> long long {
-    int kp = (first_tile + tile_index) * TILE + (int)threadIdx.x;
-    if (kp < range_lo || kp >= range_hi) return -1;
+    int kp = tile_key0(tile_index) + (int)threadIdx.x;
+    if ((kp < range_lo && kp >= p.keep) || kp >= range_hi) return -1;
     if (owner && kp == P) return -1;  // comes from registers, not from the page
     int blk = table[kp >> bs_shift];
     if (blk < 0 || blk >= p.n_blocks) {
@@ -311,12 +334,14 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
   __shared__ int w_abort;
   int ti_lo = 0, n_mine = 0, next_page = -1;
   uint8_t* ring = ring_base + (size_t)warp * S::WSTAGES * S::WSTAGE_BYTES;
-  auto group_kp0 = [&](int j) { return (first_tile + ti_lo + j) * TILE + warp * 16; };
+  auto group_kp0 = [&](int j) { return tile_key0(ti_lo + j) + warp * 16; };
+  auto group_seen = [&](int kp0) { return kp0 < range_hi && (kp0 + 16 > range_lo || kp0 < p.keep); };
   auto page_of = [&](int j) { return table[group_kp0(j) >> bs_shift]; };
   auto issue_group = [&](int j, int page) {  // the whole warp: one copy per lane (keys and values, 64-wide halves)
     const int kp0 = group_kp0(j);
     if (page < 0 || page >= p.n_blocks) {
-      if (lane == 0 && p.err) atomicExch(p.err, CUCA_ERR_BLOCK_RANGE);
+      // (a run of groups may hold one that lies behind the window, whose page is gone)
+      if (lane == 0 && p.err && group_seen(kp0)) atomicExch(p.err, CUCA_ERR_BLOCK_RANGE);
       page = 0;  // any readable page: these keys are masked or the step is lost anyway
     }
     const int row = ((page * p.nkv + kvh) << bs_shift) + (kp0 & bs_mask);
@@ -384,11 +409,10 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
       for (int st = 0; st < S::WSTAGES; ++st) mbar_init(&w_full[warp][st], 1);
       asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
-    // groups with a key in range: a run of consecutive tiles
+    // groups with a key in range: a run of consecutive tiles, from the first such to the last
     int lo = n_tiles, hi = 0;
     for (int ti = 0; ti < n_tiles; ++ti) {
-      const int kp0 = (first_tile + ti) * TILE + warp * 16;
-      if (kp0 < range_hi && kp0 + 16 > range_lo) { lo = min(lo, ti); hi = ti + 1; }
+      if (group_seen(tile_key0(ti) + warp * 16)) { lo = min(lo, ti); hi = ti + 1; }
     }
     ti_lo = lo;
     n_mine = hi > lo ? hi - lo : 0;
@@ -566,8 +590,8 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
     }
     // ---- scale, mask, online softmax (per row: g and g + 8). Tiles that every row of the warp sees whole
     // (the bulk of a long prompt) skip the per-key tests.
-    bool whole = !DECODE && kp0 >= range_lo && kp0 + 16 * SUBS <= range_hi && kp0 + 16 * SUBS - 1 <= warp_pmax - 15 &&
-                 (p.window <= 0 || kp0 >= warp_pmax - (p.window - 1));
+    bool whole = !DECODE && kp0 + 16 * SUBS <= range_hi && kp0 + 16 * SUBS - 1 <= warp_pmax - 15 &&
+                 (p.window <= 0 || kp0 >= warp_pmax - (p.window - 1) || kp0 + 16 * SUBS <= p.keep);
     uint32_t pa[SUBS][4];
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
@@ -578,6 +602,7 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
 #pragma unroll
           for (int e = 0; e < 2; ++e) {
             float v = score_log2(s[nt][2 * h + e], p);
+            if (p.slopes) v = fmaf(-slope2[h], (float)(row_pos[h] - (kp0 + nt * 8 + 2 * t + e)), v);
             s[nt][2 * h + e] = v;
             mx = fmaxf(mx, v);
           }
@@ -588,8 +613,10 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
 #pragma unroll
           for (int e = 0; e < 2; ++e) {
             int kp = kp0 + nt * 8 + 2 * t + e;
-            bool ok = row_ok[h] && kp <= row_pos[h] && kp >= lo_row && kp >= range_lo && kp < range_hi;
-            float v = ok ? score_log2(s[nt][2 * h + e], p) : -INFINITY;
+            bool ok = row_ok[h] && kp <= row_pos[h] && (kp >= lo_row || kp < p.keep);
+            float v = score_log2(s[nt][2 * h + e], p);
+            if (p.slopes) v = fmaf(-slope2[h], (float)(row_pos[h] - kp), v);
+            v = ok ? v : -INFINITY;
             s[nt][2 * h + e] = v;
             mx = fmaxf(mx, v);
           }
@@ -685,7 +712,7 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
       long long next_off = -1;
       const bool look_ahead = threadIdx.x < TILE && ti + STAGES < n_tiles;
       if (look_ahead) next_off = row_offset(ti + STAGES);
-      const int start = (first_tile + ti) * TILE;
+      const int start = tile_key0(ti);
       const __nv_bfloat16* ks = smem + (size_t)stage * 2 * S::TILE_ELEMS;
       const __nv_bfloat16* vs = ks + S::TILE_ELEMS;
       if (owner && P >= start && P < start + TILE) {
@@ -700,7 +727,7 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
       }
       const int sub0 = DECODE ? warp : 0;
       const int kp0 = start + sub0 * 16;              // first key of this update
-      bool active = kp0 < range_hi && kp0 + 16 * SUBS > range_lo;
+      bool active = kp0 < range_hi && (kp0 + 16 * SUBS > range_lo || kp0 < p.keep);
       if (!DECODE && kp0 > warp_pmax) active = false;  // every row of this warp lies before these keys (causal)
       if (active)
         update([&](int key, int dim) { return smem_u32(ks + key * S::RS + dim); },
@@ -726,7 +753,13 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
       __nv_bfloat16* o = p.out + (size_t)row_token[h] * p.out_stride + (size_t)row_head[h] * D;
 #pragma unroll
       for (int j = 0; j < D / 8; ++j) {
-        uint32_t v = pack_bf16(st.acc[j][2 * h] * inv, st.acc[j][2 * h + 1] * inv);
+        float o0 = st.acc[j][2 * h] * inv, o1 = st.acc[j][2 * h + 1] * inv;
+        if (p.gate) {
+          const __nv_bfloat16* gp = p.gate + (size_t)row_token[h] * p.gate_stride + (size_t)row_head[h] * D + j * 8 + 2 * t;
+          o0 *= sigmoid_of(gp[0]);
+          o1 *= sigmoid_of(gp[1]);
+        }
+        uint32_t v = pack_bf16(o0, o1);
         *reinterpret_cast<uint32_t*>(o + j * 8 + 2 * t) = v;
       }
     }
@@ -737,6 +770,9 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
   __syncthreads();
   float* fs = reinterpret_cast<float*>(smem_raw);   // [4 warps][16 rows][D + 2]
   constexpr int FR = D + 2;
+  auto gate_at = [&](int item, int dim) -> float {  // the factor on an output value of the group's head `item`
+    return p.gate ? sigmoid_of(p.gate[(size_t)dec_row * p.gate_stride + (size_t)(kvh * G + item) * D + dim]) : 1.f;
+  };
 #pragma unroll
   for (int h = 0; h < 2; ++h) {
     int rowi = g + 8 * h;
@@ -773,7 +809,7 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
     if (n_used == 1) {
       if (p.sink) L += sink_term(M, p, kvh * G + item);
       p.out[(size_t)dec_row * p.out_stride + (size_t)(kvh * G + item) * D + dim] =
-          __float2bfloat16_rn(L > 0.f ? O / L : 0.f);
+          __float2bfloat16_rn((L > 0.f ? O / L : 0.f) * gate_at(item, dim));
     } else {
       float* dst = by_cluster ? cpart + (size_t)item * FR : part_row + ((size_t)item * n_splits + blockIdx.x) * FR;
       dst[dim] = O;
@@ -825,7 +861,7 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
         float O = 0.f;
 #pragma unroll
         for (int sidx = 0; sidx < 8; ++sidx) O += v[sidx] * (sidx < n_used ? s_f[item][sidx] : 0.f);
-        p.out[(size_t)dec_row * p.out_stride + (size_t)(kvh * G + item) * D + dim] = __float2bfloat16_rn(O * s_inv[item]);
+        p.out[(size_t)dec_row * p.out_stride + (size_t)(kvh * G + item) * D + dim] = __float2bfloat16_rn(O * s_inv[item] * gate_at(item, dim));
       }
     }
     cluster_sync_all();
@@ -891,7 +927,7 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
       float O = 0.f;
 #pragma unroll
       for (int sidx = 0; sidx < PS; ++sidx) O += v0[e][sidx] * s_f[item][sidx];  // chunks past n_used: 0 x 0
-      p.out[(size_t)dec_row * p.out_stride + (size_t)(kvh * G + item) * D + dim] = __float2bfloat16_rn(O * s_inv[item]);
+      p.out[(size_t)dec_row * p.out_stride + (size_t)(kvh * G + item) * D + dim] = __float2bfloat16_rn(O * s_inv[item] * gate_at(item, dim));
     }
   } else {
     for (int idx = threadIdx.x; idx < G * D; idx += NTHREADS) {
@@ -903,7 +939,7 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
       float O = 0.f;
 #pragma unroll
       for (int sidx = 0; sidx < MAXS; ++sidx) O += v[sidx] * s_f[item][sidx];
-      p.out[(size_t)dec_row * p.out_stride + (size_t)(kvh * G + item) * D + dim] = __float2bfloat16_rn(O * s_inv[item]);
+      p.out[(size_t)dec_row * p.out_stride + (size_t)(kvh * G + item) * D + dim] = __float2bfloat16_rn(O * s_inv[item] * gate_at(item, dim));
     }
   }
   if (threadIdx.x == 0) p.counters[blockIdx.z * p.nkv + kvh] = 0;
@@ -989,19 +1025,25 @@ struct FusedInput {
   int table_rows, rot, has_kv;
 };
 
-void set_score_options(AttnParams& p, float scale, float softcap, int sink, const float* sink_val = nullptr) {
+void set_score_options(AttnParams& p, const CucaAttnOptions& o) {
+  const float scale = o.scale, softcap = o.softcap;
+  p.scale_log2e = scale * CUCA_LOG2E;
+  p.window = o.window;
+  p.keep = o.window > 0 ? o.keep : 0;
+  p.slopes = o.slopes;
+  p.gate = (const __nv_bfloat16*)o.gate;
+  p.gate_stride = o.gate_stride;
   p.cap_log2e = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
   p.cap_arg = softcap > 0.f ? 2.f * scale * 1.4426950408889634f / softcap : 0.f;
-  p.sink = sink ? 1 : 0;
-  p.sink_val = sink ? sink_val : nullptr;
+  p.sink = o.sink ? 1 : 0;
+  p.sink_val = o.sink ? o.sink_val : nullptr;
 }
 
 int attention_decode_impl(const void* q, int q_stride, const FusedInput* fused, void* out, int out_stride,
                           const void* kpool, const void* vpool, int n_blocks, int bs, const int* positions,
                           const int* seq_of_row, const int* tables, int table_stride, const int* rows, int n_rows,
-                          int nh, int nkv, int d, float scale, int window, int chunk, int n_splits, float* part,
-                          int* counters, int* err, cudaStream_t stream, float softcap = 0.f, int sink = 0,
-                          const float* sink_val = nullptr) {
+                          int nh, int nkv, int d, const CucaAttnOptions& opt, int chunk, int n_splits, float* part,
+                          int* counters, int* err, cudaStream_t stream) {
   int dev = 0, sms = 148;
   cudaGetDevice(&dev);
   cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
@@ -1024,9 +1066,10 @@ int attention_decode_impl(const void* q, int q_stride, const FusedInput* fused, 
   p.kpool = (const __nv_bfloat16*)kpool; p.vpool = (const __nv_bfloat16*)vpool; p.n_blocks = n_blocks; p.bs = bs;
   p.tables = tables; p.table_stride = table_stride; p.positions = positions; p.seq_of_row = seq_of_row;
   p.rows = rows; p.tile_row0 = nullptr; p.tile_nrows = nullptr; p.nh = nh; p.nkv = nkv;
-  p.scale_log2e = scale * 1.4426950408889634f; p.window = window; p.chunk = chunk; p.part = part;
+  p.chunk = chunk; p.part = part;
   p.counters = counters; p.err = err; p.slots = sms * per_sm;
-  set_score_options(p, scale, softcap, sink, sink_val);
+  CUCA_REQUIRE(opt.window >= 0 && opt.keep >= 0, "attention_decode: bad options");
+  set_score_options(p, opt);
   p.cluster = by_cluster ? 1 : 0;
   p.partial = nullptr; p.n_slices = 0; p.slice_stride = 0; p.bias = nullptr; p.cos_t = p.sin_t = nullptr;
   p.table_rows = 0; p.rot = 0; p.has_kv = 0;
@@ -1056,9 +1099,22 @@ CUCA_API int cuca_attention_decode(const void* q, int q_stride, void* out, int o
                                    const int* seq_of_row, const int* tables, int table_stride, const int* rows,
                                    int n_rows, int nh, int nkv, int d, float scale, int window, int chunk,
                                    int n_splits, float* part, int* counters, int* err, cudaStream_t stream) {
+  const CucaAttnOptions opt{scale, window, 0, 0.f, 0, 0, nullptr, nullptr, nullptr};
   return attention_decode_impl(q, q_stride, nullptr, out, out_stride, kpool, vpool, n_blocks, bs, positions,
-                               seq_of_row, tables, table_stride, rows, n_rows, nh, nkv, d, scale, window, chunk,
-                               n_splits, part, counters, err, stream);
+                               seq_of_row, tables, table_stride, rows, n_rows, nh, nkv, d, opt, chunk, n_splits, part,
+                               counters, err, stream);
+}
+
+// The decode form with every option (window, kept first keys, cap, distance bias, sink, output gate).
+CUCA_API int cuca_attention_decode_o(const void* q, int q_stride, void* out, int out_stride, const void* kpool,
+                                     const void* vpool, int n_blocks, int bs, const int* positions, const int* seq_of_row,
+                                     const int* tables, int table_stride, const int* rows, int n_rows, int nh, int nkv,
+                                     int d, const CucaAttnOptions* opt, int chunk, int n_splits, float* part,
+                                     int* counters, int* err, cudaStream_t stream) {
+  CUCA_REQUIRE(opt != nullptr, "attention_decode: no options");
+  return attention_decode_impl(q, q_stride, nullptr, out, out_stride, kpool, vpool, n_blocks, bs, positions, seq_of_row,
+                               tables, table_stride, rows, n_rows, nh, nkv, d, *opt, chunk, n_splits, part, counters, err,
+                               stream);
 }
 
 // The decode form with a smooth cap on the scaled scores (softcap c > 0: s becomes c tanh(s / c)) and, with `sink`, one
@@ -1070,9 +1126,10 @@ CUCA_API int cuca_attention_decode_sv(const void* q, int q_stride, void* out, in
                                       int n_rows, int nh, int nkv, int d, float scale, int window, float softcap,
                                       int sink, const float* sink_val, int chunk, int n_splits, float* part,
                                       int* counters, int* err, cudaStream_t stream) {
+  const CucaAttnOptions opt{scale, window, 0, softcap, sink, 0, sink_val, nullptr, nullptr};
   return attention_decode_impl(q, q_stride, nullptr, out, out_stride, kpool, vpool, n_blocks, bs, positions,
-                               seq_of_row, tables, table_stride, rows, n_rows, nh, nkv, d, scale, window, chunk,
-                               n_splits, part, counters, err, stream, softcap, sink, sink_val);
+                               seq_of_row, tables, table_stride, rows, n_rows, nh, nkv, d, opt, chunk, n_splits, part,
+                               counters, err, stream);
 }
 
 CUCA_API int cuca_attention_decode_s(const void* q, int q_stride, void* out, int out_stride, const void* kpool,
@@ -1099,20 +1156,20 @@ CUCA_API int cuca_attention_decode_fused(const float* partial, int n_slices, siz
                                          float scale, int window, int chunk, int n_splits, float* part, int* counters,
                                          int* err, cudaStream_t stream) {
   FusedInput f{partial, n_slices, slice_stride, bias, cos_t, sin_t, table_rows, rot, has_kv};
+  const CucaAttnOptions opt{scale, window, 0, 0.f, 0, 0, nullptr, nullptr, nullptr};
   return attention_decode_impl(nullptr, 2, &f, out, out_stride, kpool, vpool, n_blocks, bs, positions, seq_of_row,
-                               tables, table_stride, rows, n_rows, nh, nkv, d, scale, window, chunk, n_splits, part,
-                               counters, err, stream);
+                               tables, table_stride, rows, n_rows, nh, nkv, d, opt, chunk, n_splits, part, counters, err,
+                               stream);
 }
 
 // Prefill form: tile i covers rows tile_row0[i] .. +tile_nrows[i]-1 (at most 64 consecutive rows of one request).
-// (softcap and sink as in the decode form)
-CUCA_API int cuca_attention_prefill_sv(const void* q, int q_stride, void* out, int out_stride, const void* kpool,
-                                       const void* vpool, int n_blocks, int bs, const int* positions,
-                                       const int* seq_of_row, const int* tables, int table_stride,
-                                       const int* tile_row0, const int* tile_nrows, int n_tiles, int nh, int nkv, int d,
-                                       float scale, int window, float softcap, int sink, const float* sink_val,
-                                       int* err, cudaStream_t stream) {
+CUCA_API int cuca_attention_prefill_o(const void* q, int q_stride, void* out, int out_stride, const void* kpool,
+                                      const void* vpool, int n_blocks, int bs, const int* positions,
+                                      const int* seq_of_row, const int* tables, int table_stride,
+                                      const int* tile_row0, const int* tile_nrows, int n_tiles, int nh, int nkv, int d,
+                                      const CucaAttnOptions* opt, int* err, cudaStream_t stream) {
   if (n_tiles == 0) return 0;
+  CUCA_REQUIRE(opt != nullptr && opt->window >= 0 && opt->keep >= 0, "attention_prefill: bad options");
   CUCA_REQUIRE(cuca_attention_mma_supported(nh, nkv, d, q_stride, out_stride), "attention_prefill: unsupported "
                "shape (heads %d/%d, head size %d)", nh, nkv, d);
   CUCA_REQUIRE(nh <= 65535, "attention_prefill: too many heads");
@@ -1122,12 +1179,24 @@ CUCA_API int cuca_attention_prefill_sv(const void* q, int q_stride, void* out, i
   p.kpool = (const __nv_bfloat16*)kpool; p.vpool = (const __nv_bfloat16*)vpool; p.n_blocks = n_blocks; p.bs = bs;
   p.tables = tables; p.table_stride = table_stride; p.positions = positions; p.seq_of_row = seq_of_row;
   p.rows = nullptr; p.tile_row0 = tile_row0; p.tile_nrows = tile_nrows; p.nh = nh; p.nkv = nkv;
-  p.scale_log2e = scale * 1.4426950408889634f; p.window = window; p.chunk = 0; p.part = nullptr;
+  p.chunk = 0; p.part = nullptr;
   p.counters = nullptr; p.err = err; p.slots = 1; p.cluster = 0;
-  set_score_options(p, scale, softcap, sink, sink_val);
+  set_score_options(p, *opt);
   p.partial = nullptr; p.n_slices = 0; p.slice_stride = 0; p.bias = nullptr; p.cos_t = p.sin_t = nullptr;
   p.table_rows = 0; p.rot = 0; p.has_kv = 0;
   return dispatch<false, false>(d, p, dim3(n_tiles, nh), stream);
+}
+
+// (softcap and sink as in the decode form)
+CUCA_API int cuca_attention_prefill_sv(const void* q, int q_stride, void* out, int out_stride, const void* kpool,
+                                       const void* vpool, int n_blocks, int bs, const int* positions,
+                                       const int* seq_of_row, const int* tables, int table_stride,
+                                       const int* tile_row0, const int* tile_nrows, int n_tiles, int nh, int nkv, int d,
+                                       float scale, int window, float softcap, int sink, const float* sink_val,
+                                       int* err, cudaStream_t stream) {
+  const CucaAttnOptions opt{scale, window, 0, softcap, sink, 0, sink_val, nullptr, nullptr};
+  return cuca_attention_prefill_o(q, q_stride, out, out_stride, kpool, vpool, n_blocks, bs, positions, seq_of_row, tables,
+                                  table_stride, tile_row0, tile_nrows, n_tiles, nh, nkv, d, &opt, err, stream);
 }
 
 CUCA_API int cuca_attention_prefill_s(const void* q, int q_stride, void* out, int out_stride, const void* kpool,

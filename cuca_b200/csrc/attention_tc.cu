@@ -20,6 +20,7 @@
 //
 // Every mbarrier wait is bounded; on a timeout the kernel records CUCA_ERR_WAIT_TIMEOUT, all roles stop, TMEM
 // is freed and the kernel returns.
+#include "attention_options.cuh"
 #include "tcgen05.cuh"
 #include <math.h>
 #include <stdlib.h>
@@ -65,6 +66,10 @@ struct Params {
   int sink;              // 1: the denominator holds one more exp(0) ...
   const float* sink_val; // ... or, when given, exp(sink_val[query head]) (32-bit, neither scaled nor capped)
   int window;
+  int keep;              // beside the window, the first `keep` keys of a request are seen (0 without a window)
+  const float* slopes;   // distance bias per query head (null: none): slopes[head] (position - key) is taken off a score
+  const __nv_bfloat16* gate;  // with it the result is multiplied by sigmoid(gate[row][head D + dim])
+  int gate_stride;
   int* err;
 };
 
@@ -217,8 +222,12 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
   const int pos0 = p.positions[row0];
   const int lo_min = (p.window > 0 && pos0 - (p.window - 1) > 0) ? pos0 - (p.window - 1) : 0;
   const int hi = pos0 + n_rows;                       // keys [lo_min, hi) matter
-  const int first_tile = lo_min / KEYS;
-  const int n_tiles = (hi - 1) / KEYS - first_tile + 1;
+  // ... and the first p.keep. Key tiles are counted without the gap between: the n_kept tiles that hold the first keys,
+  // then the window's from tile number window_tile on.
+  const int window_tile = lo_min / KEYS;
+  const int n_kept = min((p.keep + KEYS - 1) / KEYS, window_tile);
+  const int n_tiles = n_kept + (hi - 1) / KEYS - window_tile + 1;
+  auto tile_key0 = [&](int j) { return (j < n_kept ? j : window_tile + j - n_kept) * KEYS; };
   const int* table = p.tables + (size_t)(seq < 0 ? 0 : seq) * p.table_stride;
 
   if (threadIdx.x == 0) {
@@ -268,7 +277,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
       const int in_batch = j % per_batch;
       if (in_batch == 0) {
         const int tj = j + lane / pages;
-        const int kp = (first_tile + tj) * KEYS + (lane % pages) * p.bs;
+        const int kp = tile_key0(tj) + (lane % pages) * p.bs;
         entry = (lane < per_batch * pages && tj < n_tiles && kp < hi) ? table[kp / p.bs] : 0;
       }
       const int s = j % KV_STAGES;
@@ -284,10 +293,10 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
       const int pg = lane >> 2, which = lane & 3;
       int blk = __shfl_sync(0xffffffffu, entry, in_batch * pages + (pg < pages ? pg : 0));
       if (pg < pages && (which & 1) < D / 64) {
-        const int kp = (first_tile + j) * KEYS + pg * p.bs;
+        const int kp = tile_key0(j) + pg * p.bs;
         if (blk < 0 || blk >= p.n_blocks) {
           // keys before the window may have given their page back; they are masked. Anything else is an error.
-          if (kp + p.bs > lo_min && kp < hi && p.err) atomicExch(p.err, CUCA_ERR_BLOCK_RANGE);
+          if ((kp + p.bs > lo_min || kp < p.keep) && kp < hi && p.err) atomicExch(p.err, CUCA_ERR_BLOCK_RANGE);
           blk = 0;
         }
         const int grow = (blk * p.nkv + kvh) * p.bs;  // row of the page in the pool seen as [rows][D]
@@ -387,18 +396,40 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
     const int row_lo = (p.window > 0 && row_pos - (p.window - 1) > 0) ? row_pos - (p.window - 1) : 0;
     float m = -INFINITY, l = 0.f;
     bool ok = x < nq;
+    const bool biased = p.slopes != nullptr;
+    const float slope2 = (biased && ok) ? p.slopes[head0 + x] * CUCA_LOG2E : 0.f;
     for (int j = 0; ok && j < n_tiles; ++j) {
       // the tcgen05.ld/st below are warp-wide: a warp leaves the loop together or not at all
       if (!__all_sync(0xffffffffu, mbar_wait(&s_full[2 * x + (j & 1)], (j >> 1) & 1, p.err, abort_flag))) { ok = false; break; }
       tc_fence_after();
-      const int key0 = (first_tile + j) * KEYS;
-      const bool whole = key0 >= lo_min && key0 + KEYS - 1 <= pos0 && (p.window <= 0 || key0 >= pos0 + ROWS - 1 - (p.window - 1));
+      const int key0 = tile_key0(j);
+      const bool whole = key0 + KEYS - 1 <= pos0 &&
+                         (p.window <= 0 || key0 >= pos0 + ROWS - 1 - (p.window - 1) || key0 + KEYS <= p.keep);
       // pass 1: the whole row of scores in one round trip to tensor memory, then scale, mask, maximum
       constexpr int NC = KEYS / 32;  // groups of 32 scores
       uint32_t raw[NC][32];
 #pragma unroll
       for (int c = 0; c < NC; ++c) tmem_ld32_nowait(tmem_s(x, j) + lane_bits + c * 32, raw[c]);
       tmem_ld_wait();
+      const bool capped = p.cap_log2e > 0.f;
+      if (biased) {
+        // the distance bias differs from key to key, so the scores are made here, in log2 units: scale (q . k) (capped or
+        // not) - slope (row_pos - key0 - i)
+        const float c0 = slope2 * (float)(key0 - row_pos);
+        const float2 scale2 = make_float2(p.scale_log2e, p.scale_log2e), slope22 = make_float2(slope2, slope2), c02 = make_float2(c0, c0);
+#pragma unroll
+        for (int c = 0; c < NC; ++c) {
+#pragma unroll
+          for (int e = 0; e < 16; ++e) {
+            const float2 bias2 = __ffma2_rn(make_float2((float)(c * 32 + 2 * e), (float)(c * 32 + 2 * e + 1)), slope22, c02);
+            const float r0 = __uint_as_float(raw[c][2 * e]), r1 = __uint_as_float(raw[c][2 * e + 1]);
+            const float2 s2 = capped ? __fadd2_rn(make_float2(capped_log2(r0, p.cap_arg, p.cap_log2e), capped_log2(r1, p.cap_arg, p.cap_log2e)), bias2)
+                                     : __ffma2_rn(make_float2(r0, r1), scale2, bias2);
+            raw[c][2 * e] = __float_as_uint(s2.x);
+            raw[c][2 * e + 1] = __float_as_uint(s2.y);
+          }
+        }
+      }
       // the scale is positive, so the maximum is taken over the raw scores and scaled once; the scaling of every
       // score happens inside the exponent's multiply-add
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
@@ -414,15 +445,15 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
             const int kp = key0 + c * 32 + i;
-            if (!(row_ok && kp <= row_pos && kp >= row_lo)) raw[c][i] = 0xff800000u;  // -inf
+            if (!(row_ok && kp <= row_pos && (kp >= row_lo || kp < p.keep))) raw[c][i] = 0xff800000u;  // -inf
             mx4[i & 3] = fmaxf(mx4[i & 3], __uint_as_float(raw[c][i]));
           }
         }
       }
-      const bool capped = p.cap_log2e > 0.f;
       float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
       // (the cap grows with the score, so the largest raw score is the largest capped one)
-      mx = capped ? (mx == -INFINITY ? mx : capped_log2(mx, p.cap_arg, p.cap_log2e)) : mx * p.scale_log2e;
+      if (!biased)
+        mx = capped ? (mx == -INFINITY ? mx : capped_log2(mx, p.cap_arg, p.cap_log2e)) : mx * p.scale_log2e;
       // The running maximum only moves when the new one exceeds it by more than 8 (in log2 units): values up to
       // 2^8 above the reference are exact enough in 32-bit sums, and O is rescaled far less often.
       float m_new = m;
@@ -436,7 +467,19 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
       float2 sum2[2] = {make_float2(0.f, 0.f), make_float2(0.f, 0.f)};
       uint32_t pw[KEYS / 2];
       const float2 scale2 = make_float2(p.scale_log2e, p.scale_log2e), neg_m2 = make_float2(-m_use, -m_use);
-      if (capped) {
+      if (biased) {
+#pragma unroll
+        for (int c = 0; c < NC; ++c) {
+#pragma unroll
+          for (int e = 0; e < 16; ++e) {
+            const float2 x2 = __fadd2_rn(make_float2(__uint_as_float(raw[c][2 * e]), __uint_as_float(raw[c][2 * e + 1])), neg_m2);
+            const float2 p2 = make_float2(fast_exp2(x2.x), fast_exp2(x2.y));
+            sum2[e & 1] = __fadd2_rn(sum2[e & 1], p2);
+            __nv_bfloat162 t2 = __floats2bfloat162_rn(p2.x, p2.y);
+            pw[c * 16 + e] = *reinterpret_cast<uint32_t*>(&t2);
+          }
+        }
+      } else if (capped) {
         // two more exponent-unit operations per score (the tanh); a masked score stays masked
 #pragma unroll
         for (int c = 0; c < NC; ++c) {
@@ -500,6 +543,16 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
         float o[32];
         tmem_ld32(tmem_o(x) + lane_bits + c * 32, o);  // warp-wide: every lane reads, only rows of the tile store
         if (row_ok) {
+          if (p.gate) {
+            const __nv_bfloat16* gp = p.gate + (size_t)(row0 + r) * p.gate_stride + (size_t)(head0 + x) * D + c * 32;
+#pragma unroll
+            for (int q4 = 0; q4 < 4; ++q4) {
+              const uint4 gw = *reinterpret_cast<const uint4*>(gp + q4 * 8);
+              const __nv_bfloat16* gv = reinterpret_cast<const __nv_bfloat16*>(&gw);
+#pragma unroll
+              for (int i = 0; i < 8; ++i) o[q4 * 8 + i] *= __fdividef(1.f, 1.f + __expf(-__bfloat162float(gv[i])));
+            }
+          }
           uint32_t w[16];
 #pragma unroll
           for (int i = 0; i < 16; ++i) {
@@ -565,15 +618,17 @@ CUCA_API void cuca_attention_pair_tiles_mode(int mode) { pair_mode = mode; }
 
 // Prefill form on tcgen05: tile i covers rows tile_row0[i] .. +tile_nrows[i]-1 (at most 128 consecutive rows of
 // one request). q: [n_rows_total][q_stride] with the rotated query heads first; out: [..][out_stride].
-// sink: one more term without a value in every row's denominator, exp(0) or, with sink_val (32-bit, one number per
-// query head), exp(sink_val[head]).
-CUCA_API int cuca_attention_prefill_tc_sv(const void* q, int q_stride, int n_rows_total, void* out, int out_stride,
+CUCA_API int cuca_attention_prefill_tc_o(const void* q, int q_stride, int n_rows_total, void* out, int out_stride,
                                           const void* kpool, const void* vpool, int n_blocks, int bs,
                                           const int* positions, const int* seq_of_row, const int* tables,
                                           int table_stride, const int* tile_row0, const int* tile_nrows, int n_tiles,
-                                          int nh, int nkv, int d, float scale, int window, float softcap, int sink,
-                                          const float* sink_val, int* err, cudaStream_t stream) {
+                                          int nh, int nkv, int d, const CucaAttnOptions* opt, int* err,
+                                          cudaStream_t stream) {
   if (n_tiles == 0) return 0;
+  CUCA_REQUIRE(opt != nullptr && opt->window >= 0 && opt->keep >= 0, "attention_prefill_tc: bad options");
+  CUCA_REQUIRE(opt->gate == nullptr || (((uintptr_t)opt->gate & 15) == 0 && opt->gate_stride % 8 == 0),
+               "attention_prefill_tc: the gate's rows must be 16-byte aligned");
+  const float scale = opt->scale, softcap = opt->softcap;
   CUCA_REQUIRE(cuca_attention_tc_supported(nh, nkv, d, bs, q_stride, out_stride, q, kpool, vpool),
                "attention_prefill_tc: unsupported shape (heads %d/%d, head size %d, page %d)", nh, nkv, d, bs);
   CUCA_REQUIRE(nh <= 65535, "attention_prefill_tc: too many heads");
@@ -586,11 +641,12 @@ CUCA_API int cuca_attention_prefill_tc_sv(const void* q, int q_stride, int n_row
   p.out = (__nv_bfloat16*)out; p.out_stride = out_stride; p.tables = tables; p.table_stride = table_stride;
   p.positions = positions; p.seq_of_row = seq_of_row; p.tile_row0 = tile_row0; p.tile_nrows = tile_nrows;
   p.n_blocks = n_blocks; p.bs = bs; p.nh = nh; p.nkv = nkv; p.scale_log2e = scale * 1.4426950408889634f;
-  p.window = window; p.err = err;
+  p.window = opt->window; p.keep = opt->window > 0 ? opt->keep : 0; p.slopes = opt->slopes; p.err = err;
+  p.gate = (const __nv_bfloat16*)opt->gate; p.gate_stride = opt->gate_stride;
   p.cap_log2e = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
   p.cap_arg = softcap > 0.f ? 2.f * scale * 1.4426950408889634f / softcap : 0.f;
-  p.sink = sink ? 1 : 0;
-  p.sink_val = sink ? sink_val : nullptr;
+  p.sink = opt->sink ? 1 : 0;
+  p.sink_val = opt->sink ? opt->sink_val : nullptr;
   p.heads_per_cta = ((nh / nkv) % NQ == 0) ? NQ : 1;
   p.n_tiles = n_tiles;
   // Two tiles per CTA, a heavy and a light one, where that makes one round of CTAs out of more than one
@@ -600,6 +656,18 @@ CUCA_API int cuca_attention_prefill_tc_sv(const void* q, int q_stride, int n_row
   p.pair_tiles = n_tiles >= 2 && (pair_mode == 2 || (pair_mode == 1 && n_tiles * head_ctas > sms &&
                                                      ((n_tiles + 1) / 2) * head_ctas <= sms)) ? 1 : 0;
   return d == 128 ? launch_attn_tc<128>(tmQ, tmK, tmV, p, n_tiles, stream) : launch_attn_tc<64>(tmQ, tmK, tmV, p, n_tiles, stream);
+}
+
+CUCA_API int cuca_attention_prefill_tc_sv(const void* q, int q_stride, int n_rows_total, void* out, int out_stride,
+                                          const void* kpool, const void* vpool, int n_blocks, int bs,
+                                          const int* positions, const int* seq_of_row, const int* tables,
+                                          int table_stride, const int* tile_row0, const int* tile_nrows, int n_tiles,
+                                          int nh, int nkv, int d, float scale, int window, float softcap, int sink,
+                                          const float* sink_val, int* err, cudaStream_t stream) {
+  const CucaAttnOptions opt{scale, window, 0, softcap, sink, 0, sink_val, nullptr, nullptr};
+  return cuca_attention_prefill_tc_o(q, q_stride, n_rows_total, out, out_stride, kpool, vpool, n_blocks, bs, positions,
+                                     seq_of_row, tables, table_stride, tile_row0, tile_nrows, n_tiles, nh, nkv, d, &opt,
+                                     err, stream);
 }
 
 CUCA_API int cuca_attention_prefill_tc(const void* q, int q_stride, int n_rows_total, void* out, int out_stride,

@@ -87,6 +87,56 @@ CUCA_API int cuca_embed(const void* table, int table_dtype, const int* tokens, f
   return cuca_embed_scaled(table, table_dtype, tokens, x, n_rows, E, V, 1.f, err, stream);
 }
 
+// ---------------------------------------------------------------- embedding plus a learned position vector
+// x[r] = table[tokens[r]] * scale + pos_table[positions[r]] into the 32-bit stream. A token or position outside its table
+// is recorded and contributes nothing.
+template <typename T>
+__global__ void __launch_bounds__(256)
+embed_pos_kernel(const T* __restrict__ table, const T* __restrict__ pos_table, const int* __restrict__ tokens,
+                 const int* __restrict__ positions, float* __restrict__ x, int E, int V, int n_pos, float scale, int* err) {
+  pdl_trigger();
+  pdl_wait();
+  const size_t row = blockIdx.y;
+  const int tok = tokens[row], pos = positions[row];
+  const bool tok_ok = tok >= 0 && tok < V, pos_ok = pos >= 0 && pos < n_pos;
+  if (!(tok_ok && pos_ok) && blockIdx.x == 0 && threadIdx.x == 0 && err) atomicExch(err, CUCA_ERR_TOKEN_RANGE);
+  const T* a = table + (size_t)(tok_ok ? tok : 0) * E;
+  const T* b = pos_table + (size_t)(pos_ok ? pos : 0) * E;
+  const float fa = tok_ok ? scale : 0.f, fb = pos_ok ? 1.f : 0.f;
+  float* dst = x + row * E;
+  const int first = blockIdx.x * blockDim.x + threadIdx.x, step = gridDim.x * blockDim.x;
+  // four values a thread and round where the rows allow it
+  constexpr int A = 4 * sizeof(T) - 1;
+  if ((E & 3) == 0 && (((size_t)table | (size_t)pos_table) & A) == 0 && (((size_t)x) & 15) == 0) {
+    for (int i = first; i < (E >> 2); i += step) {
+      float va[4], vb[4];
+#pragma unroll
+      for (int k = 0; k < 4; ++k) { va[k] = to_f32(a[4 * i + k]); vb[k] = to_f32(b[4 * i + k]); }
+      reinterpret_cast<float4*>(dst)[i] = make_float4(va[0] * fa + vb[0] * fb, va[1] * fa + vb[1] * fb, va[2] * fa + vb[2] * fb, va[3] * fa + vb[3] * fb);
+    }
+    return;
+  }
+  for (int i = first; i < E; i += step) dst[i] = to_f32(a[i]) * fa + to_f32(b[i]) * fb;
+}
+
+CUCA_API int cuca_embed_pos(const void* table, const void* pos_table, int table_dtype, const int* tokens, const int* positions,
+                            float* x, int n_rows, int E, int V, int n_pos, float scale, int* err, cudaStream_t stream) {
+  if (n_rows == 0) return 0;
+  CUCA_REQUIRE(E > 0 && V > 0 && n_pos > 0, "embed_pos: bad sizes E=%d V=%d positions=%d", E, V, n_pos);
+  CUCA_REQUIRE(n_rows <= 65535, "embed_pos: %d rows in one step exceed the launch limit 65535", n_rows);
+  const dim3 grid((E + 1023) / 1024, n_rows);
+  if (table_dtype == CUCA_F32)
+    cuca_launch(embed_pos_kernel<float>, grid, dim3(256), 0, stream, true, (const float*)table, (const float*)pos_table,
+                tokens, positions, x, E, V, n_pos, scale, err);
+  else if (table_dtype == CUCA_BF16)
+    cuca_launch(embed_pos_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, true, (const __nv_bfloat16*)table,
+                (const __nv_bfloat16*)pos_table, tokens, positions, x, E, V, n_pos, scale, err);
+  else
+    CUCA_REQUIRE(false, "embed_pos: unknown dtype %d", table_dtype);
+  CUCA_CHECK_LAUNCH("embed_pos");
+  return 0;
+}
+
 // ---------------------------------------------------------------- embedding followed by an RMS norm
 // x[r] = e / sqrt(mean(e^2) + eps) * w with e = table[tokens[r]] * scale: the stream starts as the normed embedding
 // row. One block per row, two passes over the row (the second one hits the cache); the sum's order depends on E alone.

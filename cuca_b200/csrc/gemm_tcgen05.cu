@@ -78,6 +78,7 @@ struct Params {
   const float* col_w;
   int ld_w, w_run, w_cols;
   float glu_limit_s;
+  int act;          // the storing epilogue: 0: the result (plus bias), 1: relu(.)^2 of it
 };
 
 constexpr int STAGING_BUF = 32 * 128;  // 32 rows of 128 bytes
@@ -229,6 +230,13 @@ __device__ __forceinline__ float glu_act(const Params& p, const GluAt& at, float
   return silu_mul(g, u);
 }
 
+// the storing epilogue's activation
+__device__ __forceinline__ float act_of(const Params& p, float v) {
+  if (p.act == 0) return v;
+  v = fmaxf(v, 0.f);
+  return v * v;
+}
+
 // ---- epilogue of 16 accumulator columns held by one thread (TMEM lane `lane_row` of tile rows a0.., columns c..)
 template <int BN, bool DUAL, bool SWAP>
 __device__ __forceinline__ void store16(const Params& p, int a0, int b0, int lane_row, int c, const float (&v)[16],
@@ -246,8 +254,8 @@ __device__ __forceinline__ void store16(const Params& p, int a0, int b0, int lan
       if (DUAL) ((__nv_bfloat16*)p.out)[o] = __float2bfloat16_rn(glu_act(p, glu_at(p, m, n), v[j], u[j]));
       else if (p.epilogue == EPI_RESIDUAL) atomicAdd((float*)p.out + o, v[j] + bias);  // result unused: a fire-and-forget
                                                                                        // add; one thread owns the element
-      else if (p.out_f32) ((float*)p.out)[o] = v[j] + bias;
-      else ((__nv_bfloat16*)p.out)[o] = __float2bfloat16_rn(v[j] + bias);
+      else if (p.out_f32) ((float*)p.out)[o] = act_of(p, v[j] + bias);
+      else ((__nv_bfloat16*)p.out)[o] = __float2bfloat16_rn(act_of(p, v[j] + bias));
     }
   } else {
     // lane = token, columns = 16 consecutive features
@@ -265,6 +273,10 @@ __device__ __forceinline__ void store16(const Params& p, int a0, int b0, int lan
     if (!DUAL && p.bias) {
 #pragma unroll
       for (int j = 0; j < 16; ++j) if (n + j < p.N) r[j] += __bfloat162float(p.bias[n + j]);
+    }
+    if (!DUAL && p.act) {
+#pragma unroll
+      for (int j = 0; j < 16; ++j) r[j] = act_of(p, r[j]);
     }
     if (p.epilogue == EPI_RESIDUAL || p.out_f32) {
       float* dst = (float*)p.out + o;
@@ -340,6 +352,10 @@ __device__ __forceinline__ void tma_epilogue(const Params& p, const CUtensorMap*
 #pragma unroll
         for (int j = 0; j < 16; ++j)
           if (b0 + c + h + j < p.N) v[j] += __bfloat162float(p.bias[b0 + c + h + j]);
+      }
+      if (!DUAL && p.act) {
+#pragma unroll
+        for (int j = 0; j < 16; ++j) v[j] = act_of(p, v[j]);
       }
       if (p.out_f32) {
 #pragma unroll
@@ -1106,7 +1122,7 @@ static int gemm_tc_impl(const void* A, const void* W, const void* bias, void* ou
                         int K, int lda, int ldo, int epilogue, void* workspace, size_t ws_bytes, int* counters,
                         int n_counters, int max_splits, int* n_slices_out, int* err, cudaStream_t stream,
                         float glu_limit = 0.f, float glu_alpha = 1.f, const float* col_w = nullptr, int ld_w = 0,
-                        int w_run = 16, int w_cols = 0, float glu_limit_s = 0.f) {
+                        int w_run = 16, int w_cols = 0, float glu_limit_s = 0.f, int act = 0) {
   if (M == 0 || N == 0) return 0;
   if (!cuca_gemm_tc_supported(A, W, M, N, K, lda)) return 1;
   CUCA_REQUIRE(epilogue != EPI_RESIDUAL || out_dtype == CUCA_F32, "gemm_tc: the residual stream is 32-bit");
@@ -1125,7 +1141,7 @@ static int gemm_tc_impl(const void* A, const void* W, const void* bias, void* ou
     p.out = out; p.bias = nullptr; p.workspace = nullptr; p.counters = nullptr; p.err = err;
     p.M = M; p.N = N; p.K = K; p.ldo = N; p.epilogue = EPI_PARTIAL; p.out_f32 = 1;
     p.glu_limit = 0.f; p.glu_alpha = 1.f;
-    p.col_w = nullptr; p.ld_w = p.w_cols = 0; p.w_run = 16; p.glu_limit_s = 0.f;
+    p.col_w = nullptr; p.ld_w = p.w_cols = 0; p.w_run = 16; p.glu_limit_s = 0.f; p.act = 0;
     p.tile_rows = 2 * TILE_A;
     p.tiles_a = (M + 255) / 256;
     p.tiles = p.tiles_a * ((N + 255) / 256);
@@ -1157,7 +1173,7 @@ static int gemm_tc_impl(const void* A, const void* W, const void* bias, void* ou
   if (!tma_out) tmO = tmA;  // unused
   Params p;
   p.glu_limit = glu_limit; p.glu_alpha = glu_alpha;
-  p.col_w = col_w; p.ld_w = ld_w; p.w_run = w_run; p.w_cols = w_cols; p.glu_limit_s = glu_limit_s;
+  p.col_w = col_w; p.ld_w = ld_w; p.w_run = w_run; p.w_cols = w_cols; p.glu_limit_s = glu_limit_s; p.act = act;
   p.out = out; p.bias = (const __nv_bfloat16*)bias; p.workspace = (float*)workspace; p.counters = counters;
   p.err = err; p.M = M; p.N = N; p.K = K; p.ldo = ldo; p.epilogue = epilogue; p.out_f32 = out_dtype == CUCA_F32;
   const int out_cols = swap ? bn : (dual ? 128 : 256);
@@ -1323,6 +1339,15 @@ CUCA_API int cuca_gemm_tc(const void* A, const void* W, const void* bias, void* 
   CUCA_REQUIRE(epilogue != EPI_PARTIAL, "gemm_tc: use cuca_gemm_tc_partial for partial sums");
   return gemm_tc_impl(A, W, bias, out, out_dtype, M, N, K, lda, ldo, epilogue, workspace, ws_bytes, counters,
                       n_counters, max_splits, nullptr, err, stream);
+}
+
+// out[M, N] = act(A W^T + bias), the activation as the contraction's epilogue; act 1: relu(.)^2.
+CUCA_API int cuca_gemm_tc_act(const void* A, const void* W, const void* bias, void* out, int out_dtype, int M, int N, int K,
+                              int lda, int ldo, int act, void* workspace, size_t ws_bytes, int* counters, int n_counters,
+                              int max_splits, int* err, cudaStream_t stream) {
+  CUCA_REQUIRE(act == 1, "gemm_tc_act: unknown activation %d", act);
+  return gemm_tc_impl(A, W, bias, out, out_dtype, M, N, K, lda, ldo, EPI_STORE, workspace, ws_bytes, counters, n_counters,
+                      max_splits, nullptr, err, stream, 0.f, 1.f, nullptr, 0, 16, 0, 0.f, act);
 }
 
 // out[M, N] = act(A W^T) for W [2 N, K] = [gate rows; up rows], bf16 out: the gated epilogue with capped inputs,

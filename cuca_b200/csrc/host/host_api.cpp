@@ -26,12 +26,14 @@ HOST_API int cuca_host_blockpool_free_count(void* h) { return ((BlockPool*)h)->f
 HOST_API void cuca_host_blockpool_reset(void* h) { ((BlockPool*)h)->reset(); }
 
 // ------------------------------------------------------------------ pools
-HOST_API void* cuca_host_pools_new(int n_groups, const int* n_blocks, const int* windows, int block_size) {
+// windows: < 0 all positions; keeps: the first positions a windowed group keeps beside its window (null: none)
+HOST_API void* cuca_host_pools_new(int n_groups, const int* n_blocks, const int* windows, const int* keeps, int block_size) {
   if (n_groups < 0 || block_size <= 0) return nullptr;
   std::vector<Group> groups;
   for (int g = 0; g < n_groups; ++g) {
     if (n_blocks[g] <= 0) return nullptr;
-    groups.push_back(Group{n_blocks[g], windows[g]});
+    if (keeps && keeps[g] < 0) return nullptr;
+    groups.push_back(Group{n_blocks[g], windows[g], keeps ? keeps[g] : 0});
   }
   return new KvPools(groups, block_size);
 }

@@ -210,6 +210,20 @@ void KvPools::owed(int handle, int tokens, int* out) {
   }
 }
 
+void KvPools::owed_in_steps(int handle, int tokens, int step_tokens, int* out) {
+  owed(handle, tokens, out);
+  SeqBlocks* s = handle >= 0 ? seq(handle) : nullptr;
+  for (size_t g = 0; g < groups_.size(); ++g) {
+    if (groups_[g].window < 0) continue;
+    int held = 0;
+    if (s)
+      for (int b : s->tables[g]) held += b != NO_BLOCK;
+    // (the window may begin, and the step end, inside a page)
+    const int most = blocks_for(groups_[g].window - 1 + step_tokens) + 1 + kept_blocks(g);
+    out[g] = std::min(out[g], std::max(0, most - held));
+  }
+}
+
 bool KvPools::can_give(const int* owed) const {
   for (size_t g = 0; g < groups_.size(); ++g)
     if (pools_[g].free_count() < owed[g]) return false;
@@ -243,7 +257,7 @@ int KvPools::release_window(int handle) {
     const int first_needed = std::max(0, s->length - (window - 1));
     std::vector<int>& table = s->tables[g];
     const int upto = std::min(first_needed / block_size_, (int)table.size());
-    for (int i = s->first_live[g]; i < upto; ++i) {
+    for (int i = std::max(s->first_live[g], kept_blocks(g)); i < upto; ++i) {
       if (table[i] == NO_BLOCK) continue;
       if (!pools_[g].release(table[i])) {
         fail(BOOKKEEPING, "page " + std::to_string(table[i]) + " is freed but not held");
@@ -371,8 +385,8 @@ int KvPools::new_seq_with_prefix(const int* prompt, int n) {
     if (!everywhere) break;
     names.push_back(nm);
   }
-  // a windowed group needs only the pages its window still reaches from the prefix's end; pages before that
-  // may be gone. Shrink the prefix until every windowed group has the tail it needs.
+  // a windowed group needs only the pages its window still reaches from the prefix's end, and those of the first
+  // positions it keeps; the pages between may be gone. Shrink the prefix until every windowed group has the tail it needs.
   auto tail_begin = [&](int g, int depth) {
     return std::max(0, depth * block_size_ - (groups_[g].window - 1)) / block_size_;
   };
@@ -381,6 +395,8 @@ int KvPools::new_seq_with_prefix(const int* prompt, int n) {
     bool tails = true;
     for (size_t g = 0; g < groups_.size() && tails; ++g) {
       if (groups_[g].window < 0) continue;
+      const int head = std::min(kept_blocks(g), depth);
+      for (int i = 0; i < head && tails; ++i) tails = pools_[g].holds(names[i]);
       for (int i = tail_begin((int)g, depth); i < depth && tails; ++i) tails = pools_[g].holds(names[i]);
     }
     if (tails) break;
@@ -389,8 +405,9 @@ int KvPools::new_seq_with_prefix(const int* prompt, int n) {
   SeqBlocks& s = seqs_[h];
   for (size_t g = 0; g < groups_.size(); ++g) {
     const int from = groups_[g].window >= 0 ? tail_begin((int)g, depth) : 0;
-    s.tables[g].assign(from, NO_BLOCK);
-    for (int i = from; i < depth; ++i) s.tables[g].push_back(pools_[g].take(names[i]));  // found above: never -1
+    const int head = std::min(kept_blocks(g), from);
+    for (int i = 0; i < depth; ++i)  // found above: never -1
+      s.tables[g].push_back(i < head || i >= from ? pools_[g].take(names[i]) : NO_BLOCK);
     s.first_live[g] = from;
   }
   s.length = depth * block_size_;

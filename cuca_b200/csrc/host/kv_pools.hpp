@@ -3,7 +3,8 @@
 // A page (block) is `block_size` consecutive positions of one request, for every cache of a group; layers whose
 // mixers have equal needs share a group, each group has a pool of its own, and each request has one block table
 // per group (src/provider/local/model/paged.rs:6-16,52-103,344-489 of the reference). Pages go back to the pool
-// when a request ends and, in a windowed group, as soon as the window has passed them (model/paged.rs:736-761).
+// when a request ends and, in a windowed group, as soon as the window has passed them (model/paged.rs:736-761);
+// the pages of the first positions that a group keeps beside its window stay until the request ends.
 // No device memory lives here: the page ids index slabs that the Python side allocates.
 //
 // Prefix store (behaviour of model/paged.rs:18-35,257-321,344-480,831-928): a full page is named by a hash chain over the
@@ -77,6 +78,7 @@ class BlockPool {
 struct Group {
   int n_blocks;
   int window;  // positions a query of this group sees, itself included; < 0: all
+  int keep = 0;  // beside the window, a query sees the first `keep` positions of its request: their pages stay
 };
 
 // One request's block tables (one per group) and how many positions it has cached.
@@ -105,6 +107,9 @@ class KvPools {
   SeqBlocks* seq(int handle);          // nullptr for a handle that is not in use
   int blocks_for(int tokens) const { return (tokens + block_size_ - 1) / block_size_; }
   void owed(int seq, int tokens, int* out);      // seq < 0: a request that holds nothing yet
+  // The same for a request that is run in steps of at most `step_tokens` tokens: in a windowed group pages go back on
+  // the way, so it never holds more than its window, its kept pages and one step's tokens take.
+  void owed_in_steps(int seq, int tokens, int step_tokens, int* out);
   bool can_give(const int* owed) const;
   Status reserve(int seq, int upto);             // all or nothing
   int release_window(int seq);                   // pages given back, or -1 on a bookkeeping error
@@ -123,6 +128,7 @@ class KvPools {
 
  private:
   Status fail(Status s, const std::string& msg) { error_ = msg; return s; }
+  int kept_blocks(size_t g) const { return groups_[g].window < 0 ? 0 : blocks_for(groups_[g].keep); }
   std::vector<Group> groups_;
   int block_size_;
   std::vector<BlockPool> pools_;

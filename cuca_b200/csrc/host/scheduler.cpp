@@ -52,7 +52,7 @@ void Scheduler::committed(std::vector<int>& total) {
   for (int id : running_) {
     const Sequence& s = seqs_[id];
     if (s.phase != PH_PREFILL) continue;
-    pools_.owed(s.blocks, (int)s.prompt.size() + 1, owed.data());
+    pools_.owed_in_steps(s.blocks, (int)s.prompt.size() + 1, cfg_.max_step_tokens, owed.data());
     for (int g = 0; g < G; ++g) total[g] += owed[g];
   }
 }
@@ -67,7 +67,7 @@ void Scheduler::admit() {
     // with the prefix cache the request starts from the pages that already hold the head of its prompt
     // (src/provider/local/engine/scheduler.rs:805-813)
     const int blocks = cfg_.prefix_cache ? pools_.new_seq_with_prefix(s.prompt.data(), (int)s.prompt.size()) : pools_.new_seq();
-    pools_.owed(blocks, (int)s.prompt.size() + 1, owed.data());
+    pools_.owed_in_steps(blocks, (int)s.prompt.size() + 1, cfg_.max_step_tokens, owed.data());
     for (int g = 0; g < G; ++g) need[g] = com[g] + owed[g];
     if (!pools_.can_give(need.data())) {
       const bool never = running_.empty() && !pools_.can_give(owed.data());

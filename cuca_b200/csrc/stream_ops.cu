@@ -1,7 +1,7 @@
 // Kernels around the 32-bit residual stream for blocks that norm a sublayer's input AND its output:
 //   norm_shift      h = shift(norm(x)), the previous token's normed row mixed in, its last row kept per request
 //   post_norm_add   x += norm(y) * g, and optionally f = norm(x) * g2 of the new row in the same pass
-//   gelu, scale, concat2 (two streams side by side in the compute dtype, for a contraction over both)
+//   gelu, relu2, scale, concat2 (two streams side by side in the compute dtype, for a contraction over both)
 // A norm's gain is a vector or a single number (gain_stride 1 or 0). All arithmetic is 32-bit, and a row's
 // reduction order depends on the width alone, so its bits do not depend on the batch it is in.
 #include "common.cuh"
@@ -91,14 +91,16 @@ post_norm_add_kernel(float* __restrict__ x, const float* __restrict__ y, const f
   for (int i = threadIdx.x; i < E; i += NT) out[row * E + i] = from_f32<TO>(xr[i] * ix * gain2[i * gain2_stride]);
 }
 
-__device__ __forceinline__ float gelu_of(float z, int tanh_form) {
-  if (tanh_form) return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+// form 0: gelu (erf), 1: its tanh form, 2: the square of relu
+__device__ __forceinline__ float activation_of(float z, int form) {
+  if (form == 2) return fmaxf(z, 0.f) * fmaxf(z, 0.f);
+  if (form == 1) return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
   return 0.5f * z * (1.f + erff(z * 0.7071067811865476f));
 }
 
 // 16 bytes per thread and round where the tensor allows it (n_vec pieces), the rest value by value
 template <typename T>
-__global__ void gelu_kernel(T* __restrict__ a, size_t n, size_t n_vec, int tanh_form) {
+__global__ void activation_kernel(T* __restrict__ a, size_t n, size_t n_vec, int form) {
   pdl_trigger();
   pdl_wait();
   constexpr int PER = 16 / sizeof(T);
@@ -107,10 +109,10 @@ __global__ void gelu_kernel(T* __restrict__ a, size_t n, size_t n_vec, int tanh_
     uint4 w = reinterpret_cast<uint4*>(a)[i];
     T* v = reinterpret_cast<T*>(&w);
 #pragma unroll
-    for (int k = 0; k < PER; ++k) v[k] = from_f32<T>(gelu_of(to_f32(v[k]), tanh_form));
+    for (int k = 0; k < PER; ++k) v[k] = from_f32<T>(activation_of(to_f32(v[k]), form));
     reinterpret_cast<uint4*>(a)[i] = w;
   }
-  for (size_t i = n_vec * PER + first; i < n; i += stride) a[i] = from_f32<T>(gelu_of(to_f32(a[i]), tanh_form));
+  for (size_t i = n_vec * PER + first; i < n; i += stride) a[i] = from_f32<T>(activation_of(to_f32(a[i]), form));
 }
 
 __global__ void scale_kernel(float* __restrict__ a, size_t n, float s) {
@@ -180,23 +182,29 @@ CUCA_API int cuca_post_norm_add(float* x, const float* y, const float* gain, int
   return 0;
 }
 
-// a = gelu(a) in place: the exact form (erf), or the tanh form 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))).
-CUCA_API int cuca_gelu(void* a, int dtype, size_t n, int tanh_form, cudaStream_t stream) {
+// a = act(a) in place: 0 the exact gelu (erf), 1 its tanh form 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))), 2 the
+// square of relu.
+CUCA_API int cuca_activation(void* a, int dtype, size_t n, int form, cudaStream_t stream) {
   if (n == 0) return 0;
+  CUCA_REQUIRE(form >= 0 && form <= 2, "activation: unknown form %d", form);
   const bool aligned = (((size_t)a) & 15) == 0;
   if (dtype == CUCA_F32) {
     const size_t nv = aligned ? n / 4 : 0;
-    cuca_launch(gelu_kernel<float>, dim3(flat_grid(nv > 0 ? nv : n, 256)), dim3(256), 0, stream, true, (float*)a, n, nv,
-                tanh_form);
+    cuca_launch(activation_kernel<float>, dim3(flat_grid(nv > 0 ? nv : n, 256)), dim3(256), 0, stream, true, (float*)a, n,
+                nv, form);
   } else if (dtype == CUCA_BF16) {
     const size_t nv = aligned ? n / 8 : 0;
-    cuca_launch(gelu_kernel<__nv_bfloat16>, dim3(flat_grid(nv > 0 ? nv : n, 256)), dim3(256), 0, stream, true,
-                (__nv_bfloat16*)a, n, nv, tanh_form);
+    cuca_launch(activation_kernel<__nv_bfloat16>, dim3(flat_grid(nv > 0 ? nv : n, 256)), dim3(256), 0, stream, true,
+                (__nv_bfloat16*)a, n, nv, form);
   }
   else
-    CUCA_REQUIRE(false, "gelu: unknown dtype %d", dtype);
-  CUCA_CHECK_LAUNCH("gelu");
+    CUCA_REQUIRE(false, "activation: unknown dtype %d", dtype);
+  CUCA_CHECK_LAUNCH("activation");
   return 0;
+}
+
+CUCA_API int cuca_gelu(void* a, int dtype, size_t n, int tanh_form, cudaStream_t stream) {
+  return cuca_activation(a, dtype, n, tanh_form ? 1 : 0, stream);
 }
 
 CUCA_API int cuca_scale(float* a, size_t n, float s, cudaStream_t stream) {

@@ -10,80 +10,10 @@
 //   row_norm_gate   out = o / rms(o) * w * sigmoid(gate), over whole rows
 // All arithmetic is 32-bit. Terms and slices are added in their order; a row's reduction order depends on the width
 // and on how many values a thread holds, which follows the number of rows.
-#include "common.cuh"
+#include "terms.cuh"
 #include <math.h>
 
-#define CUCA_MAX_TERMS 8
-struct CucaTerms {  // (passed from Python by address: keep in step with kernels/ops.py)
-  int n;
-  const float* data[CUCA_MAX_TERMS];
-  int slices[CUCA_MAX_TERMS];
-  size_t stride[CUCA_MAX_TERMS];  // between slices, in values
-  float scale[CUCA_MAX_TERMS];
-};
-
 namespace {
-
-template <int V> struct Pack;
-template <> struct Pack<1> { float v[1]; };
-template <> struct alignas(16) Pack<4> { float v[4]; };
-template <int V> __device__ __forceinline__ Pack<V> ld(const float* p) { return *reinterpret_cast<const Pack<V>*>(p); }
-template <int V> __device__ __forceinline__ void st(float* p, const Pack<V>& x) { *reinterpret_cast<Pack<V>*>(p) = x; }
-template <int V> __device__ __forceinline__ void st(__nv_bfloat16* p, const Pack<V>& x) {
-  if (V == 4) {
-    const __nv_bfloat162 lo = __floats2bfloat162_rn(x.v[0], x.v[V > 1 ? 1 : 0]);
-    const __nv_bfloat162 hi = __floats2bfloat162_rn(x.v[V > 2 ? 2 : 0], x.v[V > 3 ? 3 : 0]);
-    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
-  } else {
-    p[0] = __float2bfloat16_rn(x.v[0]);
-  }
-}
-// (slices come from the kernel before this one: past L1, which a dependent launch does not find invalidated)
-template <int V> __device__ __forceinline__ Pack<V> ld_cg(const float* p) {
-  Pack<V> r;
-  if (V == 4) {
-    const float4 f = __ldcg(reinterpret_cast<const float4*>(p));
-    r.v[0] = f.x;
-    if (V > 1) r.v[V > 1 ? 1 : 0] = f.y;
-    if (V > 2) r.v[V > 2 ? 2 : 0] = f.z;
-    if (V > 3) r.v[V > 3 ? 3 : 0] = f.w;
-  } else {
-    r.v[0] = __ldcg(p);
-  }
-  return r;
-}
-
-// y[at .. at + V) of the weighted sum of the terms
-template <int V>
-__device__ __forceinline__ Pack<V> term_sum(const CucaTerms& t, size_t at) {
-  Pack<V> y;
-#pragma unroll
-  for (int k = 0; k < V; ++k) y.v[k] = 0.f;
-  for (int i = 0; i < t.n; ++i) {
-    const float* p = t.data[i] + at;
-    Pack<V> s;
-#pragma unroll
-    for (int k = 0; k < V; ++k) s.v[k] = 0.f;
-    for (int k0 = 0; k0 < t.slices[i]; k0 += 4) {  // four slices' loads in flight at once, added in slice order
-      Pack<V> q[4];
-#pragma unroll
-      for (int u = 0; u < 4; ++u) {
-        if (k0 + u < t.slices[i]) q[u] = ld_cg<V>(p + (k0 + u) * t.stride[i]);
-        else {
-#pragma unroll
-          for (int k = 0; k < V; ++k) q[u].v[k] = 0.f;
-        }
-      }
-#pragma unroll
-      for (int u = 0; u < 4; ++u)
-#pragma unroll
-        for (int k = 0; k < V; ++k) s.v[k] += q[u].v[k];
-    }
-#pragma unroll
-    for (int k = 0; k < V; ++k) y.v[k] = fmaf(t.scale[i], s.v[k], y.v[k]);
-  }
-  return y;
-}
 
 __device__ __forceinline__ float block_sum(float s, float* red) {
   s = warp_sum(s);
@@ -258,14 +188,6 @@ row_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ w, c
   }
 }
 
-bool aligned(const void* p, size_t a) { return ((uintptr_t)p & (a - 1)) == 0; }
-
-bool terms_wide(const CucaTerms& t) {
-  for (int i = 0; i < t.n; ++i)
-    if (!aligned(t.data[i], 16) || t.stride[i] % 4 != 0) return false;
-  return true;
-}
-
 // threads and held packs for rows of `packs` packs: few rows get as many threads as a row has packs, many rows a
 // quarter of that with four packs each
 void norm_shape(int packs, int n_rows, int* threads, int* held) {
@@ -300,7 +222,7 @@ CUCA_API int cuca_norm_add(float* x, const CucaTerms* terms, const float* w, voi
                            float eps, int center, cudaStream_t stream) {
   if (n_rows == 0) return 0;
   CUCA_REQUIRE(E > 0 && terms && terms->n >= 0 && terms->n <= CUCA_MAX_TERMS, "norm_add: bad sizes (E=%d)", E);
-  const bool wide = E % 4 == 0 && terms_wide(*terms) && aligned(x, 16) && aligned(w, 16) && aligned(out, 16);
+  const bool wide = E % 4 == 0 && terms_wide(*terms) && aligned_to(x, 16) && aligned_to(w, 16) && aligned_to(out, 16);
 #define NA(TO)                                                                                                         \
   do {                                                                                                                 \
     if (wide) launch_norm<TO, true, 4>(x, *terms, w, (TO*)out, nullptr, n_rows, E, eps, center, stream);               \
@@ -321,7 +243,7 @@ CUCA_API int cuca_layer_norm(const float* x, const float* w, void* out, int out_
   CUCA_REQUIRE(E > 0, "layer_norm: bad width %d", E);
   CucaTerms none = {};
   float* xm = const_cast<float*>(x);  // not written
-  const bool wide = E % 4 == 0 && aligned(x, 16) && aligned(w, 16) && aligned(out, 16);
+  const bool wide = E % 4 == 0 && aligned_to(x, 16) && aligned_to(w, 16) && aligned_to(out, 16);
 #define LN(TO)                                                                                                         \
   do {                                                                                                                 \
     if (wide) launch_norm<TO, false, 4>(xm, none, w, (TO*)out, rows, n_rows, E, eps, 1, stream);                       \
@@ -343,7 +265,7 @@ static unsigned grid_for(size_t work) {
 CUCA_API int cuca_add_terms(float* x, const CucaTerms* terms, int store, size_t n, cudaStream_t stream) {
   if (n == 0) return 0;
   CUCA_REQUIRE(terms && terms->n >= 0 && terms->n <= CUCA_MAX_TERMS, "add_terms: bad terms");
-  if (n % 4 == 0 && terms_wide(*terms) && aligned(x, 16))
+  if (n % 4 == 0 && terms_wide(*terms) && aligned_to(x, 16))
     cuca_launch(add_terms_kernel<4>, dim3(grid_for(n / 4)), dim3(256), 0, stream, true, x, *terms, store, n);
   else
     cuca_launch(add_terms_kernel<1>, dim3(grid_for(n)), dim3(256), 0, stream, true, x, *terms, store, n);
@@ -353,7 +275,7 @@ CUCA_API int cuca_add_terms(float* x, const CucaTerms* terms, int store, size_t 
 
 CUCA_API int cuca_round_rows(const float* x, void* out, int out_dtype, size_t n, cudaStream_t stream) {
   if (n == 0) return 0;
-  const bool wide = n % 4 == 0 && aligned(x, 16) && aligned(out, 16);
+  const bool wide = n % 4 == 0 && aligned_to(x, 16) && aligned_to(out, 16);
 #define RR(TO)                                                                                                         \
   do {                                                                                                                 \
     if (wide) cuca_launch(round_rows_kernel<TO, 4>, dim3(grid_for(n / 4)), dim3(256), 0, stream, true, x, (TO*)out, n); \
@@ -372,8 +294,8 @@ CUCA_API int cuca_row_norm_gate(const float* o, const float* w, const void* gate
                                 int out_dtype, int n_rows, int n, float eps, cudaStream_t stream) {
   if (n_rows == 0) return 0;
   CUCA_REQUIRE(n > 0, "row_norm_gate: bad width %d", n);
-  const bool wide = n % 4 == 0 && ldg % 4 == 0 && aligned(o, 16) && aligned(w, 16) && aligned(gate, gate_dtype == CUCA_F32 ? 16 : 8) &&
-                    aligned(out, 16);
+  const bool wide = n % 4 == 0 && ldg % 4 == 0 && aligned_to(o, 16) && aligned_to(w, 16) && aligned_to(gate, gate_dtype == CUCA_F32 ? 16 : 8) &&
+                    aligned_to(out, 16);
   const int packs = wide ? n / 4 : n;
   int threads = (packs + 31) / 32 * 32;
   threads = threads > 512 ? 512 : threads;

@@ -160,6 +160,20 @@ _SIGNATURES = {
     "cuca_moe_router_grouped": [_P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P, _P, _P],
     "cuca_gemm_tc_glu_experts": [_P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _F, _P, _I, _I, _I, _P, c_size_t, _P, _I, _I, _P,
                                  _P],
+    "cuca_attention_generic_o": [_P, _I, _P, _I, _I, _P, _P, _I, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _P, _P],
+    "cuca_attention_decode_o": [_P, _I, _P, _I, _P, _P, _I, _I, _P, _P, _P, _I, _P, _I, _I, _I, _I, _P, _I, _I, _P, _P, _P,
+                                _P],
+    "cuca_attention_prefill_o": [_P, _I, _P, _I, _P, _P, _I, _I, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _P, _P, _P],
+    "cuca_attention_prefill_tc_o": [_P, _I, _I, _P, _I, _P, _P, _I, _I, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _P, _P, _P],
+    "cuca_norm_rope_store_u": [_P, _I, _I, _I, _I, _P, _I, _P, _P, _P, _I, _P, _P, _I, _I, _I, _P, _P, _I, _F, _P, _P,
+                               _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _P, _P, _P],
+    "cuca_gemm_tc_act": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, c_size_t, _P, _I, _I, _P, _P],
+    "cuca_activation": [_P, _I, c_size_t, _I, _P],
+    "cuca_embed_pos": [_P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _F, _P, _P],
+    "cuca_sum_norm": [_P, _P, _P, _P, _F, _F, _P, _I, _I, _I, _P],
+    "cuca_sum_norm_shift_supported": [_I],
+    "cuca_sum_norm_shift": [_P, _P, _P, _P, _F, _F, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _P],
+    "cuca_shift_rows": [_P, _P, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _P],
     "cuca_moe_glu_capped_dense": [_P, _P, _I, _P, _I, _I, _I, _I, _I, _F, _F, _F, _P],
 }
 

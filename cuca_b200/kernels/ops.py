@@ -56,6 +56,15 @@ def embed(table: torch.Tensor, tokens: torch.Tensor, out: torch.Tensor, err: tor
                                         float(scale), _p(err), _stream()), "embed")
 
 
+def embed_pos(table, pos_table, tokens, positions, out, err, scale: float = 1.0) -> None:
+    """out[r] = table[tokens[r]] * scale + pos_table[positions[r]], into the 32-bit stream."""
+    _cuda(table, pos_table, tokens, positions, out)
+    V, E = table.shape
+    library.check(library.load().cuca_embed_pos(_p(table), _p(pos_table), dtype_code(table.dtype), _p(tokens), _p(positions),
+                                                _p(out), tokens.shape[0], E, V, pos_table.shape[0], float(scale), _p(err),
+                                                _stream()), "embed_pos")
+
+
 def embed_norm(table, tokens, out, weight, eps: float, err, scale: float = 1.0) -> None:
     """out[r] = e / sqrt(mean(e^2) + eps) * weight with e = table[tokens[r]] * scale, into the 32-bit stream."""
     _cuda(table, tokens, out, weight)
@@ -155,6 +164,34 @@ def gemm_simt(a, w, out, epilogue=EPI_STORE, bias=None) -> None:
                                      M, N, K, a.stride(0), out.stride(0), epilogue, _stream()), "gemm_simt")
 
 
+class AttentionOptions(ctypes.Structure):
+    """What the attention kernels take besides queries, pages and sizes (`csrc/attention_options.cuh`)."""
+
+    _fields_ = [("scale", ctypes.c_float), ("window", ctypes.c_int), ("keep", ctypes.c_int), ("softcap", ctypes.c_float),
+                ("sink", ctypes.c_int), ("gate_stride", ctypes.c_int), ("sink_val", ctypes.c_void_p),
+                ("slopes", ctypes.c_void_p), ("gate", ctypes.c_void_p)]
+
+
+def attention_options(n_heads, scale, window=None, softcap=0.0, sink=False, sink_values=None, keep_first=0, slopes=None,
+                      gate=None, gate_width=None) -> AttentionOptions:
+    """`window` w: a query sees the last w keys, itself included, and with `keep_first` k the first k of its request as
+    well (None: all keys). `softcap` c > 0: a scaled score s becomes c tanh(s / c). `slopes` (32-bit, one per query
+    head): slope * distance is taken off a score. `sink`: every row's denominator holds one more exp(0) that has no
+    value, or exp(sink_values[head]) (32-bit, one number per query head) when those are given. `gate` ([rows,
+    gate_width], of the output's dtype): the result is multiplied by sigmoid(gate)."""
+    o = AttentionOptions()
+    o.scale, o.window, o.softcap = float(scale), int(window or 0), float(softcap or 0.0)
+    o.keep = int(keep_first or 0) if window else 0
+    o.sink, o.sink_val = int(bool(sink)), _per_head(sink_values, n_heads, "a sink's scores")
+    o.slopes = _per_head(slopes, n_heads, "distance slopes")
+    if gate is not None:
+        _cuda(gate)
+        if gate.dim() != 2 or gate.stride(1) != 1 or (gate_width is not None and gate.shape[1] < gate_width):
+            raise library.KernelError(f"an output gate is [rows, {gate_width}] with contiguous rows, not {tuple(gate.shape)}")
+        o.gate, o.gate_stride = gate.data_ptr(), gate.stride(0)
+    return o
+
+
 def attention_generic(q, q_stride, out, kpool, vpool, positions, seq_of_row, tables, n_heads, n_kv_heads,
                       head_dim, scale, window, err) -> None:
     _cuda(q, out, kpool, vpool)
@@ -212,6 +249,20 @@ def gemm_tc(a, w, out, epilogue=EPI_STORE, bias=None, err=None, max_splits=16) -
     library.check(lib.cuca_gemm_tc(_p(a), _p(w), _p(bias), _p(out), dtype_code(out.dtype), M, N, K, a.stride(0),
                                    out.stride(0), epilogue, _p(ws), ws.numel() * 4, _p(counters), counters.numel(),
                                    int(max_splits), _p(err), _stream()), "gemm_tc")
+
+
+ACT_RELU2 = 1  # `gemm_tc_act`
+
+
+def gemm_tc_act(a, w, out, act: int, bias=None, err=None, max_splits=16) -> None:
+    """out = act(a @ w.T + bias) as the contraction's epilogue, from the 32-bit sums; act: ACT_RELU2."""
+    _cuda(a, w, out)
+    M, K = a.shape
+    ws, counters = gemm_scratch(a.device)
+    library.check(library.load().cuca_gemm_tc_act(_p(a), _p(w), _p(bias), _p(out), dtype_code(out.dtype), M, out.shape[1], K,
+                                                  a.stride(0), out.stride(0), int(act), _p(ws), ws.numel() * 4,
+                                                  _p(counters), counters.numel(), int(max_splits), _p(err), _stream()),
+                  "gemm_tc_act")
 
 
 def gemm_tc_glu(a, w, out, limit: float, alpha: float, err=None, max_splits=16) -> None:
@@ -327,10 +378,14 @@ class AttentionPlan:
         if want_rows:
             self._decode_rows = rows
 
-    def chunk(self, n_kv_heads: int, head_dim: int):
-        key = (n_kv_heads, head_dim)
+    def chunk(self, n_kv_heads: int, head_dim: int, window=None, keep_first: int = 0):
+        """(chunk, most chunks of a row) of the decode form; a window bounds the 64-key tiles that a row walks."""
+        max_len = self.max_len
+        if window:
+            max_len = min(max_len, (-(-int(keep_first or 0) // 64) + -(-int(window) // 64) + 1) * 64)
+        key = (n_kv_heads, head_dim, max_len)
         if key not in self._chunking:
-            self._chunking[key] = decode_chunking(self.n_decode, n_kv_heads, self.max_len, head_dim)
+            self._chunking[key] = decode_chunking(self.n_decode, n_kv_heads, max_len, head_dim)
         return self._chunking[key]
 
 
@@ -454,28 +509,30 @@ def _decode_scratch(device, n_rows, n_heads, n_kv_heads, head_dim, n_splits):
 
 
 def attention_decode(q, q_stride, out, kpool, vpool, positions, seq_of_row, tables, rows, n_rows, n_heads,
-                     n_kv_heads, head_dim, scale, window, chunk, n_splits, err, softcap: float = 0.0,
-                     sink: bool = False, sink_values=None) -> None:
-    """The split-key decode form. `softcap` c > 0: a scaled score s becomes c tanh(s / c); `sink`: every row's
-    denominator holds one more exp(0) that has no value, or exp(sink_values[head]) (32-bit, one number per query
-    head) when those are given."""
+                     n_kv_heads, head_dim, scale, window, chunk, n_splits, err, **options) -> None:
+    """The split-key decode form; `options`: see `attention_options`."""
     lib = library.load()
     part, cnt = _decode_scratch(out.device, n_rows, n_heads, n_kv_heads, head_dim, n_splits)
-    library.check(lib.cuca_attention_decode_sv(
+    opt = attention_options(n_heads, scale, window, gate_width=n_heads * head_dim, **options)
+    library.check(lib.cuca_attention_decode_o(
         _p(q), int(q_stride), _p(out), out.stride(0), _p(kpool), _p(vpool), kpool.shape[0], kpool.shape[2],
         _p(positions), _p(seq_of_row), _p(tables), tables.shape[1], _p(rows), n_rows, n_heads, n_kv_heads, head_dim,
-        float(scale), int(window or 0), float(softcap or 0.0), int(bool(sink)), _sink_values(sink_values, n_heads), chunk,
-        n_splits, _p(part), _p(cnt), _p(err), _stream()), "attention_decode")
+        ctypes.addressof(opt), chunk, n_splits, _p(part), _p(cnt), _p(err), _stream()), "attention_decode")
+
+
+def _per_head(values, n_heads: int, what: str):
+    """The pointer of one number per query head (None: null), checked for what the kernels assume."""
+    if values is None:
+        return None
+    if values.dtype != torch.float32 or values.numel() != n_heads or not values.is_contiguous():
+        raise library.KernelError(f"{what} are {n_heads} contiguous 32-bit numbers, one per query head")
+    _cuda(values)
+    return values.data_ptr()
 
 
 def _sink_values(sink_values, n_heads: int):
-    """The pointer of a sink's per-head scores (None: the sink's score is 0), checked for what the kernels assume."""
-    if sink_values is None:
-        return None
-    if sink_values.dtype != torch.float32 or sink_values.numel() != n_heads or not sink_values.is_contiguous():
-        raise library.KernelError(f"a sink's scores are {n_heads} contiguous 32-bit numbers, one per query head")
-    _cuda(sink_values)
-    return sink_values.data_ptr()
+    """The pointer of a sink's per-head scores (None: the sink's score is 0)."""
+    return _per_head(sink_values, n_heads, "a sink's scores")
 
 
 def attention_decode_fused(partial, bias, cos, sin, rotary_dim, has_kv, out, kpool, vpool, positions, seq_of_row, tables,
@@ -502,14 +559,13 @@ def attention_decode_fused_supported(plan, cache, out_dtype, n_rows, n_heads, n_
 
 
 def attention_prefill(q, q_stride, out, kpool, vpool, positions, seq_of_row, tables, tile_row0, tile_nrows, n_tiles,
-                      n_heads, n_kv_heads, head_dim, scale, window, err, softcap: float = 0.0, sink: bool = False,
-                      sink_values=None) -> None:
+                      n_heads, n_kv_heads, head_dim, scale, window, err, **options) -> None:
     lib = library.load()
-    library.check(lib.cuca_attention_prefill_sv(
+    opt = attention_options(n_heads, scale, window, gate_width=n_heads * head_dim, **options)
+    library.check(lib.cuca_attention_prefill_o(
         _p(q), int(q_stride), _p(out), out.stride(0), _p(kpool), _p(vpool), kpool.shape[0], kpool.shape[2],
         _p(positions), _p(seq_of_row), _p(tables), tables.shape[1], _p(tile_row0), _p(tile_nrows), n_tiles, n_heads,
-        n_kv_heads, head_dim, float(scale), int(window or 0), float(softcap or 0.0), int(bool(sink)),
-        _sink_values(sink_values, n_heads), _p(err), _stream()), "attention_prefill")
+        n_kv_heads, head_dim, ctypes.addressof(opt), _p(err), _stream()), "attention_prefill")
 
 
 def attention_tc_supported(q, out, kpool, vpool, n_heads, n_kv_heads, head_dim) -> bool:
@@ -531,47 +587,48 @@ def attention_pair_tiles_mode(mode: int) -> None:
 
 
 def attention_prefill_tc(q, out, kpool, vpool, positions, seq_of_row, tables, tile_row0, tile_nrows, n_tiles,
-                         n_heads, n_kv_heads, head_dim, scale, window, err, softcap: float = 0.0,
-                         sink: bool = False, sink_values=None) -> None:
+                         n_heads, n_kv_heads, head_dim, scale, window, err, **options) -> None:
     """Prefill attention on tcgen05; tiles of up to 128 consecutive rows of one request."""
     lib = library.load()
-    library.check(lib.cuca_attention_prefill_tc_sv(
+    opt = attention_options(n_heads, scale, window, gate_width=n_heads * head_dim, **options)
+    library.check(lib.cuca_attention_prefill_tc_o(
         _p(q), q.stride(0), q.shape[0], _p(out), out.stride(0), _p(kpool), _p(vpool), kpool.shape[0], kpool.shape[2],
         _p(positions), _p(seq_of_row), _p(tables), tables.shape[1], _p(tile_row0), _p(tile_nrows), n_tiles, n_heads,
-        n_kv_heads, head_dim, float(scale), int(window or 0), float(softcap or 0.0), int(bool(sink)),
-        _sink_values(sink_values, n_heads), _p(err), _stream()), "attention_prefill_tc")
+        n_kv_heads, head_dim, ctypes.addressof(opt), _p(err), _stream()), "attention_prefill_tc")
 
 
-def attention(qkv, out, cache, step, plan, n_heads, n_kv_heads, head_dim, scale, window, err, softcap: float = 0.0,
-              sink: bool = False, sink_values=None) -> None:
+def _gate_aligned(gate) -> bool:
+    """Whether the tcgen05 attention takes this output gate (16 bytes a load)."""
+    return gate is None or (gate.data_ptr() % 16 == 0 and gate.stride(0) % 8 == 0)
+
+
+def attention(qkv, out, cache, step, plan, n_heads, n_kv_heads, head_dim, scale, window, err, **options) -> None:
     """Paged causal attention of every row of the step; q is the head of each `qkv` row. bfloat16 with head
     sizes 16..128 in steps of 16 runs on tensor cores: single-token requests through the split-key decode form,
     portions of prompts through the prefill form; everything else (the 32-bit path, other head sizes) through
-    the plain kernel. `softcap` c > 0: a scaled score s becomes c tanh(s / c); `sink`: one more exp(0) without a
-    value in every row's denominator, or exp(sink_values[head]) when those (32-bit, one per query head) are given."""
+    the plain kernel. `options` (cap, sink, kept first keys, distance bias, output gate): see `attention_options`."""
     bs = cache.block_size
     if (out.dtype == torch.bfloat16 and plan is not None and bs & (bs - 1) == 0
             and attention_mma_supported(n_heads, n_kv_heads, head_dim, qkv.stride(0), out.stride(0))):
         if plan.n_portions:
-            if USE_TC_ATTENTION and attention_tc_supported(qkv, out, cache.k, cache.v, n_heads, n_kv_heads, head_dim):
+            if (USE_TC_ATTENTION and attention_tc_supported(qkv, out, cache.k, cache.v, n_heads, n_kv_heads, head_dim)
+                    and _gate_aligned(options.get("gate"))):
                 row0, nrows, n = plan.tiles(tile_rows(1))
                 attention_prefill_tc(qkv, out, cache.k, cache.v, step.positions, step.seq_of_row, cache.tables,
-                                     row0, nrows, n, n_heads, n_kv_heads, head_dim, scale, window, err, softcap, sink,
-                                     sink_values)
+                                     row0, nrows, n, n_heads, n_kv_heads, head_dim, scale, window, err, **options)
             else:
                 row0, nrows, n = plan.tiles(tile_rows(0))
                 attention_prefill(qkv, qkv.stride(0), out, cache.k, cache.v, step.positions, step.seq_of_row,
                                   cache.tables, row0, nrows, n, n_heads, n_kv_heads, head_dim, scale, window, err,
-                                  softcap, sink, sink_values)
+                                  **options)
         if plan.n_decode:
-            chunk, n_splits = plan.chunk(n_kv_heads, head_dim)
+            chunk, n_splits = plan.chunk(n_kv_heads, head_dim, window, options.get("keep_first", 0))
             attention_decode(qkv, qkv.stride(0), out, cache.k, cache.v, step.positions, step.seq_of_row,
                              cache.tables, plan.decode_rows, plan.n_decode, n_heads, n_kv_heads, head_dim, scale,
-                             window, chunk, n_splits, err, softcap, sink, sink_values)
+                             window, chunk, n_splits, err, **options)
         return
     attention_generic_v(qkv, qkv.stride(0), out, cache.k, cache.v, step.positions, step.seq_of_row, cache.tables,
-                        n_heads, n_kv_heads, head_dim, head_dim, scale, window, err, softcap=softcap, sink=sink,
-                        sink_values=sink_values)
+                        n_heads, n_kv_heads, head_dim, head_dim, scale, window, err, **options)
 
 
 def scatter_int(dst, idx, val) -> None:
@@ -760,8 +817,18 @@ def post_norm_add(x, y, gain, eps, gain2=None, out=None) -> None:
 
 
 def gelu_(a, tanh_form: bool = False) -> None:
+    """a = gelu(a) in place: the exact form (erf), or its tanh form."""
+    _activation(a, 1 if tanh_form else 0)
+
+
+def relu2_(a) -> None:
+    """a = relu(a)^2 in place."""
+    _activation(a, 2)
+
+
+def _activation(a, form: int) -> None:
     _cuda(a)
-    library.check(library.load().cuca_gelu(_p(a), dtype_code(a.dtype), a.numel(), int(tanh_form), _stream()), "gelu")
+    library.check(library.load().cuca_activation(_p(a), dtype_code(a.dtype), a.numel(), form, _stream()), "activation")
 
 
 def scale_(a, s: float) -> None:
@@ -919,37 +986,38 @@ def rope_store_general(qkv, k_col, v_col, positions, seq_of_row, tables, cos, si
 
 
 def attention_generic_v(q, q_stride, out, kpool, vpool, positions, seq_of_row, tables, n_heads, n_kv_heads,
-                        head_dim, v_head_dim, scale, window, err, softcap: float = 0.0, sink: bool = False,
-                        sink_values=None) -> None:
-    """The plain attention kernel with value heads of their own size (`vpool`: [pages, kv heads, block, v_head_dim]).
-    `softcap` c > 0: a score s becomes c tanh(s / c); `sink`: the softmax's denominator holds one more exp(0), or
-    exp(sink_values[head]) when those are given."""
+                        head_dim, v_head_dim, scale, window, err, **options) -> None:
+    """The plain attention kernel with value heads of their own size (`vpool`: [pages, kv heads, block, v_head_dim]);
+    `options`: see `attention_options`."""
     _cuda(q, out, kpool, vpool)
-    library.check(library.load().cuca_attention_generic_sv(
+    opt = attention_options(n_heads, scale, window, gate_width=n_heads * v_head_dim, **options)
+    library.check(library.load().cuca_attention_generic_o(
         _p(q), int(q_stride), _p(out), out.stride(0), dtype_code(out.dtype), _p(kpool), _p(vpool), kpool.shape[0],
         kpool.shape[2], _p(positions), _p(seq_of_row), _p(tables), tables.shape[1], out.shape[0], n_heads,
-        n_kv_heads, head_dim, v_head_dim, float(scale), int(window or 0), float(softcap or 0.0), int(bool(sink)),
-        _sink_values(sink_values, n_heads), _p(err), _stream()), "attention_generic")
+        n_kv_heads, head_dim, v_head_dim, ctypes.addressof(opt), _p(err), _stream()), "attention_generic")
 
 
 def norm_rope_store(qkv, k_col, v_col, positions, seq_of_row, tables, cos, sin, rotary_dim, adjacent, q_norm, k_norm,
                     v_norm: bool, eps: float, kpool, vpool, block_size, n_heads, n_kv_heads, head_dim, v_head_dim, err,
-                    v_split: int = 1, q_out=None, v_row_dim: int = 0, whole: bool = False, q_temp=None) -> None:
+                    v_split: int = 1, q_out=None, v_row_dim: int = 0, whole: bool = False, q_temp=None,
+                    unit: bool = False, q_mul=None) -> None:
     """`rope_store_general` with norms per head in 32-bit before the rotation: q / rms(q) * q_norm, k likewise with
     k_norm (None: no norm), and with `v_norm` v / rms(v) before it is kept. q is rewritten in place, or goes to
     `q_out` [rows, heads * head_dim] of the pools' dtype (32-bit rows beside 16-bit pools). `v_row_dim` n > 0: a row's
     value heads hold n values (the norm is over those) and the pool's `v_head_dim` >= n; the rest is kept as zeros.
     `whole`: the norm of q (and of k) is over the whole projection, all heads at once, with weights [heads * head_dim].
-    `q_temp` (coef, every): the query at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1)."""
+    `q_temp` (coef, every): the query at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1).
+    `unit`: the norms per head have no weight. `q_mul` (32-bit, one per query head): a factor on the head's queries, after
+    the norm. `v_col` may be `k_col`: the values are then the keys as projected."""
     _cuda(qkv, positions, seq_of_row, kpool, vpool, q_norm, k_norm, q_out)
     coef, every = (float(q_temp[0]), int(q_temp[1])) if q_temp else (0.0, 0)
-    library.check(library.load().cuca_norm_rope_store_w(
+    library.check(library.load().cuca_norm_rope_store_u(
         _p(qkv), dtype_code(qkv.dtype), qkv.stride(0), int(k_col), int(v_col), _p(q_out), dtype_code(kpool.dtype),
         _p(positions), _p(seq_of_row), _p(tables), tables.shape[1], _p(cos), _p(sin),
         cos.shape[0] if cos is not None else 0, int(rotary_dim), int(bool(adjacent)), _p(q_norm), _p(k_norm),
         int(bool(v_norm)), float(eps), _p(kpool), _p(vpool), kpool.shape[0], int(block_size), qkv.shape[0], n_heads,
-        n_kv_heads, head_dim, v_head_dim, int(v_split), int(v_row_dim), int(bool(whole)), coef, every, _p(err),
-        _stream()), "norm_rope_store")
+        n_kv_heads, head_dim, v_head_dim, int(v_split), int(v_row_dim), int(bool(whole)), coef, every, int(bool(unit)),
+        _per_head(q_mul, n_heads, "factors on the queries"), _p(err), _stream()), "norm_rope_store")
 
 
 def sigmoid_gate_(a, gate) -> None:
@@ -1271,3 +1339,37 @@ def round_rows(x, out) -> None:
     _cuda(x, out)
     library.check(library.load().cuca_round_rows(_p(x), _p(out), dtype_code(out.dtype), x.numel(), _stream()),
                   "round_rows")
+
+
+# ------------------------------------------------------------------ blocks that norm the sum
+def sum_norm(x, terms, scale, weight, alpha: float, eps: float, out=None) -> None:
+    """x <- N(alpha x + scale * y) * weight in place with y the weighted sum of `terms` and N the RMS norm; `out` (or None)
+    = the new x in out's dtype. `scale`: a factor per channel, or None."""
+    _cuda(x, scale, weight, out)
+    t = _terms(terms)
+    library.check(library.load().cuca_sum_norm(_p(x), ctypes.addressof(t), _p(scale), _p(weight), float(alpha), float(eps),
+                                               _p(out), dtype_code(out.dtype) if out is not None else 0, x.shape[0],
+                                               x.shape[1], _stream()), "sum_norm")
+
+
+def sum_norm_shift_supported(width: int) -> bool:
+    return bool(library.load().cuca_sum_norm_shift_supported(int(width)))
+
+
+def sum_norm_shift(x, terms, scale, weight, alpha: float, eps: float, x_out, mix, kept, out, step) -> None:
+    """`sum_norm` out of place, and out[r] = x_out[r] + (x_out[r-1] - x_out[r]) * mix of the new rows; the row before a
+    request's first row of the step is `kept[slot]`, which then becomes the request's last row."""
+    _cuda(x, scale, weight, x_out, mix, kept, out)
+    t = _terms(terms)
+    library.check(library.load().cuca_sum_norm_shift(
+        _p(x), ctypes.addressof(t), _p(scale), _p(weight), float(alpha), float(eps), _p(x_out), _p(mix), _p(kept), _p(out),
+        dtype_code(out.dtype), _p(step.seq_of_row), _p(step.req_row0), _p(step.req_count), x.shape[0], step.n_seqs,
+        x.shape[1], _stream()), "sum_norm_shift")
+
+
+def shift_rows(x, mix, kept, out, step) -> None:
+    """out[r] = x[r] + (x[r-1] - x[r]) * mix; the kept rows as in `sum_norm_shift`."""
+    _cuda(x, mix, kept, out)
+    library.check(library.load().cuca_shift_rows(_p(x), _p(mix), _p(kept), _p(out), dtype_code(out.dtype),
+                                                 _p(step.seq_of_row), _p(step.req_row0), _p(step.req_count), _p(step.slots),
+                                                 x.shape[0], step.n_seqs, x.shape[1], _stream()), "shift_rows")

@@ -102,7 +102,7 @@ class Model:
     def forward(self, step, cache) -> torch.Tensor | None:
         """Run the step's rows through the model; logits [wanted rows, vocab] in 32-bit, or None."""
         x = torch.empty(step.n_rows, self.spec.width, dtype=torch.float32, device=self.rt.device)
-        self.embedding.forward(step.tokens, x)
+        self.embedding.forward(step.tokens, x, step.positions)
         if self.spec.streams is not None:  # every copy of the stream starts as the embedding output
             wide = torch.empty(step.n_rows, self.spec.streams * self.spec.width, dtype=torch.float32,
                                device=self.rt.device)
@@ -112,7 +112,7 @@ class Model:
         origin = None
         if self.stream_ops:  # they read the embedding output, which the layers overwrite in place
             origin = torch.empty_like(x)
-            self.embedding.forward(step.tokens, origin)
+            self.embedding.forward(step.tokens, origin, step.positions)
         n_run = 0
         for run in self.spec.schedule:
             if isinstance(run, Between):

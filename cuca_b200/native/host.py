@@ -73,7 +73,7 @@ _SIGNATURES = {
     "cuca_host_blockpool_new": (_P, [_I]), "cuca_host_blockpool_free": (None, [_P]),
     "cuca_host_blockpool_alloc": (_I, [_P]), "cuca_host_blockpool_release": (_I, [_P, _I]),
     "cuca_host_blockpool_free_count": (_I, [_P]), "cuca_host_blockpool_reset": (None, [_P]),
-    "cuca_host_pools_new": (_P, [_I, _IP, _IP, _I]), "cuca_host_pools_free": (None, [_P]),
+    "cuca_host_pools_new": (_P, [_I, _IP, _IP, _IP, _I]), "cuca_host_pools_free": (None, [_P]),
     "cuca_host_pools_new_seq": (_I, [_P]), "cuca_host_pools_drop_seq": (None, [_P, _I]),
     "cuca_host_pools_owed": (None, [_P, _I, _I, _IP]), "cuca_host_pools_can_give": (_I, [_P, _IP]),
     "cuca_host_pools_reserve": (_I, [_P, _I, _I]), "cuca_host_pools_release_window": (_I, [_P, _I]),

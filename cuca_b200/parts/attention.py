@@ -26,7 +26,14 @@ tensor-core kernels take the rest of the shape (bfloat16, key sizes in steps of 
 rows, the attention output and the output projection's input columns (zero columns, added at load) are that wide, and
 the layer runs slab by slab like one whose values are a multiple. The norm on values is over the stored ones.
 
-Three more options of the general path. `qk_norm` "whole": the RMS norm of q (and of k) is taken over the whole
+More options of the general path. `qk_norm` "unit": the RMS norm per head has no weight. `values` "keys": there is no value
+projection, the values are the keys as projected (with their bias), before norm and rotation. `q_scale`: a stored factor
+per query head (`q_scale` [heads]) multiplies the head's scores; it goes into the queries, with the scale. `slopes` (one
+number per query head): slope * distance between query and key is taken off a score (after scale and cap). `keep_first` k
+beside a `window`: the first k keys of a request stay visible at their true distances; the pages that hold them stay with
+the request.
+
+Three more. `qk_norm` "whole": the RMS norm of q (and of k) is taken over the whole
 projection, all heads at once, with a weight of that size (`q_norm` [heads * head_dim], `k_norm` [kv heads * head_dim]).
 `q_temp` {coef, every}: the query at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1) (after norm
 and rotation). `sink` "learned": the sink's score is a stored number per query head (`sink` [heads], neither scaled nor
@@ -48,9 +55,10 @@ from .base import POSITIONS, CacheNeeds, KvNeeds, Mixer, PartSpec, TensorNeed, r
 class PagedAttention(Mixer):
     """params: width, n_heads, n_kv_heads, head_dim, window (None: all keys), scale (None: 1/sqrt(head_dim)),
     position (PartSpec or None), shares_cache (bool), v_head_dim (None: head_dim), gate (bool, or "head"), qk_norm
-    (bool, or "whole"), v_norm (bool), eps (of those norms), softcap (None or 0: none), sink (bool, or "learned"),
-    q_temp ({coef, every} or None). tensors: q, k, v, o, g (with `gate`), q_norm and k_norm (with `qk_norm`), sink
-    (with a learned sink) and optional q_bias, k_bias, v_bias, o_bias."""
+    (bool, "whole" or "unit"), v_norm (bool), eps (of those norms), softcap (None or 0: none), sink (bool, or "learned"),
+    q_temp ({coef, every} or None), values (None, or "keys"), q_scale (bool), slopes (None or a list), keep_first (0).
+    tensors: q, k, v (without `values`), o, g (with `gate`), q_norm and k_norm (with a `qk_norm` that has weights), sink
+    (with a learned sink), q_scale (with `q_scale`) and optional q_bias, k_bias, v_bias, o_bias."""
 
     graph_safe = True
 
@@ -69,6 +77,12 @@ class PagedAttention(Mixer):
         self.gated = bool(p.get("gate", False)) and not self.head_gate
         self.qk_norm, self.v_norm = bool(p.get("qk_norm", False)), bool(p.get("v_norm", False))
         self.norm_whole = p.get("qk_norm") == "whole"  # over the whole projection instead of per head
+        self.norm_unit = p.get("qk_norm") == "unit"  # per head, without a weight
+        self.keys_as_values = p.get("values") == "keys"
+        self.q_scaled = bool(p.get("q_scale", False))
+        slopes = p.get("slopes")
+        self.slope_list = [float(s) for s in slopes] if slopes else None
+        self.keep_first = int(p.get("keep_first") or 0) if self.window is not None else 0
         self.eps = float(p.get("eps", 1e-6))
         self.softcap = float(p.get("softcap") or 0.0)
         self.sink = bool(p.get("sink", False))
@@ -79,6 +93,13 @@ class PagedAttention(Mixer):
             raise ValueError(f"attention: a query temperature every {self.q_temp[1]} positions is not positive")
         if self.norm_whole and self.v_norm:
             raise ValueError("attention: a norm over the whole projection is not combined with a norm on values")
+        if self.slope_list is not None and len(self.slope_list) != self.n_heads:
+            raise ValueError(f"attention: {len(self.slope_list)} distance slopes for {self.n_heads} query heads")
+        if self.keep_first < 0:
+            raise ValueError(f"attention: {self.keep_first} kept first keys")
+        if self.keys_as_values and (self.v_head_dim != self.head_dim or self.v_norm or self.norm_whole):
+            raise ValueError("attention: values that are the keys are as wide as keys, and neither normed nor combined with "
+                             "a norm over the whole projection")
         if self.softcap < 0:
             raise ValueError(f"attention: a score cap of {self.softcap} is not positive")
         if self.n_heads % self.n_kv_heads:
@@ -89,13 +110,16 @@ class PagedAttention(Mixer):
         pos = p.get("position")
         self.position = POSITIONS.get(pos.kind)(pos, runtime) if isinstance(pos, PartSpec) else None
         self.w_qkv = self.b_qkv = self.w_o = self.b_o = self.w_qn = self.w_kn = self.sink_values = None
+        self.slopes = self.q_mul = None
         # what the stacked-projection kernels of the usual path do not take
-        self.normed = self.qk_norm or self.v_norm or self.q_temp is not None
+        self.normed = self.qk_norm or self.v_norm or self.q_temp is not None or self.q_scaled
         self.general = (self.v_head_dim != self.head_dim or self.gated or self.head_gate or self.normed
-                        or self.softcap > 0 or self.sink or getattr(self.position, "pairs", "half") != "half")
+                        or self.softcap > 0 or self.sink or getattr(self.position, "pairs", "half") != "half"
+                        or self.keys_as_values or self.slope_list is not None or self.keep_first > 0)
         if self.general and self.shares_cache:
             raise ValueError("attention: a layer that reads another layer's pages takes neither a value size of its "
-                             "own, an output gate, head norms, a score cap, a sink nor adjacent rotation pairs")
+                             "own, an output gate, head norms, a score cap, a sink, a distance bias, kept first keys nor "
+                             "adjacent rotation pairs")
         # the width of a value row in the pool: padded to a multiple of the key size for the tensor-core kernels
         self.v_pool_dim = self.v_head_dim
         d, dv = self.head_dim, self.v_head_dim
@@ -109,7 +133,7 @@ class PagedAttention(Mixer):
     # ------------------------------------------------------------ description
     def cache_needs(self):
         return CacheNeeds(kv=KvNeeds(self.n_kv_heads, self.head_dim, self.window,
-                                     None if self.v_pool_dim == self.head_dim else self.v_pool_dim))
+                                     None if self.v_pool_dim == self.head_dim else self.v_pool_dim, self.keep_first))
 
     def tensors(self):
         t, d, dv = self.spec.tensors, self.head_dim, self.v_head_dim
@@ -119,7 +143,9 @@ class PagedAttention(Mixer):
             out[t["g"]] = TensorNeed((self.n_heads * dv, self.width))
         if self.head_gate:
             out[t["g"]] = TensorNeed((self.n_heads, self.width))
-        if self.qk_norm:
+        if self.q_scaled:
+            out[t["q_scale"]] = TensorNeed((self.n_heads,), keep_fp32=True, init="ones")
+        if self.qk_norm and not self.norm_unit:
             whole = self.norm_whole
             out[t["q_norm"]] = TensorNeed((self.n_heads * d if whole else d,), keep_fp32=True, init="ones")
             out[t["k_norm"]] = TensorNeed((self.n_kv_heads * d if whole else d,), keep_fp32=True, init="ones")
@@ -127,7 +153,8 @@ class PagedAttention(Mixer):
             out[t["sink"]] = TensorNeed((self.n_heads,), keep_fp32=True)
         if not self.shares_cache:
             out[t["k"]] = TensorNeed((self.n_kv_heads * d, self.width))
-            out[t["v"]] = TensorNeed((self.n_kv_heads * dv, self.width))
+            if not self.keys_as_values:
+                out[t["v"]] = TensorNeed((self.n_kv_heads * dv, self.width))
         for role, rows in (("q_bias", self.n_heads * d), ("k_bias", self.n_kv_heads * d),
                            ("v_bias", self.n_kv_heads * dv), ("o_bias", self.width)):
             if role in t and not (self.shares_cache and role in ("k_bias", "v_bias")):
@@ -136,7 +163,8 @@ class PagedAttention(Mixer):
 
     def load(self, get):
         t = self.spec.tensors
-        roles = ["q"] if self.shares_cache else ["q", "k", "v"] + (["g"] if self.gated or self.head_gate else [])
+        kv = ["k"] if self.keys_as_values else ["k", "v"]
+        roles = ["q"] if self.shares_cache else ["q"] + kv + (["g"] if self.gated or self.head_gate else [])
         stacked = [get(t[r]) for r in roles]
         biases = [get(t[r + "_bias"]) if r + "_bias" in t else None for r in roles]
         rows = sum(w.shape[0] for w in stacked)
@@ -145,7 +173,7 @@ class PagedAttention(Mixer):
             biases.append(None)
         self.w_qkv = torch.cat(stacked, dim=0).contiguous()
         if any(b is not None for b in biases):
-            if any(b is None for b in biases[:3]):
+            if any(b is None for r, b in zip(roles, biases) if r in ("q", "k", "v")):
                 raise ValueError("attention biases must be given for q, k and v together")
             biases = [b if b is not None else biases[0].new_zeros(w.shape[0]) for b, w in zip(biases, stacked)]
             self.b_qkv = torch.cat(biases).contiguous()
@@ -156,14 +184,18 @@ class PagedAttention(Mixer):
             wide[:, :, :self.v_head_dim] = w
             self.w_o = wide.view(self.width, self.n_heads * self.v_pool_dim).contiguous()
         self.b_o = get(t["o_bias"]) if "o_bias" in t else None
-        if self.qk_norm:
+        if self.slope_list is not None:
+            self.slopes = torch.tensor(self.slope_list, dtype=torch.float32, device=self.rt.device)
+        if self.q_scaled:  # the stored factors and the scale are one factor on the queries
+            self.q_mul = (get(t["q_scale"]).float() * self.scale).contiguous()
+        if self.qk_norm and not self.norm_unit:
             self.w_qn, self.w_kn = get(t["q_norm"]), get(t["k_norm"])
         if self.sink_learned:
             self.sink_values = get(t["sink"]).contiguous()
 
     def weight_bytes(self):
         return sum(w.numel() * w.element_size() for w in (self.w_qkv, self.w_o, self.b_qkv, self.b_o, self.w_qn, self.w_kn,
-                                                          self.sink_values) if w is not None)
+                                                          self.sink_values, self.q_mul) if w is not None)
 
     def prepare(self, context_length: int) -> None:
         if self.position is not None:
@@ -194,6 +226,9 @@ class PagedAttention(Mixer):
         dv_row = self.v_head_dim if dv != self.v_head_dim else 0  # the projection's value heads, where narrower
         rows = h.shape[0]
         proj = self.rt.linear(h, self.w_qkv, bias=self.b_qkv)
+        v_col = nh * d if self.keys_as_values else (nh + nkv) * d
+        g_col = v_col + nkv * self.v_head_dim
+        scale = 1.0 if self.q_scaled else self.scale
         cos, sin, rot, adjacent = self.position.tables() if self.position is not None else (None, None, 0, False)
         split = self.value_split(cache)
         plan = self.plan(step) if split else None
@@ -203,32 +238,31 @@ class PagedAttention(Mixer):
         tensor_cores = split >= 1 and plan is not None
         split = max(split, 1)
         if self.normed:
-            ops.norm_rope_store(proj, nh * d, (nh + nkv) * d, step.positions, step.seq_of_row, cache.tables, cos, sin,
+            ops.norm_rope_store(proj, nh * d, v_col, step.positions, step.seq_of_row, cache.tables, cos, sin,
                                 rot, adjacent, self.w_qn, self.w_kn, self.v_norm, self.eps, cache.k, cache.v,
                                 cache.block_size, nh, nkv, d, dv, self.rt.err, v_split=split, v_row_dim=dv_row,
-                                whole=self.norm_whole, q_temp=self.q_temp)
+                                whole=self.norm_whole, q_temp=self.q_temp, unit=self.norm_unit, q_mul=self.q_mul)
         else:
-            ops.rope_store_general(proj, nh * d, (nh + nkv) * d, step.positions, step.seq_of_row, cache.tables, cos, sin,
+            ops.rope_store_general(proj, nh * d, v_col, step.positions, step.seq_of_row, cache.tables, cos, sin,
                                    rot, adjacent, cache.k, cache.v, cache.block_size, nh, nkv, d, dv, self.rt.err,
                                    v_split=split, v_row_dim=dv_row)
-        g_col = (nh + nkv) * d + nkv * self.v_head_dim
-        gate = proj[:, g_col:] if self.gated else None  # (a layer with a gate per value is never padded)
+        gate = proj[:, g_col:g_col + nh * dv] if self.gated else None  # (a layer with a gate per value is never padded)
+        options = {"softcap": self.softcap, "sink": self.sink, "sink_values": self.sink_values, "keep_first": self.keep_first,
+                   "slopes": self.slopes}
         attn = self.rt.empty(rows, nh * dv)
         if tensor_cores:
             slabs = cache.v.view(split, *cache.k.shape)
-            parts = self.rt.empty(split, rows, nh * d) if (split > 1 or gate is not None) else attn.view(1, rows, nh * d)
+            parts = self.rt.empty(split, rows, nh * d) if split > 1 else attn.view(1, rows, nh * d)
+            if split == 1:  # the gate is the attention kernels' own last step
+                options["gate"] = gate
             for j in range(split):
-                ops.attention(proj, parts[j], dataclasses.replace(cache, v=slabs[j]), step, plan, nh, nkv, d, self.scale,
-                              self.window, self.rt.err, softcap=self.softcap, sink=self.sink,
-                              sink_values=self.sink_values)
+                ops.attention(proj, parts[j], dataclasses.replace(cache, v=slabs[j]), step, plan, nh, nkv, d, scale,
+                              self.window, self.rt.err, **options)
             if parts.data_ptr() != attn.data_ptr():
                 ops.gate_merge(parts, gate, attn, nh, dv)
         else:
             ops.attention_generic_v(proj, proj.stride(0), attn, cache.k, cache.v, step.positions, step.seq_of_row,
-                                    cache.tables, nh, nkv, d, dv, self.scale, self.window, self.rt.err,
-                                    softcap=self.softcap, sink=self.sink, sink_values=self.sink_values)
-            if gate is not None:
-                ops.sigmoid_gate_(attn, gate)
+                                    cache.tables, nh, nkv, d, dv, scale, self.window, self.rt.err, gate=gate, **options)
         if self.head_gate:
             ops.head_gate_(attn, proj[:, g_col:g_col + nh], nh, dv)
         stream.add_linear(attn, self.w_o, bias=self.b_o)
@@ -250,7 +284,7 @@ class PagedAttention(Mixer):
             if ops.attention_decode_fused_supported(plan, cache, h.dtype, h.shape[0], nh, self.n_kv_heads, d):
                 # single tokens only: adding the slices, rotation, the page write and attention are one launch
                 attn = self.rt.empty(h.shape[0], nh * d)
-                chunk, n_splits = plan.chunk(self.n_kv_heads, d)
+                chunk, n_splits = plan.chunk(self.n_kv_heads, d, self.window)
                 ops.attention_decode_fused(parts, self.b_qkv, cos, sin, rot, nkv > 0, attn, cache.k, cache.v,
                                            step.positions, step.seq_of_row, cache.tables, None,
                                            plan.n_decode, nh, self.n_kv_heads, d, self.scale, self.window, chunk,

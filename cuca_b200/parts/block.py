@@ -4,7 +4,9 @@
 token's: x += n1b(mixer(shift(n1(x)))); x += n2b(ffn(n2(x))).
 `hyper_connections`: several copies of the stream; a sublayer reads a weighted sum of them and writes into all.
 `parallel_residual`: one norm, both sublayers read its output: x += mixer(h) + ffn(h) with h = norm(x).
-`post_norm`: the sublayers read the stream as it is, their outputs are normed: x += norm(mixer(x)); x += norm(ffn(x))."""
+`post_norm`: the sublayers read the stream as it is, their outputs are normed: x += norm(mixer(x)); x += norm(ffn(x)).
+`sum_norm_shift`: the sublayers read the stream as it is (the mixer mixed with the previous token's), the sum is normed:
+x = norm(a x + s1 * mixer(shift(x))); x = norm(a x + s2 * ffn(x))."""
 from __future__ import annotations
 
 from ..kernels import ops
@@ -55,6 +57,70 @@ class PostNormBlock(Block):
             stream.add_normed(y, self.ffn_norm)
 
 
+@register_block("sum_norm_shift")
+class SumNormShiftBlock(Block):
+    """x <- mixer_norm(alpha x + s1 * mixer(shift(x))), then x <- ffn_norm(alpha x + s2 * ffn(x)), with a factor per channel
+    on each sublayer's output and shift(x)_t = x_t + (x_(t-1) - x_t) * mix (x_(-1) = 0). The previous token's x is kept per
+    request in the layer run's state `shift`, 32-bit, beside whatever the mixer keeps.
+
+    params: width, alpha. tensors: mix [width], mixer_scale [width] and, with a feed-forward, ffn_scale [width].
+
+    A sublayer's output is gathered as terms (`SublayerOutput`). The layer's last sum is left to the next reader of the
+    stream (`ResidualStream.defer_sum_norm`): the next layer's shift takes it in the same pass, so that a layer costs two
+    passes over the stream."""
+
+    def __init__(self, spec, runtime, mixer, feed_forward, mixer_norm, ffn_norm):
+        super().__init__(spec, runtime, mixer, feed_forward, mixer_norm, ffn_norm)
+        self.width = int(spec.params["width"])
+        self.alpha = float(spec.params["alpha"])
+        for norm in (mixer_norm, ffn_norm):
+            if norm is not None and not hasattr(norm, "sum_norm"):
+                raise ValueError(f"sum_norm_shift: the norm `{norm.spec.kind}` is not applied to a sum")
+        self.mix = self.scale1 = self.scale2 = None
+
+    def tensors(self):
+        t = self.spec.tensors
+        out = {t["mix"]: TensorNeed((self.width,), keep_fp32=True),
+               t["mixer_scale"]: TensorNeed((self.width,), keep_fp32=True, init="ones")}
+        if self.feed_forward is not None:
+            out[t["ffn_scale"]] = TensorNeed((self.width,), keep_fp32=True, init="ones")
+        return out
+
+    def load(self, get):
+        t = self.spec.tensors
+        self.mix, self.scale1 = get(t["mix"]), get(t["mixer_scale"])
+        if self.feed_forward is not None:
+            self.scale2 = get(t["ffn_scale"])
+
+    def weight_bytes(self):
+        return sum(w.numel() * w.element_size() for w in (self.mix, self.scale1, self.scale2) if w is not None)
+
+    def cache_needs(self):
+        return _with_shift_state(self.mixer.cache_needs(), self.width)
+
+    def forward(self, stream, step, cache) -> None:
+        rt = self.rt
+        stream = rt.stream(stream)
+        h = stream.shifted(self.mix, cache.state["shift"], step)
+        y = SublayerOutput(rt, step.n_rows, self.width)
+        self.mixer.forward(h, y, step, cache)
+        if self.feed_forward is None:
+            stream.defer_sum_norm(y, self.mixer_norm, self.alpha, self.scale1)
+            return
+        stream.sum_normed(y, self.mixer_norm, self.alpha, self.scale1)
+        y = SublayerOutput(rt, step.n_rows, self.width)
+        self.feed_forward.forward(stream.rounded(), y, step)
+        stream.defer_sum_norm(y, self.ffn_norm, self.alpha, self.scale2)
+
+
+def _with_shift_state(needs: CacheNeeds, width: int) -> CacheNeeds:
+    """A mixer's needs and the previous token's row beside them, state `shift`."""
+    state = needs.state if isinstance(needs.state, dict) else ({} if needs.state is None else {"mixer": needs.state})
+    if "shift" in state:
+        raise ValueError("the mixer names a state `shift`, which is this block's")
+    return CacheNeeds(kv=needs.kv, state={"shift": StateNeeds((width,)), **state})
+
+
 @register_block("sandwich_shift")
 class SandwichShiftBlock(Block):
     """x += post1(mixer(shift(pre1(x)))); x += post2(ffn(pre2(x))), with shift(h)_t = h_t + (h_(t-1) - h_t) * mix
@@ -95,11 +161,7 @@ class SandwichShiftBlock(Block):
         return sum(w.numel() * w.element_size() for w in (self.mix, self.post1, self.post2) if w is not None)
 
     def cache_needs(self):
-        needs = self.mixer.cache_needs()
-        state = needs.state if isinstance(needs.state, dict) else ({} if needs.state is None else {"mixer": needs.state})
-        if "shift" in state:
-            raise ValueError("the mixer names a state `shift`, which is this block's")
-        return CacheNeeds(kv=needs.kv, state={"shift": StateNeeds((self.width,)), **state})
+        return _with_shift_state(self.mixer.cache_needs(), self.width)
 
     def forward(self, stream, step, cache) -> None:
         rt = self.rt

@@ -14,8 +14,9 @@ from .base import Part, TensorNeed
 
 class TokenEmbedding(Part):
     """params: vocab, width, scale (a factor on every embedding row, default 1), norm_eps (None: none; a number: the
-    row is RMS-normed, e / sqrt(mean(e^2) + norm_eps) times the tensor `norm`, before it becomes the stream).
-    tensors: weight [vocab, width], norm [width] (with norm_eps)."""
+    row is RMS-normed, e / sqrt(mean(e^2) + norm_eps) times the tensor `norm`, before it becomes the stream), positions
+    (None: none; n: a learned vector per position is added to the scaled row, row p of the tensor `positions`; not combined
+    with the norm). tensors: weight [vocab, width], norm [width] (with norm_eps), positions [positions, width]."""
 
     def __init__(self, spec, runtime):
         super().__init__(spec, runtime)
@@ -24,20 +25,31 @@ class TokenEmbedding(Part):
         self.scale = float(spec.params.get("scale", 1.0))
         eps = spec.params.get("norm_eps")
         self.norm_eps = float(eps) if eps is not None else None
-        self.weight = self.norm_weight = None
+        self.positions = int(spec.params.get("positions") or 0)
+        if self.positions and self.norm_eps is not None:
+            raise ValueError("embedding: learned positions are not combined with a norm on the embedding row")
+        self.weight = self.norm_weight = self.pos_weight = None
 
     def tensors(self):
         out = {self.spec.tensors["weight"]: TensorNeed((self.vocab, self.width))}
         if self.norm_eps is not None:
             out[self.spec.tensors["norm"]] = TensorNeed((self.width,), keep_fp32=True, init="ones")
+        if self.positions:
+            out[self.spec.tensors["positions"]] = TensorNeed((self.positions, self.width))
         return out
 
     def load(self, get):
         self.weight = get(self.spec.tensors["weight"])
         if self.norm_eps is not None:
             self.norm_weight = get(self.spec.tensors["norm"])
+        if self.positions:
+            self.pos_weight = get(self.spec.tensors["positions"])
 
-    def forward(self, tokens, out) -> None:
+    def forward(self, tokens, out, positions=None) -> None:
+        """`positions`: the rows' positions, wanted when the embedding has learned ones."""
+        if self.positions:
+            ops.embed_pos(self.weight, self.pos_weight, tokens, positions, out, self.rt.err, self.scale)
+            return
         if self.norm_eps is not None:
             ops.embed_norm(self.weight, tokens, out, self.norm_weight, self.norm_eps, self.rt.err, self.scale)
         else:

@@ -128,8 +128,8 @@ class GatedUnit(FeedForward):
 
 @register_feed_forward("dense_act")
 class DenseActivation(FeedForward):
-    """y = down(act(up f + b_up)) + b_down with act the exact (erf) GELU or its tanh form.
-    params: width, inner, act ("gelu" | "gelu_tanh"), bias (bool). tensors: up [inner, width], down [width, inner]
+    """y = down(act(up f + b_up)) + b_down with act the exact (erf) GELU, its tanh form or the square of relu.
+    params: width, inner, act ("gelu" | "gelu_tanh" | "relu2"), bias (bool). tensors: up [inner, width], down [width, inner]
     and, with bias, up_bias [inner], down_bias [width]."""
 
     graph_safe = True
@@ -139,8 +139,8 @@ class DenseActivation(FeedForward):
         self.width = int(spec.params["width"])
         self.inner = int(spec.params["inner"])
         self.act = str(spec.params.get("act", "gelu"))
-        if self.act not in ("gelu", "gelu_tanh"):
-            raise ValueError(f"dense feed-forward: activation `{self.act}` is unknown; known: gelu, gelu_tanh")
+        if self.act not in ("gelu", "gelu_tanh", "relu2"):
+            raise ValueError(f"dense feed-forward: activation `{self.act}` is unknown; known: gelu, gelu_tanh, relu2")
         self.bias = bool(spec.params.get("bias", True))
         self.w_up = self.w_down = self.b_up = self.b_down = None
 
@@ -163,8 +163,16 @@ class DenseActivation(FeedForward):
                    if w is not None)
 
     def forward(self, h, stream, step) -> None:
-        a = self.rt.linear(h, self.w_up, bias=self.b_up)
-        ops.gelu_(a, tanh_form=self.act == "gelu_tanh")
+        if self.act == "relu2" and h.dtype == torch.bfloat16 and ops.gemm_tc_supported(h, self.w_up):
+            # the activation is the contraction's epilogue, from the 32-bit sums
+            a = self.rt.empty(h.shape[0], self.inner)
+            ops.gemm_tc_act(h, self.w_up, a, ops.ACT_RELU2, self.b_up, self.rt.err)
+        else:
+            a = self.rt.linear(h, self.w_up, bias=self.b_up)
+            if self.act == "relu2":
+                ops.relu2_(a)
+            else:
+                ops.gelu_(a, tanh_form=self.act == "gelu_tanh")
         self.rt.stream(stream).add_linear(a, self.w_down, bias=self.b_down)
 
 

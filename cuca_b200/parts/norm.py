@@ -49,6 +49,17 @@ class RMSNorm(Norm):
             raise ValueError("rmsnorm: a norm in parts is not applied to a sublayer's output")
         ops.norm_add(x, terms, self.weight, self.eps, out, center=False)
 
+    def sum_norm(self, x, terms, alpha: float, scale, out, x_out=None, shift=None) -> None:
+        """x <- this norm of alpha x + scale * (the terms' weighted sum), in place or, with `x_out`, there; `out` (or None):
+        the new x in the compute dtype, with `shift` (mix, kept, step) every row mixed with the one before it."""
+        if self.groups != 1:
+            raise ValueError("rmsnorm: a norm in parts is not applied to the sum of stream and output")
+        if shift is None:
+            ops.sum_norm(x, terms, scale, self.weight, alpha, self.eps, out)
+        else:
+            mix, kept, step = shift
+            ops.sum_norm_shift(x, terms, scale, self.weight, alpha, self.eps, x_out, mix, kept, out, step)
+
 
 @register_norm("layernorm")
 class LayerNorm(Norm):

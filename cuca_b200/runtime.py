@@ -82,6 +82,7 @@ class ResidualStream:
         self._pending = None
         self._unwritten = False
         self._rounded = None  # the stream in the compute dtype, while nothing has touched the stream since it was made
+        self._unsummed = None  # (output, norm, alpha, scale) of `defer_sum_norm`: the stream is what that makes of it
 
     @classmethod
     def unwritten(cls, runtime: "Runtime", rows: int, width: int) -> "ResidualStream":
@@ -95,7 +96,7 @@ class ResidualStream:
         """The stream is `tensor` from now on (an operation that rewrote the whole stream out of place)."""
         if tensor.dtype != torch.float32 or tensor.shape != self._tensor.shape:
             raise ValueError("a residual stream is replaced by a 32-bit tensor of its own shape")
-        self._pending = self._rounded = None
+        self._pending = self._rounded = self._unsummed = None
         self._tensor = tensor
 
     @property
@@ -105,6 +106,8 @@ class ResidualStream:
     @property
     def data(self) -> torch.Tensor:
         """The stream's tensor with everything added; it may be read and updated in place."""
+        if self._unsummed is not None:
+            self._sum_norm(*self._take_unsummed())
         self._rounded = None
         if self._unwritten:
             self._tensor.zero_()
@@ -117,6 +120,8 @@ class ResidualStream:
     def take(self):
         """(tensor, pending slices or None) for a reader that adds the slices itself, in the stream too: after
         the reader's kernel the tensor must hold the sum."""
+        if self._unsummed is not None:
+            return self.data, None
         self._rounded = None
         if self._unwritten:
             self._tensor.zero_()
@@ -153,7 +158,7 @@ class ResidualStream:
 
     def drop_pending(self) -> None:
         """Forget unadded slices: the stream will not be read again (no logits are wanted)."""
-        self._pending = None
+        self._pending = self._unsummed = None
 
     # ------------------------------------------------ arrangements whose sublayers read the stream as it is
     def rounded(self) -> torch.Tensor:
@@ -175,6 +180,43 @@ class ResidualStream:
         out = None if x.dtype == self.rt.dtype else self.rt.empty(*x.shape)
         norm.add_normed(x, output.terms, out)
         self._rounded = out
+
+    # ------------------------------------------------ arrangements that norm the sum of stream and output
+    def sum_normed(self, output: "SublayerOutput", norm, alpha: float, scale) -> None:
+        """stream <- norm(alpha stream + scale * output), `norm` a part with `sum_norm`, `scale` a factor per channel (or
+        None); the rounded copy for the next sublayer's reader comes from the same pass."""
+        self.data
+        self._sum_norm(output, norm, alpha, scale)
+
+    def defer_sum_norm(self, output: "SublayerOutput", norm, alpha: float, scale) -> None:
+        """`sum_normed`, left to whoever reads the stream next: a reader that mixes rows (`shifted`) does it in its own
+        pass."""
+        self.data
+        self._rounded = None
+        self._unsummed = (output, norm, alpha, scale)
+
+    def _take_unsummed(self):
+        d, self._unsummed = self._unsummed, None
+        return d
+
+    def _sum_norm(self, output, norm, alpha, scale) -> None:
+        x = self._tensor
+        out = None if x.dtype == self.rt.dtype else self.rt.empty(*x.shape)
+        norm.sum_norm(x, output.terms, alpha, scale, out)
+        self._rounded = out
+
+    def shifted(self, mix, kept, step) -> torch.Tensor:
+        """Every row mixed with its request's row before it, x[r] + (x[r-1] - x[r]) * mix, in the compute dtype, to be read
+        only. `kept[slot]` stands for the row before a request's first row of the step, and becomes its last row."""
+        h = self.rt.empty(*self.shape)
+        if self._unsummed is not None and ops.sum_norm_shift_supported(self.shape[-1]):
+            output, norm, alpha, scale = self._take_unsummed()
+            x_out = torch.empty_like(self._tensor)
+            norm.sum_norm(self._tensor, output.terms, alpha, scale, h, x_out=x_out, shift=(mix, kept, step))
+            self._tensor, self._rounded = x_out, None
+        else:
+            ops.shift_rows(self.data, mix, kept, h, step)
+        return h
 
 
 class SublayerOutput(ResidualStream):
