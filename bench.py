@@ -291,6 +291,18 @@ def _nudorax_config(width, ff, heads, layers, vocab, window):
             "embedding": {"scale": width ** 0.5}, "layers": [layer] * layers}
 
 
+def _pafutar_config(width, ff, heads, layers, vocab, window):
+    """`layers` layers alike: softmax attention whose values are its keys (as many heads of 128 as the width holds, a quarter
+    as many key heads, a window and four kept first keys, a distance bias, a gate per value) and a dense squared-relu unit;
+    the sum of stream and output is normed."""
+    H = max(1, width // 128)
+    layer = {"type": "attention", "mlp": {"kind": "dense", "ff": ff},
+             "mixer": {"heads": H, "kv_heads": max(1, H // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                       "mask": {"size": window, "keep_first": 4}}}
+    return {"architecture": "Pafutar", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "postln_alpha": 2.0,
+            "embedding": {"scale": width ** 0.5}, "max_positions": 16384, "layers": [layer] * layers}
+
+
 def _llama_config(width, ff, heads, layers, vocab):
     return {"architectures": ["LlamaForCausalLM"], "model_type": "llama", "num_hidden_layers": layers,
             "hidden_size": width, "num_attention_heads": heads, "num_key_value_heads": max(1, heads // 4),
@@ -305,8 +317,8 @@ DESIGN_SIZES = {  # name -> (width, feed-forward, heads, layers, vocabulary)
 
 def design_table(args) -> int:
     """Prefill of one prompt and decode steps of `--batch` requests for the chosen design and for a Llama of the
-    same width, feed-forward size and number of layer runs (for Sutosun also a Pudinex and for Nudorax also a Sutosun,
-    the closest of the other designs), one JSON line per size and model: tokens/s of both phases, the decode step's bytes (weights once,
+    same width, feed-forward size and number of layer runs (for Sutosun also a Pudinex, for Nudorax also a Sutosun and
+    for Pafutar also a Nudorax, the closest of the other designs), one JSON line per size and model: tokens/s of both phases, the decode step's bytes (weights once,
     what a request keeps) over the measured copy bandwidth."""
     import numpy as np
     import torch
@@ -321,14 +333,16 @@ def design_table(args) -> int:
     ctx = max(T, P + steps + warmup + 64) + 64
     for size in (args.sizes.split(",") if args.sizes else list(DESIGN_SIZES)):
         width, ff, heads, layers, vocab = DESIGN_SIZES[size]
-        runs = layers if args.design in ("pudinex", "sutosun", "nudorax") else layers + layers // 2  # (a looped half runs twice)
+        runs = layers if args.design in ("pudinex", "sutosun", "nudorax", "pafutar") else layers + layers // 2  # (a looped half runs twice)
         make = {"bananex": _bananex_config, "dupenex": _dupenex_config, "pudinex": _pudinex_config,
-                "sutosun": _sutosun_config, "nudorax": _nudorax_config}[args.design]
+                "sutosun": _sutosun_config, "nudorax": _nudorax_config, "pafutar": _pafutar_config}[args.design]
         pair = [(args.design, make(width, ff, heads, layers, vocab, window=1024))]
         if args.design == "sutosun":
             pair.append(("pudinex", _pudinex_config(width, ff, heads, layers, vocab, window=1024)))
         if args.design == "nudorax":
             pair.append(("sutosun", _sutosun_config(width, ff, heads, layers, vocab, window=1024)))
+        if args.design == "pafutar":
+            pair.append(("nudorax", _nudorax_config(width, ff, heads, layers, vocab, window=1024)))
         pair.append(("llama", _llama_config(width, ff, heads, runs, vocab)))
         for name, cfg in pair:
             if args.only_model and name != args.only_model:
@@ -375,7 +389,7 @@ def design_table(args) -> int:
             # a windowed cache is read up to its window; state is read and written once per step
             per_request = 0
             for gi, grp in enumerate(core.groups):
-                seen = mean_ctx if grp.window is None else min(mean_ctx, grp.window)
+                seen = mean_ctx if grp.window is None else min(mean_ctx, grp.window + grp.keep_first)
                 vd = grp.head_dim if grp.v_head_dim is None else grp.v_head_dim
                 per_request += seen * len(grp.cache_ids) * grp.n_kv_heads * (grp.head_dim + vd) * 2
             per_request += 2 * core.cache.state_bytes_per_request()
@@ -417,7 +431,7 @@ def main() -> int:
     ap.add_argument("--decode-only", action="store_true",
                     help="with --shape llama-3.2-1b: the plain decode line at --batch instead of the mixed workload")
     ap.add_argument("--only-model", default=None, help="with --design: run only this model of the pair (the design's name or llama)")
-    ap.add_argument("--design", default=None, choices=["bananex", "dupenex", "nudorax", "pudinex", "sutosun"],
+    ap.add_argument("--design", default=None, choices=["bananex", "dupenex", "nudorax", "pafutar", "pudinex", "sutosun"],
                     help="instead of the bench: prefill and decode of this design beside a Llama of equal width, "
                          "feed-forward size and layer runs, at --sizes (1b,3b,8b layer sizes; a few layers each)")
     ap.add_argument("--sizes", default=None, help="with --design: which of 1b,3b,8b (all else)")

@@ -71,6 +71,12 @@ struct AttnParams {
   const float* sin_t;
   int table_rows, rot;
   int has_kv;            // 0: the layer reads another layer's pages and has only q
+  int width;             // columns of a slice's row: q heads at 0, k heads at nh D, v heads at v_col
+  int v_col;             // (nh D: the values are the keys as projected)
+  int unit;              // 1: instead of the rotation, q and k are divided by their root mean square per head, and ...
+  float norm_eps;
+  const float* q_mul;    // ... q is multiplied by its head's factor (or null)
+  int gate_col;          // >= 0: the pre-activations of an output gate stand there, one per output value
 };
 
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool valid) {
@@ -126,9 +132,10 @@ struct Smem {
   static constexpr int RS = D + 8;  // row stride in elements: 16 bytes of padding
   static constexpr int TILE_ELEMS = TILE * RS;
   static constexpr int BYTES = STAGES * 2 /*k, v*/ * TILE_ELEMS * 2;
-  // fused form: the 16 query rows, then the new key and the new value of the row
+  // fused form: the 16 query rows, then the new key and the new value of the row, then the gate's values
   static constexpr int Q_ELEMS = 16 * RS;
-  static constexpr int FUSED_BYTES = BYTES + (Q_ELEMS + 2 * D) * 2;
+  static constexpr int GATE_BYTES = 16 * D * 4;  // the output gate of the group's heads
+  static constexpr int FUSED_BYTES = BYTES + (Q_ELEMS + 2 * D) * 2 + GATE_BYTES;
   // decode with TMA: every warp has a ring of its own; a stage holds the warp's 16 keys and values as
   // 64-wide halves of 16 rows x 128 bytes, 128-byte swizzled: K half 0, K half 1, ..., V half 0, ...
   static constexpr int HALVES = D / 64;
@@ -136,7 +143,7 @@ struct Smem {
   static constexpr int WSTAGE_BYTES = 2 * (HALVES > 0 ? HALVES : 1) * SUB_BYTES;
   static constexpr int WSTAGES = 3;
   static constexpr int RING_BYTES = 4 * WSTAGES * WSTAGE_BYTES;
-  static constexpr int TMA_BYTES = RING_BYTES + 1024 /*alignment*/ + (Q_ELEMS + 2 * D) * 2;
+  static constexpr int TMA_BYTES = RING_BYTES + 1024 /*alignment*/ + (Q_ELEMS + 2 * D) * 2 + GATE_BYTES;
 };
 
 // One warp's state over its 16 MMA rows: thread (g, t) holds rows g and g + 8.
@@ -361,29 +368,37 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
   // are used further down. (One value at a time, as the general form below does it, the prologue took 6 us of the
   // kernel's 20 at batch 8.)
   const int f_half = FUSED ? p.rot / 2 : 0;
-  const size_t f_width = FUSED ? (size_t)(p.nh + (p.has_kv ? 2 * p.nkv : 0)) * D : 0;
+  const size_t f_width = FUSED ? (size_t)p.width : 0;
   const float* f_row = FUSED ? p.partial + (size_t)dec_row * f_width : nullptr;
   const bool f_in_table = FUSED && P >= 0 && P < p.table_rows;
-  const bool f_vec = FUSED && p.rot == D && D % 8 == 0 && ((p.slice_stride | f_width) & 3) == 0 &&
+  const bool f_unit = FUSED && p.unit;
+  const bool f_vec = FUSED && !f_unit && p.rot == D && D % 8 == 0 && ((p.slice_stride | f_width) & 3) == 0 &&
                      (((uintptr_t)p.partial | (uintptr_t)p.cos_t | (uintptr_t)p.sin_t) & 15) == 0;
   const int f_hq = f_half / 4;                                   // items per rotated head
-  const int f_rope_items = (G + (owner ? 1 : 0)) * f_hq;
-  const int f_items = f_rope_items + (owner ? D / 4 : 0);       // then the row's own value
+  const int f_rope_items = f_unit ? 0 : (G + (owner ? 1 : 0)) * f_hq;
+  // (with unit norms an item is four columns of a head: the q heads, the row's own key and, if it has columns of its own,
+  // the row's own value)
+  const int f_items = f_unit ? (G + (owner ? (p.v_col == p.nh * D ? 1 : 2) : 0)) * (D / 4)
+                             : f_rope_items + (owner ? D / 4 : 0);  // then the row's own value
   // columns of item `it`: ca (and ca + half for a rotated head); head index hh (G: the key), offset inside the head
   auto f_item = [&](int it, int& ca, int& hh, int& off) {
-    if (it < f_rope_items) {
+    if (f_unit) {
+      hh = it / (D / 4);
+      off = (it - hh * (D / 4)) * 4;
+      ca = (hh < G ? (kvh * G + hh) * D : hh == G ? (p.nh + kvh) * D : p.v_col + kvh * D) + off;
+    } else if (it < f_rope_items) {
       hh = it / f_hq;
       off = (it - hh * f_hq) * 4;
       ca = (hh < G ? (kvh * G + hh) * D : (p.nh + kvh) * D) + off;
     } else {
       hh = -1;
       off = (it - f_rope_items) * 4;
-      ca = (p.nh + p.nkv + kvh) * D + off;
+      ca = p.v_col + kvh * D + off;
     }
   };
   float4 pre_a[4], pre_b[4], pre_c = make_float4(1.f, 1.f, 1.f, 1.f), pre_s = make_float4(0.f, 0.f, 0.f, 0.f);
   auto preload = [&]() {
-  if (FUSED && f_vec && (int)threadIdx.x < f_items) {
+  if (FUSED && (f_vec || f_unit) && (int)threadIdx.x < f_items) {
     int ca, hh, off;
     f_item(threadIdx.x, ca, hh, off);
 #pragma unroll
@@ -391,10 +406,10 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
       pre_a[u] = pre_b[u] = make_float4(0.f, 0.f, 0.f, 0.f);
       if (u < p.n_slices) {
         pre_a[u] = __ldcg(reinterpret_cast<const float4*>(f_row + (size_t)u * p.slice_stride + ca));
-        if (hh >= 0) pre_b[u] = __ldcg(reinterpret_cast<const float4*>(f_row + (size_t)u * p.slice_stride + ca + f_half));
+        if (hh >= 0 && !f_unit) pre_b[u] = __ldcg(reinterpret_cast<const float4*>(f_row + (size_t)u * p.slice_stride + ca + f_half));
       }
     }
-    if (hh >= 0 && f_in_table) {
+    if (hh >= 0 && !f_unit && f_in_table) {
       pre_c = *reinterpret_cast<const float4*>(p.cos_t + (size_t)P * f_half + off);
       pre_s = *reinterpret_cast<const float4*>(p.sin_t + (size_t)P * f_half + off);
     }
@@ -452,9 +467,9 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
                            : smem + (size_t)STAGES * 2 * S::TILE_ELEMS;  // [16][RS]: the group's rotated query heads
   __nv_bfloat16* k_new = q_s + S::Q_ELEMS;                          // [D] rotated key of the row's own position
   __nv_bfloat16* v_new = k_new + D;                                 // [D] its value
+  float* gate_s = reinterpret_cast<float*>(v_new + D);              // [16][D] the output gate of the group's heads
   if (FUSED) {
-    const size_t width = (size_t)(p.nh + (p.has_kv ? 2 * p.nkv : 0)) * D;
-    const float* prow = p.partial + (size_t)dec_row * width;
+    const float* prow = f_row;
     auto value = [&](int col) -> float {
       float v = p.bias ? __bfloat162float(p.bias[col]) : 0.f;
       for (int k0 = 0; k0 < p.n_slices; k0 += 4) {  // four slices' loads in flight at once, added in slice order
@@ -469,6 +484,56 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
     const int half = p.rot / 2;
     const bool in_table = P >= 0 && P < p.table_rows;
     if (!in_table && half > 0 && threadIdx.x == 0 && p.err) atomicExch(p.err, CUCA_ERR_TOKEN_RANGE);
+    if (f_unit) {
+      auto sum4 = [&](int col, bool first) {  // four columns over the slices in order (plus bias)
+        float4 a = p.bias ? make_float4(__bfloat162float(p.bias[col]), __bfloat162float(p.bias[col + 1]),
+                                        __bfloat162float(p.bias[col + 2]), __bfloat162float(p.bias[col + 3]))
+                          : make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int k0 = 0; k0 < p.n_slices; k0 += 4) {
+          float4 x[4];
+#pragma unroll
+          for (int u = 0; u < 4; ++u) {
+            x[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (first && k0 == 0) x[u] = pre_a[u];
+            else if (k0 + u < p.n_slices) x[u] = __ldcg(reinterpret_cast<const float4*>(f_row + (size_t)(k0 + u) * p.slice_stride + col));
+          }
+#pragma unroll
+          for (int u = 0; u < 4; ++u) { a.x += x[u].x; a.y += x[u].y; a.z += x[u].z; a.w += x[u].w; }
+        }
+        return a;
+      };
+      auto put4 = [](__nv_bfloat16* dst, const float4 a, float m) {
+        *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16(a.x * m, a.y * m), pack_bf16(a.z * m, a.w * m));
+      };
+      for (int base = warp * 32; base < f_items; base += NTHREADS) {  // whole warps: D / 4 neighbouring lanes hold a head
+        const int it = base + lane;
+        int ca = 0, hh = 0, off = 0;
+        float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (it < f_items) {
+          f_item(it, ca, hh, off);
+          a = sum4(ca, it == (int)threadIdx.x);
+        }
+        float ss = a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;
+#pragma unroll
+        for (int o = D / 8; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        const float inv = 1.f / sqrtf(ss / (float)D + p.norm_eps);
+        if (it >= f_items) continue;
+        if (hh < G) {
+          put4(q_s + hh * S::RS + off, a, inv * (p.q_mul ? p.q_mul[kvh * G + hh] : 1.f));
+        } else {
+          if (hh == G) put4(k_new + off, a, inv);
+          if (hh > G || p.v_col == p.nh * D) put4(v_new + off, a, 1.f);
+        }
+      }
+      // the output gate, where this CTA may be the one that writes the result
+      if (p.gate_col >= 0 && (!p.cluster || n_used == 1 || cluster_rank() == 0)) {
+        for (int it = threadIdx.x; it < G * (D / 4); it += NTHREADS) {
+          const float4 a = sum4(p.gate_col + kvh * G * D + it * 4, false);
+          *reinterpret_cast<float4*>(gate_s + it * 4) =
+              make_float4(1.f / (1.f + __expf(-a.x)), 1.f / (1.f + __expf(-a.y)), 1.f / (1.f + __expf(-a.z)), 1.f / (1.f + __expf(-a.w)));
+        }
+      }
+    }
     if (f_vec) {
       auto add4 = [](float4& x, const float4 y) { x.x += y.x; x.y += y.y; x.z += y.z; x.w += y.w; };
       auto put4 = [](__nv_bfloat16* dst, float a, float b, float c, float d) {
@@ -516,7 +581,7 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
     }
     // per head: `half` rotated pairs (i, i + half), then the values beyond the rotary part as they are
     const int units = D - half;
-    const int heads_here = f_vec ? 0 : G + (owner ? 1 : 0);
+    const int heads_here = (f_vec || f_unit) ? 0 : G + (owner ? 1 : 0);
     for (int idx = threadIdx.x; idx < heads_here * units; idx += NTHREADS) {
       const int hh = idx / units, u = idx % units;
       const int col0 = hh < G ? (kvh * G + hh) * D : (p.nh + kvh) * D;
@@ -531,9 +596,9 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
         dst[u + half] = __float2bfloat16_rn(value(col0 + u + half));
       }
     }
-    if (owner && !f_vec)
+    if (owner && !f_vec && !f_unit)
       for (int i = threadIdx.x; i < D; i += NTHREADS)
-        v_new[i] = __float2bfloat16_rn(value((p.nh + p.nkv + kvh) * D + i));
+        v_new[i] = __float2bfloat16_rn(value(p.v_col + kvh * D + i));
     for (int idx = threadIdx.x; idx < (16 - G) * D; idx += NTHREADS)
       q_s[(G + idx / D) * S::RS + idx % D] = __float2bfloat16_rn(0.f);
     __syncthreads();
@@ -771,6 +836,7 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
   float* fs = reinterpret_cast<float*>(smem_raw);   // [4 warps][16 rows][D + 2]
   constexpr int FR = D + 2;
   auto gate_at = [&](int item, int dim) -> float {  // the factor on an output value of the group's head `item`
+    if (FUSED && p.gate_col >= 0) return gate_s[item * D + dim];
     return p.gate ? sigmoid_of(p.gate[(size_t)dec_row * p.gate_stride + (size_t)(kvh * G + item) * D + dim]) : 1.f;
   };
 #pragma unroll
@@ -1023,6 +1089,11 @@ struct FusedInput {
   const float* cos_t;
   const float* sin_t;
   int table_rows, rot, has_kv;
+  int width, v_col;
+  int unit = 0;
+  float norm_eps = 0.f;
+  const float* q_mul = nullptr;
+  int gate_col = -1;
 };
 
 void set_score_options(AttnParams& p, const CucaAttnOptions& o) {
@@ -1073,6 +1144,7 @@ int attention_decode_impl(const void* q, int q_stride, const FusedInput* fused, 
   p.cluster = by_cluster ? 1 : 0;
   p.partial = nullptr; p.n_slices = 0; p.slice_stride = 0; p.bias = nullptr; p.cos_t = p.sin_t = nullptr;
   p.table_rows = 0; p.rot = 0; p.has_kv = 0;
+  p.width = p.v_col = p.unit = 0; p.norm_eps = 0.f; p.q_mul = nullptr; p.gate_col = -1;
   static int env_tma = -1;
   if (env_tma < 0) { const char* e = getenv("CUCA_ATTN_TMA"); env_tma = e ? atoi(e) : 1; }
   // key/value groups of 16 positions by TMA: a group must lie in one page
@@ -1087,6 +1159,13 @@ int attention_decode_impl(const void* q, int q_stride, const FusedInput* fused, 
   p.partial = fused->partial; p.n_slices = fused->n_slices; p.slice_stride = fused->slice_stride;
   p.bias = (const __nv_bfloat16*)fused->bias; p.cos_t = fused->cos_t; p.sin_t = fused->sin_t;
   p.table_rows = fused->table_rows; p.rot = fused->rot; p.has_kv = fused->has_kv;
+  p.width = fused->width; p.v_col = fused->v_col; p.unit = fused->unit; p.norm_eps = fused->norm_eps;
+  p.q_mul = fused->q_mul; p.gate_col = fused->gate_col;
+  CUCA_REQUIRE(!fused->unit || (((d & (d - 1)) == 0) && fused->rot == 0 && fused->has_kv && fused->width % 4 == 0 &&
+                                fused->v_col % 4 == 0 && fused->slice_stride % 4 == 0 && ((uintptr_t)fused->partial & 15) == 0),
+               "attention_decode_fused: unit norms take head sizes 16, 32, 64 and 128, rows of 16-byte multiples and no rotation");
+  CUCA_REQUIRE(fused->gate_col < 0 || (fused->unit && fused->gate_col % 4 == 0 && fused->gate_col + nh * d <= fused->width),
+               "attention_decode_fused: the gate's %d columns at %d do not fit rows of %d", nh * d, fused->gate_col, fused->width);
   return dispatch<true, true>(d, p, dim3(n_splits, nkv, n_rows), stream, tma);
 }
 }  // namespace
@@ -1155,11 +1234,30 @@ CUCA_API int cuca_attention_decode_fused(const float* partial, int n_slices, siz
                                          int table_stride, const int* rows, int n_rows, int nh, int nkv, int d,
                                          float scale, int window, int chunk, int n_splits, float* part, int* counters,
                                          int* err, cudaStream_t stream) {
-  FusedInput f{partial, n_slices, slice_stride, bias, cos_t, sin_t, table_rows, rot, has_kv};
+  FusedInput f{partial, n_slices, slice_stride, bias, cos_t, sin_t, table_rows, rot, has_kv,
+               (nh + (has_kv ? 2 * nkv : 0)) * d, (nh + nkv) * d};
   const CucaAttnOptions opt{scale, window, 0, 0.f, 0, 0, nullptr, nullptr, nullptr};
   return attention_decode_impl(nullptr, 2, &f, out, out_stride, kpool, vpool, n_blocks, bs, positions, seq_of_row,
                                tables, table_stride, rows, n_rows, nh, nkv, d, opt, chunk, n_splits, part, counters, err,
                                stream);
+}
+
+// The same for layers without rotation whose queries and keys are divided by their root mean square per head (no weight):
+// slices of rows of `width` columns, q heads at 0, k heads at nh d, v heads at v_col (nh d: the values are the keys as
+// projected), the pre-activations of an output gate at gate_col (< 0: no gate). q_mul (or null): a factor on the queries of
+// each head. Window, kept first keys, cap, distance bias and sink as `opt` says (its own gate must be null).
+CUCA_API int cuca_attention_decode_fused_unit(const float* partial, int n_slices, size_t slice_stride, const void* bias,
+                                              int width, int v_col, int gate_col, float norm_eps, const float* q_mul,
+                                              void* out, int out_stride, void* kpool, void* vpool, int n_blocks, int bs,
+                                              const int* positions, const int* seq_of_row, const int* tables,
+                                              int table_stride, const int* rows, int n_rows, int nh, int nkv, int d,
+                                              const CucaAttnOptions* opt, int chunk, int n_splits, float* part,
+                                              int* counters, int* err, cudaStream_t stream) {
+  CUCA_REQUIRE(opt != nullptr && opt->gate == nullptr, "attention_decode_fused: bad options");
+  CUCA_REQUIRE(v_col >= nh * d && v_col + nkv * d <= width, "attention_decode_fused: values at column %d do not fit rows of %d", v_col, width);
+  FusedInput f{partial, n_slices, slice_stride, bias, nullptr, nullptr, 0, 0, 1, width, v_col, 1, norm_eps, q_mul, gate_col};
+  return attention_decode_impl(nullptr, 2, &f, out, out_stride, kpool, vpool, n_blocks, bs, positions, seq_of_row, tables,
+                               table_stride, rows, n_rows, nh, nkv, d, *opt, chunk, n_splits, part, counters, err, stream);
 }
 
 // Prefill form: tile i covers rows tile_row0[i] .. +tile_nrows[i]-1 (at most 64 consecutive rows of one request).
@@ -1184,6 +1282,7 @@ CUCA_API int cuca_attention_prefill_o(const void* q, int q_stride, void* out, in
   set_score_options(p, *opt);
   p.partial = nullptr; p.n_slices = 0; p.slice_stride = 0; p.bias = nullptr; p.cos_t = p.sin_t = nullptr;
   p.table_rows = 0; p.rot = 0; p.has_kv = 0;
+  p.width = p.v_col = p.unit = 0; p.norm_eps = 0.f; p.q_mul = nullptr; p.gate_col = -1;
   return dispatch<false, false>(d, p, dim3(n_tiles, nh), stream);
 }
 

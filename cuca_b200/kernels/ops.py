@@ -549,6 +549,23 @@ def attention_decode_fused(partial, bias, cos, sin, rotary_dim, has_kv, out, kpo
         _p(err), _stream()), "attention_decode_fused")
 
 
+def attention_decode_fused_unit(partial, bias, v_col, gate_col, eps, q_mul, out, cache, step, n_rows, n_heads, n_kv_heads,
+                                head_dim, scale, window, chunk, n_splits, err, **options) -> None:
+    """The decode form fed by a stacked projection's unadded K slices for layers without rotation whose queries and keys are
+    divided by their root mean square per head: adds the slices, norms, multiplies the queries by `q_mul` (one factor per
+    query head, or None), stores the page rows, attends and applies the output gate whose pre-activations stand at column
+    `gate_col` (None: no gate), in one launch. Columns: q heads at 0, k heads behind them, v heads at `v_col` (the k heads'
+    column: the values are the keys as projected). Every row of the step is a single token."""
+    part, cnt = _decode_scratch(out.device, n_rows, n_heads, n_kv_heads, head_dim, n_splits)
+    opt = attention_options(n_heads, scale, window, **options)
+    library.check(library.load().cuca_attention_decode_fused_unit(
+        _p(partial.data), partial.slices, partial.slice_stride, _p(bias), partial.data.shape[2], int(v_col),
+        -1 if gate_col is None else int(gate_col), float(eps), _per_head(q_mul, n_heads, "factors on the queries"), _p(out),
+        out.stride(0), _p(cache.k), _p(cache.v), cache.k.shape[0], cache.k.shape[2], _p(step.positions),
+        _p(step.seq_of_row), _p(cache.tables), cache.tables.shape[1], None, n_rows, n_heads, n_kv_heads, head_dim,
+        ctypes.addressof(opt), chunk, n_splits, _p(part), _p(cnt), _p(err), _stream()), "attention_decode_fused_unit")
+
+
 def attention_decode_fused_supported(plan, cache, out_dtype, n_rows, n_heads, n_kv_heads, head_dim) -> bool:
     """True when every row of the step is a single token of its request and the tensor-core decode form takes
     the shape: then rotate-and-store and attention are one launch."""

@@ -120,6 +120,9 @@ class PagedAttention(Mixer):
             raise ValueError("attention: a layer that reads another layer's pages takes neither a value size of its "
                              "own, an output gate, head norms, a score cap, a sink, a distance bias, kept first keys nor "
                              "adjacent rotation pairs")
+        # what the decode kernel that makes its own queries and keys takes
+        self.fusable = (self.norm_unit and self.position is None and self.q_temp is None and not self.v_norm
+                        and not self.head_gate and self.v_head_dim == self.head_dim and self.head_dim in (16, 32, 64, 128))
         # the width of a value row in the pool: padded to a multiple of the key size for the tensor-core kernels
         self.v_pool_dim = self.v_head_dim
         d, dv = self.head_dim, self.v_head_dim
@@ -225,13 +228,28 @@ class PagedAttention(Mixer):
         nh, nkv, d, dv = self.n_heads, self.n_kv_heads, self.head_dim, self.v_pool_dim  # (dv: of pool and output)
         dv_row = self.v_head_dim if dv != self.v_head_dim else 0  # the projection's value heads, where narrower
         rows = h.shape[0]
-        proj = self.rt.linear(h, self.w_qkv, bias=self.b_qkv)
         v_col = nh * d if self.keys_as_values else (nh + nkv) * d
         g_col = v_col + nkv * self.v_head_dim
         scale = 1.0 if self.q_scaled else self.scale
         cos, sin, rot, adjacent = self.position.tables() if self.position is not None else (None, None, 0, False)
         split = self.value_split(cache)
         plan = self.plan(step) if split else None
+        options = {"softcap": self.softcap, "sink": self.sink, "sink_values": self.sink_values, "keep_first": self.keep_first,
+                   "slopes": self.slopes}
+        if (self.fusable and split == 1 and self.rt.use_partials and rows <= ops.ROPE_PARTIAL_MAX_ROWS
+                and ops.attention_decode_fused_supported(plan, cache, h.dtype, rows, nh, nkv, d)
+                and ops.gemm_partial_supported(h, self.w_qkv)):
+            # single tokens only: the projection leaves its K slices unadded; adding them, the norms, the page write,
+            # attention and the gate are one launch
+            parts = ops.gemm_partial(h, self.w_qkv, self.rt.err)
+            attn = self.rt.empty(rows, nh * d)
+            chunk, n_splits = plan.chunk(nkv, d, self.window, self.keep_first)
+            ops.attention_decode_fused_unit(parts, self.b_qkv, v_col, g_col if self.gated else None, self.eps, self.q_mul,
+                                            attn, cache, step, rows, nh, nkv, d, scale, self.window, chunk, n_splits,
+                                            self.rt.err, **options)
+            stream.add_linear(attn, self.w_o, bias=self.b_o)
+            return
+        proj = self.rt.linear(h, self.w_qkv, bias=self.b_qkv)
         if split > 1 and plan is None:
             raise ValueError("attention: this layer's value pool is laid out for the tensor-core kernels, which need "
                              "the step's per-request description")
@@ -247,8 +265,6 @@ class PagedAttention(Mixer):
                                    rot, adjacent, cache.k, cache.v, cache.block_size, nh, nkv, d, dv, self.rt.err,
                                    v_split=split, v_row_dim=dv_row)
         gate = proj[:, g_col:g_col + nh * dv] if self.gated else None  # (a layer with a gate per value is never padded)
-        options = {"softcap": self.softcap, "sink": self.sink, "sink_values": self.sink_values, "keep_first": self.keep_first,
-                   "slopes": self.slopes}
         attn = self.rt.empty(rows, nh * dv)
         if tensor_cores:
             slabs = cache.v.view(split, *cache.k.shape)
