@@ -73,8 +73,7 @@ struct AttnParams {
   int has_kv;            // 0: the layer reads another layer's pages and has only q
   int width;             // columns of a slice's row: q heads at 0, k heads at nh D, v heads at v_col
   int v_col;             // (nh D: the values are the keys as projected)
-  int unit;              // 1: instead of the rotation, q and k are divided by their root mean square per head, and ...
-  float norm_eps;
+  float norm_eps;        // unit norms: q and k are divided by their root mean square per head, and ...
   const float* q_mul;    // ... q is multiplied by its head's factor (or null)
   int gate_col;          // >= 0: the pre-activations of an output gate stand there, one per output value
 };
@@ -132,10 +131,9 @@ struct Smem {
   static constexpr int RS = D + 8;  // row stride in elements: 16 bytes of padding
   static constexpr int TILE_ELEMS = TILE * RS;
   static constexpr int BYTES = STAGES * 2 /*k, v*/ * TILE_ELEMS * 2;
-  // fused form: the 16 query rows, then the new key and the new value of the row, then the gate's values
+  // fused form: the 16 query rows, then the new key and the new value of the row
   static constexpr int Q_ELEMS = 16 * RS;
-  static constexpr int GATE_BYTES = 16 * D * 4;  // the output gate of the group's heads
-  static constexpr int FUSED_BYTES = BYTES + (Q_ELEMS + 2 * D) * 2 + GATE_BYTES;
+  static constexpr int FUSED_BYTES = BYTES + (Q_ELEMS + 2 * D) * 2;
   // decode with TMA: every warp has a ring of its own; a stage holds the warp's 16 keys and values as
   // 64-wide halves of 16 rows x 128 bytes, 128-byte swizzled: K half 0, K half 1, ..., V half 0, ...
   static constexpr int HALVES = D / 64;
@@ -143,7 +141,7 @@ struct Smem {
   static constexpr int WSTAGE_BYTES = 2 * (HALVES > 0 ? HALVES : 1) * SUB_BYTES;
   static constexpr int WSTAGES = 3;
   static constexpr int RING_BYTES = 4 * WSTAGES * WSTAGE_BYTES;
-  static constexpr int TMA_BYTES = RING_BYTES + 1024 /*alignment*/ + (Q_ELEMS + 2 * D) * 2 + GATE_BYTES;
+  static constexpr int TMA_BYTES = RING_BYTES + 1024 /*alignment*/ + (Q_ELEMS + 2 * D) * 2;
 };
 
 // One warp's state over its 16 MMA rows: thread (g, t) holds rows g and g + 8.
@@ -166,7 +164,8 @@ __device__ __forceinline__ float sink_term(float m, const AttnParams& p, int hea
   return exp2f((p.sink_val ? p.sink_val[head] * 1.4426950408889634f : 0.f) - m);
 }
 
-template <int D, bool DECODE, bool FUSED, bool TMA>
+// FUSED: 1: decode fed by the projection's K slices, with rotation; 2: with unit norms per head instead (and an output gate)
+template <int D, bool DECODE, int FUSED, bool TMA>
 __global__ void __launch_bounds__(NTHREADS)
 attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV) {
   static_assert(!FUSED || DECODE, "only the decode form takes the projection's K slices");
@@ -183,7 +182,7 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
   // page tables were brought up to date before that, and every key it copies was written by an earlier step
   // (the row's own key comes from registers). So its lookups and its first copies go out before the dependency
   // wait and overlap the projection's tail. Every other form waits here.
-  constexpr bool EARLY = FUSED && TMA;
+  constexpr bool EARLY = FUSED != 0 && TMA;
   if (!EARLY) pdl_wait();
 
   // ---------------------------------------------------------------- what this CTA and warp own
@@ -371,7 +370,7 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
   const size_t f_width = FUSED ? (size_t)p.width : 0;
   const float* f_row = FUSED ? p.partial + (size_t)dec_row * f_width : nullptr;
   const bool f_in_table = FUSED && P >= 0 && P < p.table_rows;
-  const bool f_unit = FUSED && p.unit;
+  constexpr bool f_unit = FUSED == 2;
   const bool f_vec = FUSED && !f_unit && p.rot == D && D % 8 == 0 && ((p.slice_stride | f_width) & 3) == 0 &&
                      (((uintptr_t)p.partial | (uintptr_t)p.cos_t | (uintptr_t)p.sin_t) & 15) == 0;
   const int f_hq = f_half / 4;                                   // items per rotated head
@@ -463,11 +462,36 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
     preload();
   }
   // ---------------------------------------------------------------- fused form: q (and k, v) from the K slices
+  auto sum4 = [&](int col, bool first) {  // four columns over the slices in order (plus bias)
+    float4 a = p.bias ? make_float4(__bfloat162float(p.bias[col]), __bfloat162float(p.bias[col + 1]),
+                                    __bfloat162float(p.bias[col + 2]), __bfloat162float(p.bias[col + 3]))
+                      : make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int k0 = 0; k0 < p.n_slices; k0 += 4) {
+      float4 x[4];
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        x[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (first && k0 == 0) x[u] = pre_a[u];
+        else if (k0 + u < p.n_slices) x[u] = __ldcg(reinterpret_cast<const float4*>(f_row + (size_t)(k0 + u) * p.slice_stride + col));
+      }
+#pragma unroll
+      for (int u = 0; u < 4; ++u) { a.x += x[u].x; a.y += x[u].y; a.z += x[u].z; a.w += x[u].w; }
+    }
+    return a;
+  };
+  // The output gate of the group's heads, where this CTA may be the one that writes the result: asked for here, kept in
+  // registers (four columns a thread; more heads than that are read at the end).
+  const bool f_gated = f_unit && p.gate_col >= 0;
+  auto gate4 = [&](int it) {
+    const float4 a = sum4(p.gate_col + kvh * G * D + it * 4, false);
+    return make_float4(1.f / (1.f + __expf(-a.x)), 1.f / (1.f + __expf(-a.y)), 1.f / (1.f + __expf(-a.z)), 1.f / (1.f + __expf(-a.w)));
+  };
+  float4 gate_r = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (f_gated && (int)threadIdx.x < G * (D / 4) && (!p.cluster || n_used == 1 || cluster_rank() == 0)) gate_r = gate4(threadIdx.x);
   __nv_bfloat16* q_s = TMA ? reinterpret_cast<__nv_bfloat16*>(ring_base + S::RING_BYTES)
                            : smem + (size_t)STAGES * 2 * S::TILE_ELEMS;  // [16][RS]: the group's rotated query heads
   __nv_bfloat16* k_new = q_s + S::Q_ELEMS;                          // [D] rotated key of the row's own position
   __nv_bfloat16* v_new = k_new + D;                                 // [D] its value
-  float* gate_s = reinterpret_cast<float*>(v_new + D);              // [16][D] the output gate of the group's heads
   if (FUSED) {
     const float* prow = f_row;
     auto value = [&](int col) -> float {
@@ -485,23 +509,6 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
     const bool in_table = P >= 0 && P < p.table_rows;
     if (!in_table && half > 0 && threadIdx.x == 0 && p.err) atomicExch(p.err, CUCA_ERR_TOKEN_RANGE);
     if (f_unit) {
-      auto sum4 = [&](int col, bool first) {  // four columns over the slices in order (plus bias)
-        float4 a = p.bias ? make_float4(__bfloat162float(p.bias[col]), __bfloat162float(p.bias[col + 1]),
-                                        __bfloat162float(p.bias[col + 2]), __bfloat162float(p.bias[col + 3]))
-                          : make_float4(0.f, 0.f, 0.f, 0.f);
-        for (int k0 = 0; k0 < p.n_slices; k0 += 4) {
-          float4 x[4];
-#pragma unroll
-          for (int u = 0; u < 4; ++u) {
-            x[u] = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (first && k0 == 0) x[u] = pre_a[u];
-            else if (k0 + u < p.n_slices) x[u] = __ldcg(reinterpret_cast<const float4*>(f_row + (size_t)(k0 + u) * p.slice_stride + col));
-          }
-#pragma unroll
-          for (int u = 0; u < 4; ++u) { a.x += x[u].x; a.y += x[u].y; a.z += x[u].z; a.w += x[u].w; }
-        }
-        return a;
-      };
       auto put4 = [](__nv_bfloat16* dst, const float4 a, float m) {
         *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16(a.x * m, a.y * m), pack_bf16(a.z * m, a.w * m));
       };
@@ -523,14 +530,6 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
         } else {
           if (hh == G) put4(k_new + off, a, inv);
           if (hh > G || p.v_col == p.nh * D) put4(v_new + off, a, 1.f);
-        }
-      }
-      // the output gate, where this CTA may be the one that writes the result
-      if (p.gate_col >= 0 && (!p.cluster || n_used == 1 || cluster_rank() == 0)) {
-        for (int it = threadIdx.x; it < G * (D / 4); it += NTHREADS) {
-          const float4 a = sum4(p.gate_col + kvh * G * D + it * 4, false);
-          *reinterpret_cast<float4*>(gate_s + it * 4) =
-              make_float4(1.f / (1.f + __expf(-a.x)), 1.f / (1.f + __expf(-a.y)), 1.f / (1.f + __expf(-a.z)), 1.f / (1.f + __expf(-a.w)));
         }
       }
     }
@@ -661,29 +660,32 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
       float mx = -INFINITY;
+#pragma unroll
+      for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) s[nt][2 * h + e] = score_log2(s[nt][2 * h + e], p);
+      if (p.slopes) {
+        const float d0 = (float)(row_pos[h] - kp0 - 2 * t);  // the distance of the thread's first key
+#pragma unroll
+        for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+          for (int e = 0; e < 2; ++e) s[nt][2 * h + e] = fmaf(-slope2[h], d0 - (float)(nt * 8 + e), s[nt][2 * h + e]);
+      }
       if (whole) {
 #pragma unroll
         for (int nt = 0; nt < NT; ++nt)
 #pragma unroll
-          for (int e = 0; e < 2; ++e) {
-            float v = score_log2(s[nt][2 * h + e], p);
-            if (p.slopes) v = fmaf(-slope2[h], (float)(row_pos[h] - (kp0 + nt * 8 + 2 * t + e)), v);
-            s[nt][2 * h + e] = v;
-            mx = fmaxf(mx, v);
-          }
+          for (int e = 0; e < 2; ++e) mx = fmaxf(mx, s[nt][2 * h + e]);
       } else {
-        int lo_row = (p.window > 0 && row_pos[h] - (p.window - 1) > 0) ? row_pos[h] - (p.window - 1) : 0;
+        const int lo_row = (p.window > 0 && row_pos[h] - (p.window - 1) > 0) ? row_pos[h] - (p.window - 1) : 0;
 #pragma unroll
         for (int nt = 0; nt < NT; ++nt)
 #pragma unroll
           for (int e = 0; e < 2; ++e) {
-            int kp = kp0 + nt * 8 + 2 * t + e;
-            bool ok = row_ok[h] && kp <= row_pos[h] && (kp >= lo_row || kp < p.keep);
-            float v = score_log2(s[nt][2 * h + e], p);
-            if (p.slopes) v = fmaf(-slope2[h], (float)(row_pos[h] - kp), v);
-            v = ok ? v : -INFINITY;
-            s[nt][2 * h + e] = v;
-            mx = fmaxf(mx, v);
+            const int kp = kp0 + nt * 8 + 2 * t + e;
+            const bool ok = row_ok[h] && kp <= row_pos[h] && (kp >= lo_row || kp < p.keep);
+            if (!ok) s[nt][2 * h + e] = -INFINITY;
+            mx = fmaxf(mx, s[nt][2 * h + e]);
           }
       }
       mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
@@ -835,8 +837,12 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
   __syncthreads();
   float* fs = reinterpret_cast<float*>(smem_raw);   // [4 warps][16 rows][D + 2]
   constexpr int FR = D + 2;
+  float* gate_s = fs + (size_t)5 * 16 * FR;  // [16][D] the output gate of the group's heads
+  if (f_gated)
+    for (int it = threadIdx.x; it < G * (D / 4); it += NTHREADS)
+      *reinterpret_cast<float4*>(gate_s + it * 4) = it == (int)threadIdx.x ? gate_r : gate4(it);
   auto gate_at = [&](int item, int dim) -> float {  // the factor on an output value of the group's head `item`
-    if (FUSED && p.gate_col >= 0) return gate_s[item * D + dim];
+    if (f_gated) return gate_s[item * D + dim];
     return p.gate ? sigmoid_of(p.gate[(size_t)dec_row * p.gate_stride + (size_t)(kvh * G + item) * D + dim]) : 1.f;
   };
 #pragma unroll
@@ -1011,11 +1017,12 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
   if (threadIdx.x == 0) p.counters[blockIdx.z * p.nkv + kvh] = 0;
 }
 
-template <int D, bool DECODE, bool FUSED, bool TMA>
+template <int D, bool DECODE, int FUSED, bool TMA>
 int launch(const AttnParams& p, const CUtensorMap& tmK, const CUtensorMap& tmV, dim3 grid, cudaStream_t stream) {
   int smem = TMA ? Smem<D>::TMA_BYTES : FUSED ? Smem<D>::FUSED_BYTES : Smem<D>::BYTES;
   if (DECODE) {
-    int need = 5 * 16 * (D + 2) * (int)sizeof(float) + (TMA ? 1024 : 0);  // four warps' results, then the CTA's
+    // four warps' results, then the CTA's, then the output gate
+    int need = (5 * 16 * (D + 2) + (FUSED == 2 ? 16 * D : 0)) * (int)sizeof(float) + (TMA ? 1024 : 0);
     if (need > smem) smem = need;
   }
   static bool configured = false;
@@ -1036,7 +1043,7 @@ int launch(const AttnParams& p, const CUtensorMap& tmK, const CUtensorMap& tmV, 
 }
 
 // tma: key/value groups by TMA (decode, head sizes 64 and 128, pages of at least 16 positions)
-template <bool DECODE, bool FUSED = false>
+template <bool DECODE, int FUSED = 0>
 int dispatch(int d, const AttnParams& p, dim3 grid, cudaStream_t stream, bool tma = false) {
   CUtensorMap tmK, tmV;
   memset(&tmK, 0, sizeof(tmK));
@@ -1053,12 +1060,16 @@ int dispatch(int d, const AttnParams& p, dim3 grid, cudaStream_t stream, bool tm
   switch (d) {
     case 16: return launch<16, DECODE, FUSED, false>(p, tmK, tmV, grid, stream);
     case 32: return launch<32, DECODE, FUSED, false>(p, tmK, tmV, grid, stream);
-    case 48: return launch<48, DECODE, FUSED, false>(p, tmK, tmV, grid, stream);
     case 64: return launch<64, DECODE, FUSED, false>(p, tmK, tmV, grid, stream);
-    case 80: return launch<80, DECODE, FUSED, false>(p, tmK, tmV, grid, stream);
-    case 96: return launch<96, DECODE, FUSED, false>(p, tmK, tmV, grid, stream);
-    case 112: return launch<112, DECODE, FUSED, false>(p, tmK, tmV, grid, stream);
     case 128: return launch<128, DECODE, FUSED, false>(p, tmK, tmV, grid, stream);
+  }
+  if constexpr (FUSED != 2) {  // (whose heads are a power of two lanes wide)
+    switch (d) {
+      case 48: return launch<48, DECODE, FUSED, false>(p, tmK, tmV, grid, stream);
+      case 80: return launch<80, DECODE, FUSED, false>(p, tmK, tmV, grid, stream);
+      case 96: return launch<96, DECODE, FUSED, false>(p, tmK, tmV, grid, stream);
+      case 112: return launch<112, DECODE, FUSED, false>(p, tmK, tmV, grid, stream);
+    }
   }
   cuca_set_error("attention_mma: head size %d is not one of 16, 32, ..., 128", d);
   return 1;
@@ -1144,12 +1155,12 @@ int attention_decode_impl(const void* q, int q_stride, const FusedInput* fused, 
   p.cluster = by_cluster ? 1 : 0;
   p.partial = nullptr; p.n_slices = 0; p.slice_stride = 0; p.bias = nullptr; p.cos_t = p.sin_t = nullptr;
   p.table_rows = 0; p.rot = 0; p.has_kv = 0;
-  p.width = p.v_col = p.unit = 0; p.norm_eps = 0.f; p.q_mul = nullptr; p.gate_col = -1;
+  p.width = p.v_col = 0; p.norm_eps = 0.f; p.q_mul = nullptr; p.gate_col = -1;
   static int env_tma = -1;
   if (env_tma < 0) { const char* e = getenv("CUCA_ATTN_TMA"); env_tma = e ? atoi(e) : 1; }
   // key/value groups of 16 positions by TMA: a group must lie in one page
   const bool tma = env_tma && d % 64 == 0 && bs >= 16 && ((uintptr_t)kpool & 15) == 0 && ((uintptr_t)vpool & 15) == 0;
-  if (!fused) return dispatch<true, false>(d, p, dim3(n_splits, nkv, n_rows), stream, tma);
+  if (!fused) return dispatch<true, 0>(d, p, dim3(n_splits, nkv, n_rows), stream, tma);
   CUCA_REQUIRE(fused->partial && fused->n_slices >= 1, "attention_decode_fused: no projection slices");
   CUCA_REQUIRE(fused->rot >= 0 && fused->rot <= d && fused->rot % 2 == 0,
                "attention_decode_fused: rotary size %d does not fit head size %d", fused->rot, d);
@@ -1159,14 +1170,15 @@ int attention_decode_impl(const void* q, int q_stride, const FusedInput* fused, 
   p.partial = fused->partial; p.n_slices = fused->n_slices; p.slice_stride = fused->slice_stride;
   p.bias = (const __nv_bfloat16*)fused->bias; p.cos_t = fused->cos_t; p.sin_t = fused->sin_t;
   p.table_rows = fused->table_rows; p.rot = fused->rot; p.has_kv = fused->has_kv;
-  p.width = fused->width; p.v_col = fused->v_col; p.unit = fused->unit; p.norm_eps = fused->norm_eps;
+  p.width = fused->width; p.v_col = fused->v_col; p.norm_eps = fused->norm_eps;
   p.q_mul = fused->q_mul; p.gate_col = fused->gate_col;
   CUCA_REQUIRE(!fused->unit || (((d & (d - 1)) == 0) && fused->rot == 0 && fused->has_kv && fused->width % 4 == 0 &&
                                 fused->v_col % 4 == 0 && fused->slice_stride % 4 == 0 && ((uintptr_t)fused->partial & 15) == 0),
                "attention_decode_fused: unit norms take head sizes 16, 32, 64 and 128, rows of 16-byte multiples and no rotation");
   CUCA_REQUIRE(fused->gate_col < 0 || (fused->unit && fused->gate_col % 4 == 0 && fused->gate_col + nh * d <= fused->width),
                "attention_decode_fused: the gate's %d columns at %d do not fit rows of %d", nh * d, fused->gate_col, fused->width);
-  return dispatch<true, true>(d, p, dim3(n_splits, nkv, n_rows), stream, tma);
+  return fused->unit ? dispatch<true, 2>(d, p, dim3(n_splits, nkv, n_rows), stream, tma)
+                     : dispatch<true, 1>(d, p, dim3(n_splits, nkv, n_rows), stream, tma);
 }
 }  // namespace
 
@@ -1282,8 +1294,8 @@ CUCA_API int cuca_attention_prefill_o(const void* q, int q_stride, void* out, in
   set_score_options(p, *opt);
   p.partial = nullptr; p.n_slices = 0; p.slice_stride = 0; p.bias = nullptr; p.cos_t = p.sin_t = nullptr;
   p.table_rows = 0; p.rot = 0; p.has_kv = 0;
-  p.width = p.v_col = p.unit = 0; p.norm_eps = 0.f; p.q_mul = nullptr; p.gate_col = -1;
-  return dispatch<false, false>(d, p, dim3(n_tiles, nh), stream);
+  p.width = p.v_col = 0; p.norm_eps = 0.f; p.q_mul = nullptr; p.gate_col = -1;
+  return dispatch<false, 0>(d, p, dim3(n_tiles, nh), stream);
 }
 
 // (softcap and sink as in the decode form)

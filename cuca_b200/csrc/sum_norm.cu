@@ -21,12 +21,13 @@ struct SumNorm {
   int E;
 };
 
-template <int V>
+template <int V, int AHEAD = 4>
 __device__ __forceinline__ Pack<V> summed(const SumNorm& p, size_t row, int i) {
-  Pack<V> z = term_sum<V>(p.terms, row * p.E + i);
   const Pack<V> x = ld_cg<V>(p.x + row * p.E + i);
+  Pack<V> s;
+  if (p.s) s = ld<V>(p.s + i);
+  Pack<V> z = term_sum<V, AHEAD>(p.terms, row * p.E + i);
   if (p.s) {
-    const Pack<V> s = ld<V>(p.s + i);
 #pragma unroll
     for (int k = 0; k < V; ++k) z.v[k] *= s.v[k];
   }
@@ -58,7 +59,7 @@ __device__ __forceinline__ void block_sums(float (&s)[N], float* red) {
 // One block per row. R > 0: a thread holds R packs of V values (blockDim R V >= E); R = 0: the sum stays in x between the
 // passes (rows wider than a block can hold).
 template <typename TO, int V, int R>
-__global__ void __launch_bounds__(1024)
+__global__ void __launch_bounds__(1024, 1)
 sum_norm_kernel(const SumNorm p, float* __restrict__ x, TO* __restrict__ out) {
   __shared__ float red[32];
   pdl_trigger();
@@ -68,19 +69,20 @@ sum_norm_kernel(const SumNorm p, float* __restrict__ x, TO* __restrict__ out) {
   constexpr int HELD = R > 0 ? R : 1;
   Pack<V> z[HELD];
   float q[1] = {0.f};
-  auto finish = [&](int i, Pack<V> v, float inv) {
-    const Pack<V> w = ld<V>(p.w + i);
+  auto finish = [&](int i, Pack<V> v, const Pack<V> w, float inv) {
 #pragma unroll
     for (int k = 0; k < V; ++k) v.v[k] = v.v[k] * inv * w.v[k];
     st<V>(x + row * p.E + i, v);
     if (out) st<V>(out + row * p.E + i, v);
   };
+  Pack<V> wv[HELD];  // (asked for before the reduction)
   if (R > 0) {
 #pragma unroll
     for (int r = 0; r < R; ++r) {
       const int i = threadIdx.x * V + r * step;
       if (i >= p.E) continue;
-      z[r] = summed<V>(p, row, i);
+      wv[r] = ld<V>(p.w + i);
+      z[r] = summed<V, R == 1 ? 8 : 4>(p, row, i);
 #pragma unroll
       for (int k = 0; k < V; ++k) q[0] = fmaf(z[r].v[k], z[r].v[k], q[0]);
     }
@@ -98,10 +100,10 @@ sum_norm_kernel(const SumNorm p, float* __restrict__ x, TO* __restrict__ out) {
 #pragma unroll
     for (int r = 0; r < R; ++r) {
       const int i = threadIdx.x * V + r * step;
-      if (i < p.E) finish(i, z[r], inv);
+      if (i < p.E) finish(i, z[r], wv[r], inv);
     }
   } else {
-    for (int i = threadIdx.x * V; i < p.E; i += step) finish(i, ld<V>(x + row * p.E + i), inv);
+    for (int i = threadIdx.x * V; i < p.E; i += step) finish(i, ld<V>(x + row * p.E + i), ld<V>(p.w + i), inv);
   }
 }
 
@@ -119,7 +121,7 @@ struct Shift {
 // first row of the step and written by the same block after that, be the last row its own or not (then it is worked out
 // here once more), so no two blocks touch it.
 template <typename TO, int V, int R, int ROWS>
-__global__ void __launch_bounds__(1024)
+__global__ void __launch_bounds__(1024, 1)
 sum_norm_shift_kernel(const SumNorm p, const Shift sh, float* __restrict__ x_out, TO* __restrict__ out) {
   __shared__ float red[32 * (ROWS + 1)];
   __shared__ int s_last;
@@ -136,6 +138,15 @@ sum_norm_shift_kernel(const SumNorm p, const Shift sh, float* __restrict__ x_out
   if (seq[0] != seq[1]) seq[0] = -1;  // the row before belongs to another request
   Pack<V> z[ROWS + 1][R];
   float q[ROWS + 1];
+  // one row a block (single tokens, mostly): what the rest of the row needs is asked for before the reduction
+  constexpr bool EARLY = ROWS == 1 && R == 1;
+  Pack<V> wv, mixv, keptv;
+  const int i0 = threadIdx.x * V;
+  if (EARLY && i0 < p.E && seq[1] >= 0) {
+    wv = ld<V>(p.w + i0);
+    mixv = ld<V>(sh.mix + i0);
+    if (seq[0] < 0) keptv = ld_cg<V>(sh.kept + (size_t)seq[1] * p.E + i0);
+  }
 #pragma unroll
   for (int j = 0; j <= ROWS; ++j) {
     q[j] = 0.f;
@@ -145,7 +156,7 @@ sum_norm_shift_kernel(const SumNorm p, const Shift sh, float* __restrict__ x_out
 #pragma unroll
       for (int k = 0; k < V; ++k) z[j][r].v[k] = 0.f;
       if (seq[j] < 0 || i >= p.E) continue;
-      z[j][r] = summed<V>(p, r0 - 1 + j, i);
+      z[j][r] = summed<V, EARLY ? 8 : 4>(p, r0 - 1 + j, i);
 #pragma unroll
       for (int k = 0; k < V; ++k) q[j] = fmaf(z[j][r].v[k], z[j][r].v[k], q[j]);
     }
@@ -157,8 +168,8 @@ sum_norm_shift_kernel(const SumNorm p, const Shift sh, float* __restrict__ x_out
 #pragma unroll
     for (int r = 0; r < R; ++r) {
       const int i = threadIdx.x * V + r * step;
-      if (i >= p.E) continue;
-      const Pack<V> w = ld<V>(p.w + i);
+      if (i >= p.E || seq[j] < 0) continue;
+      const Pack<V> w = EARLY ? wv : ld<V>(p.w + i);
 #pragma unroll
       for (int k = 0; k < V; ++k) z[j][r].v[k] = z[j][r].v[k] * inv * w.v[k];
     }
@@ -178,7 +189,7 @@ sum_norm_shift_kernel(const SumNorm p, const Shift sh, float* __restrict__ x_out
       Pack<V> h = z[j][r];
       if (seq[j] >= 0) {
         float* keep = sh.kept + (size_t)seq[j] * p.E + i;
-        const Pack<V> before = first ? ld_cg<V>(keep) : z[j - 1][r], mix = ld<V>(sh.mix + i);
+        const Pack<V> before = first ? (EARLY ? keptv : ld_cg<V>(keep)) : z[j - 1][r], mix = EARLY ? mixv : ld<V>(sh.mix + i);
 #pragma unroll
         for (int k = 0; k < V; ++k) h.v[k] = fmaf(before.v[k] - h.v[k], mix.v[k], h.v[k]);
         if (last && open == seq[j]) st<V>(keep, z[j][r]);

@@ -44,7 +44,8 @@ template <int V> __device__ __forceinline__ Pack<V> ld_cg(const float* p) {
 }
 
 // y[at .. at + V) of the weighted sum of the terms
-template <int V>
+// (AHEAD slices' loads in flight at once, added in slice order)
+template <int V, int AHEAD = 4>
 __device__ __forceinline__ Pack<V> term_sum(const CucaTerms& t, size_t at) {
   Pack<V> y;
 #pragma unroll
@@ -54,10 +55,10 @@ __device__ __forceinline__ Pack<V> term_sum(const CucaTerms& t, size_t at) {
     Pack<V> s;
 #pragma unroll
     for (int k = 0; k < V; ++k) s.v[k] = 0.f;
-    for (int k0 = 0; k0 < t.slices[i]; k0 += 4) {  // four slices' loads in flight at once, added in slice order
-      Pack<V> q[4];
+    for (int k0 = 0; k0 < t.slices[i]; k0 += AHEAD) {
+      Pack<V> q[AHEAD];
 #pragma unroll
-      for (int u = 0; u < 4; ++u) {
+      for (int u = 0; u < AHEAD; ++u) {
         if (k0 + u < t.slices[i]) q[u] = ld_cg<V>(p + (k0 + u) * t.stride[i]);
         else {
 #pragma unroll
@@ -65,7 +66,7 @@ __device__ __forceinline__ Pack<V> term_sum(const CucaTerms& t, size_t at) {
         }
       }
 #pragma unroll
-      for (int u = 0; u < 4; ++u)
+      for (int u = 0; u < AHEAD; ++u)
 #pragma unroll
         for (int k = 0; k < V; ++k) s.v[k] += q[u].v[k];
     }
