@@ -33,14 +33,14 @@ def plan_groups(cache_needs: dict, kv_tokens: int, block_size: int, max_sequence
         if kv is None:
             continue
         keep = kv.keep_first if kv.window is not None else 0
-        by_key.setdefault((kv.n_kv_heads, kv.head_dim, kv.window, kv.v_head_dim, keep), []).append(cid)
+        by_key.setdefault((kv.n_kv_heads, kv.head_dim, kv.window, kv.v_head_dim, keep, kv.key_scale), []).append(cid)
     full = -(-kv_tokens // block_size)
     groups = []
-    for (nkv, d, window, vd, keep), ids in by_key.items():
+    for (nkv, d, window, vd, keep, scaled), ids in by_key.items():
         n = full
         if window is not None and window_pools == "sized":
             n = min(full, max_sequences * (-(-(window - 1 + max_step_tokens) // block_size) + 2 + -(-keep // block_size)))
-        groups.append(GroupLayout(nkv, d, window, tuple(ids), max(1, n), vd, keep))
+        groups.append(GroupLayout(nkv, d, window, tuple(ids), max(1, n), vd, keep, scaled))
     return groups
 
 
@@ -55,6 +55,7 @@ class CacheView:
     group: int
     state: object  # [max_sequences, ...] this cache's per-request state, or {name: tensor} of several
     slots: Optional[torch.Tensor]  # [requests in the step] int32 slot of each request (a row's is step.seq_of_row)
+    key_scale: Optional[torch.Tensor] = None  # [pages, kv heads, block] 32-bit, where the mixer asked for it
 
 
 class DeviceCache:
@@ -65,7 +66,7 @@ class DeviceCache:
         self.block_size = block_size
         self.max_sequences = max_sequences
         self.table_width = -(-context_length // block_size)
-        self.k, self.v = [], []
+        self.k, self.v, self.key_scale = [], [], []
         self._where = {}
         # page tables live on the device, one row per slot; a step only uploads the entries that changed
         self.tables = [torch.full((max_sequences, self.table_width), -1, dtype=torch.int32, device=runtime.device)
@@ -75,6 +76,7 @@ class DeviceCache:
             self.k.append(torch.zeros(shape, dtype=runtime.dtype, device=runtime.device))
             vd = g.head_dim if g.v_head_dim is None else g.v_head_dim
             self.v.append(torch.zeros(shape[:-1] + (vd,), dtype=runtime.dtype, device=runtime.device) if vd else None)
+            self.key_scale.append(torch.zeros(shape[:-1], dtype=torch.float32, device=runtime.device) if g.key_scale else None)
             for j, cid in enumerate(g.cache_ids):
                 self._where[cid] = (gi, j)
         def make(need):
@@ -92,13 +94,14 @@ class DeviceCache:
             yield from (t.values() if isinstance(t, dict) else (t,))
 
     def bytes(self) -> int:
-        return sum(t.numel() * t.element_size() for t in self.k + self.v if t is not None) + \
+        return sum(t.numel() * t.element_size() for t in self.k + self.v + self.key_scale if t is not None) + \
             sum(t.numel() * t.element_size() for t in self._state_tensors())
 
     def bytes_per_token(self) -> int:
         """Key/value bytes one cached position occupies over all caches."""
-        return sum(len(g.cache_ids) * g.n_kv_heads * self.k[i].element_size()
-                   * (g.head_dim + (g.head_dim if g.v_head_dim is None else g.v_head_dim))
+        return sum(len(g.cache_ids) * g.n_kv_heads
+                   * (self.k[i].element_size() * (g.head_dim + (g.head_dim if g.v_head_dim is None else g.v_head_dim))
+                      + (4 if g.key_scale else 0))
                    for i, g in enumerate(self.groups))
 
     def state_bytes_per_request(self) -> int:
@@ -113,5 +116,5 @@ class DeviceCache:
         if gi is None:
             return CacheView(None, None, None, self.block_size, -1, self.state.get(cache_id), step.slots)
         return CacheView(self.k[gi][j], self.v[gi][j] if self.v[gi] is not None else None, self.tables[gi],
-                         self.block_size, gi,
-                         self.state.get(cache_id), step.slots)
+                         self.block_size, gi, self.state.get(cache_id), step.slots,
+                         self.key_scale[gi][j] if self.key_scale[gi] is not None else None)

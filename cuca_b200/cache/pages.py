@@ -46,6 +46,7 @@ class GroupLayout:
     n_blocks: int
     v_head_dim: Optional[int] = None  # None: values as wide as keys; 0: the group has no value slab
     keep_first: int = 0  # positions at a request's start that stay visible beside the window
+    key_scale: bool = False  # the group has a slab of one 32-bit number per position and key head
 
 
 def _raise(code: int) -> None:

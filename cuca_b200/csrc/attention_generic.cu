@@ -65,6 +65,7 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ 
       const T* kr = kpool + base * d;
       float dot = 0.f;
       for (int i = 0; i < d; ++i) dot = fmaf(qv[i], to_f32(kr[i]), dot);
+      if (opt.key_scale) dot *= opt.key_scale[base];
       s = dot * scale;
       if (softcap > 0.f) s = softcap * tanhf(s / softcap);  // a smooth cap on the score
       if (opt.slopes) s -= slope * (float)(P - kp);
@@ -127,6 +128,7 @@ CUCA_API int cuca_attention_generic_o(const void* q, int q_stride, void* out, in
                                       const CucaAttnOptions* opt, int* err, cudaStream_t stream) {
   if (n_rows == 0) return 0;
   CUCA_REQUIRE(opt != nullptr && opt->window >= 0 && opt->keep >= 0, "attention: bad options");
+  CUCA_REQUIRE(!opt->key_scale || (vpool == kpool && dv == d), "attention: keys with factors of their own are the values too");
   CUCA_REQUIRE(d > 0 && d <= cuca_attention_max_head_dim(), "attention: head size %d is outside 1..%d", d, cuca_attention_max_head_dim());
   CUCA_REQUIRE(dv > 0 && dv <= 2 * cuca_attention_max_head_dim(), "attention: value size %d is outside 1..%d", dv,
                2 * cuca_attention_max_head_dim());
@@ -157,7 +159,7 @@ CUCA_API int cuca_attention_generic_sv(const void* q, int q_stride, void* out, i
                                        int table_stride, int n_rows, int nh, int nkv, int d, int dv, float scale,
                                        int window, float softcap, int sink, const float* sink_val, int* err,
                                        cudaStream_t stream) {
-  const CucaAttnOptions opt{scale, window, 0, softcap, sink, 0, sink_val, nullptr, nullptr};
+  const CucaAttnOptions opt{scale, window, 0, softcap, sink, 0, sink_val, nullptr, nullptr, nullptr};
   return cuca_attention_generic_o(q, q_stride, out, out_stride, dtype, kpool, vpool, n_blocks, bs, positions, seq_of_row,
                                   tables, table_stride, n_rows, nh, nkv, d, dv, &opt, err, stream);
 }
@@ -296,7 +298,8 @@ CUCA_API int cuca_rope_store_general(void* qkv, int dtype, int ld, int k_col, in
 // qt_every > 0: the query of a row at position p is multiplied by 1 + qt_coef ln(floor((p + 1) / qt_every) + 1), after
 // norm and rotation.
 // unit != 0: the norms per head without a weight (q_norm and k_norm null). q_mul [nh]: a factor on every query of a head,
-// after the norm. v_col may be k_col: the values are then the keys as projected.
+// after the norm. v_col may be k_col: the values are then the keys as projected. key_scale (with unit): the page row of a key
+// holds the key as projected and key_scale the factor its norm would have been; there are no value rows.
 namespace {
 template <typename T, typename TP>
 __global__ void __launch_bounds__(256)
@@ -307,7 +310,7 @@ norm_rope_store_kernel(T* __restrict__ qkv, int ld, int k_col, int v_col, TP* __
                        const float* __restrict__ q_norm, const float* __restrict__ k_norm, int v_norm, float eps,
                        TP* __restrict__ kpool, TP* __restrict__ vpool, int n_blocks, int bs, int nh, int nkv, int d, int dv,
                        int v_split, int dv_src, int whole, float qt_coef, int qt_every, int unit,
-                       const float* __restrict__ q_mul_head, int* err) {
+                       const float* __restrict__ q_mul_head, float* __restrict__ key_scale, int* err) {
   __shared__ float red[2][8];
   pdl_trigger();
   pdl_wait();
@@ -347,7 +350,7 @@ norm_rope_store_kernel(T* __restrict__ qkv, int ld, int k_col, int v_col, TP* __
   const float* cr = cos_t + (size_t)(in_table ? pos : 0) * half;
   const float* sr = sin_t + (size_t)(in_table ? pos : 0) * half;
   const long long slab_rows = (long long)n_blocks * nkv * bs;
-  for (int head = warp; head < nh + 2 * nkv; head += n_warps) {
+  for (int head = warp; head < nh + (key_scale ? 1 : 2) * nkv; head += n_warps) {
     const int kind = head < nh ? 0 : (head < nh + nkv ? 1 : 2);  // q, k, v
     if (kind != 0 && page_row < 0) continue;
     const int hh = kind == 0 ? head : (kind == 1 ? head - nh : head - nh - nkv);
@@ -364,6 +367,10 @@ norm_rope_store_kernel(T* __restrict__ qkv, int ld, int k_col, int v_col, TP* __
       inv = 1.f / sqrtf(warp_sum(ss) / (float)n + eps);
     }
     __syncwarp();  // every lane has read the head before any lane rewrites it
+    if (key_scale && kind == 1) {
+      if (lane == 0) key_scale[page_row + (long long)hh * bs] = inv;
+      inv = 1.f;
+    }
     if (kind == 2) {
       const int ds = dv / v_split;
       for (int e = lane; e < dv; e += 32)
@@ -400,19 +407,18 @@ __global__ void __launch_bounds__(256)
 norm_store_kernel(__nv_bfloat16* __restrict__ qkv, int ld, int k_col, int v_col, const int* __restrict__ positions,
                   const int* __restrict__ seq_of_row, const int* __restrict__ tables, int table_stride,
                   const float* __restrict__ q_norm, const float* __restrict__ k_norm, int v_norm, float eps,
-                  __nv_bfloat16* __restrict__ kpool, __nv_bfloat16* __restrict__ vpool, int n_blocks, int bs, int n_rows,
+                  __nv_bfloat16* __restrict__ kpool, __nv_bfloat16* __restrict__ vpool, int n_blocks, int bs,
                   int nh, int nkv, int d, int group, float qt_coef, int qt_every, int unit,
-                  const float* __restrict__ q_mul_head, int* err) {
+                  const float* __restrict__ q_mul_head, float* __restrict__ key_scale, int* err) {
   pdl_trigger();
   pdl_wait();
   const int heads = nh + nkv * (v_col == k_col ? 1 : 2);
-  const long long item = ((long long)blockIdx.x * blockDim.x + threadIdx.x) / group;
-  const int row = (int)(item / heads), head = (int)(item % heads), c = (threadIdx.x % group) * 8;
-  const int seq = row < n_rows ? seq_of_row[row] : -1;
-  const bool active = seq >= 0 && c < d;  // (the shuffles below are the whole warp's)
+  const int row = blockIdx.x, head = (blockIdx.y * blockDim.x + threadIdx.x) / group, c = (threadIdx.x & (group - 1)) * 8;
+  const int seq = seq_of_row[row];
+  const bool active = seq >= 0 && head < heads && c < d;  // (the shuffles below are the whole warp's)
   const int kind = head < nh ? 0 : (head < nh + nkv ? 1 : 2);  // q, k, v
   const int hh = kind == 0 ? head : (kind == 1 ? head - nh : head - nh - nkv);
-  __nv_bfloat16* src = qkv + (size_t)(row < n_rows ? row : 0) * ld + (kind == 0 ? 0 : (kind == 1 ? k_col : v_col)) + (size_t)hh * d + c;
+  __nv_bfloat16* src = qkv + (size_t)row * ld + (kind == 0 ? 0 : (kind == 1 ? k_col : v_col)) + (size_t)hh * d + c;
   const int pos = seq >= 0 ? positions[row] : 0;
   uint4 raw = make_uint4(0, 0, 0, 0);
   if (active) raw = *reinterpret_cast<const uint4*>(src);
@@ -444,6 +450,11 @@ norm_store_kernel(__nv_bfloat16* __restrict__ qkv, int ld, int k_col, int v_col,
     return;
   }
   const size_t at = (((size_t)blk * nkv + hh) * bs + pos % bs) * d + c;
+  if (kind == 1 && key_scale) {  // the key as projected, and its factor
+    *reinterpret_cast<uint4*>(kpool + at) = raw;
+    if (c == 0) key_scale[((size_t)blk * nkv + hh) * bs + pos % bs] = mul;
+    return;
+  }
   if (kind == 1) *reinterpret_cast<uint4*>(kpool + at) = res;
   if (kind == 2) *reinterpret_cast<uint4*>(vpool + at) = res;
   if (kind == 1 && v_col == k_col) {
@@ -466,8 +477,11 @@ CUCA_API int cuca_norm_rope_store_u(void* qkv, int dtype, int ld, int k_col, int
                                     const float* q_norm, const float* k_norm, int v_norm, float eps, void* kpool,
                                     void* vpool, int n_blocks, int bs, int n_rows, int nh, int nkv, int d, int dv,
                                     int v_split, int dv_src, int whole, float qt_coef, int qt_every, int unit,
-                                    const float* q_mul, int* err, cudaStream_t stream) {
+                                    const float* q_mul, float* key_scale, int* err, cudaStream_t stream) {
   if (n_rows == 0) return 0;
+  CUCA_REQUIRE(!key_scale || (unit && rot == 0 && !v_norm && v_col == k_col),
+               "norm_rope_store: factors of keys are for norms without a weight, keys without rotation and values that are the keys");
+  CUCA_REQUIRE(nkv == 0 || (kpool && (vpool || key_scale)), "norm_rope_store: no pool to store into");
   CUCA_REQUIRE(!unit || (!whole && !q_norm && !k_norm), "norm_rope_store: a norm without a weight is given none");
   CUCA_REQUIRE(!whole || (q_norm && (nkv == 0 || k_norm) && !v_norm),
                "norm_rope_store: a norm over the whole projection needs both weights and takes no value norm");
@@ -481,11 +495,12 @@ CUCA_API int cuca_norm_rope_store_u(void* qkv, int dtype, int ld, int k_col, int
       dv == d && dv_src == d && v_split == 1 && ld % 8 == 0 && k_col % 8 == 0 && v_col % 8 == 0 && aligned) {
     int group = 1;
     while (group * 8 < d) group *= 2;
-    const long long lanes = (long long)n_rows * (nh + nkv * (v_col == k_col ? 1 : 2)) * group;
-    cuca_launch(norm_store_kernel, dim3((unsigned)((lanes + 255) / 256)), dim3(256), 0, stream, true, (__nv_bfloat16*)qkv, ld,
+    const int lanes = (nh + nkv * (v_col == k_col ? 1 : 2)) * group;
+    const int threads = lanes < 256 ? (lanes + 31) / 32 * 32 : 256;
+    cuca_launch(norm_store_kernel, dim3(n_rows, (lanes + threads - 1) / threads), dim3(threads), 0, stream, true, (__nv_bfloat16*)qkv, ld,
                 k_col, v_col, positions, seq_of_row, tables, table_stride, q_norm, k_norm, v_norm, eps,
-                (__nv_bfloat16*)kpool, (__nv_bfloat16*)vpool, n_blocks, bs, n_rows, nh, nkv, d, group, qt_coef, qt_every,
-                unit, q_mul, err);
+                (__nv_bfloat16*)kpool, (__nv_bfloat16*)vpool, n_blocks, bs, nh, nkv, d, group, qt_coef, qt_every, unit,
+                q_mul, key_scale, err);
     CUCA_CHECK_LAUNCH("norm_store");
     return 0;
   }
@@ -493,7 +508,7 @@ CUCA_API int cuca_norm_rope_store_u(void* qkv, int dtype, int ld, int k_col, int
   cuca_launch(norm_rope_store_kernel<T, TP>, dim3(n_rows), dim3(256), 0, stream, true, (T*)qkv, ld, k_col, v_col,      \
               (TP*)q_out, positions, seq_of_row, tables, table_stride, cos_t, sin_t, table_rows, rot, pairs, q_norm,   \
               k_norm, v_norm, eps, (TP*)kpool, (TP*)vpool, n_blocks, bs, nh, nkv, d, dv, v_split, dv_src, whole,       \
-              qt_coef, qt_every, unit, q_mul, err)
+              qt_coef, qt_every, unit, q_mul, key_scale, err)
   if (dtype == CUCA_F32 && pool_dtype == CUCA_F32) NRS(float, float);
   else if (dtype == CUCA_BF16 && pool_dtype == CUCA_BF16) NRS(__nv_bfloat16, __nv_bfloat16);
   else if (dtype == CUCA_F32 && pool_dtype == CUCA_BF16) {
@@ -515,7 +530,7 @@ CUCA_API int cuca_norm_rope_store_w(void* qkv, int dtype, int ld, int k_col, int
   return cuca_norm_rope_store_u(qkv, dtype, ld, k_col, v_col, q_out, pool_dtype, positions, seq_of_row, tables,
                                 table_stride, cos_t, sin_t, table_rows, rot, pairs, q_norm, k_norm, v_norm, eps, kpool,
                                 vpool, n_blocks, bs, n_rows, nh, nkv, d, dv, v_split, dv_src, whole, qt_coef, qt_every, 0,
-                                nullptr, err, stream);
+                                nullptr, nullptr, err, stream);
 }
 
 CUCA_API int cuca_norm_rope_store(void* qkv, int dtype, int ld, int k_col, int v_col, void* q_out, int pool_dtype,

@@ -55,6 +55,7 @@ struct AttnParams {
   const float* slopes;   // distance bias per query head (null: none): slopes[head] (P - key) is taken off a score
   const __nv_bfloat16* gate;  // with it the result is multiplied by sigmoid(gate[row][head D + dim])
   int gate_stride;
+  float* key_scale;      // [pages][nkv][bs]: values that are the keys (see CucaAttnOptions), or null
   int chunk;             // decode: key positions per split (multiple of 64); 0: each row divides its own length
   int slots;             // decode, chunk 0: CTAs the GPU holds at once (for the choice of chunks per row)
   float* part;           // decode: [rows][nh][splits][D + 2] partial (acc, m, l)
@@ -126,11 +127,13 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
   return *reinterpret_cast<uint32_t*>(&v);
 }
 
-template <int D>
+// SHARED: the values are the keys: one tile serves both contractions, and every key has a 32-bit factor on its scores
+template <int D, bool SHARED>
 struct Smem {
+  static constexpr int KV = SHARED ? 1 : 2;  // tiles of a stage
   static constexpr int RS = D + 8;  // row stride in elements: 16 bytes of padding
   static constexpr int TILE_ELEMS = TILE * RS;
-  static constexpr int BYTES = STAGES * 2 /*k, v*/ * TILE_ELEMS * 2;
+  static constexpr int BYTES = STAGES * KV * TILE_ELEMS * 2;
   // fused form: the 16 query rows, then the new key and the new value of the row
   static constexpr int Q_ELEMS = 16 * RS;
   static constexpr int FUSED_BYTES = BYTES + (Q_ELEMS + 2 * D) * 2;
@@ -138,10 +141,11 @@ struct Smem {
   // 64-wide halves of 16 rows x 128 bytes, 128-byte swizzled: K half 0, K half 1, ..., V half 0, ...
   static constexpr int HALVES = D / 64;
   static constexpr int SUB_BYTES = 16 * 128;
-  static constexpr int WSTAGE_BYTES = 2 * (HALVES > 0 ? HALVES : 1) * SUB_BYTES;
-  static constexpr int WSTAGES = 3;
+  static constexpr int WSTAGE_BYTES = KV * (HALVES > 0 ? HALVES : 1) * SUB_BYTES;
+  static constexpr int WSTAGES = SHARED ? 4 : 3;
+  static constexpr int FACTOR_BYTES = SHARED ? 16 * 4 : 0;  // of a stage's keys
   static constexpr int RING_BYTES = 4 * WSTAGES * WSTAGE_BYTES;
-  static constexpr int TMA_BYTES = RING_BYTES + 1024 /*alignment*/ + (Q_ELEMS + 2 * D) * 2;
+  static constexpr int TMA_BYTES = RING_BYTES + 1024 /*alignment*/ + (Q_ELEMS + 2 * D) * 2 + 4 * WSTAGES * FACTOR_BYTES;
 };
 
 // One warp's state over its 16 MMA rows: thread (g, t) holds rows g and g + 8.
@@ -165,14 +169,15 @@ __device__ __forceinline__ float sink_term(float m, const AttnParams& p, int hea
 }
 
 // FUSED: 1: decode fed by the projection's K slices, with rotation; 2: with unit norms per head instead (and an output gate)
-template <int D, bool DECODE, int FUSED, bool TMA>
+template <int D, bool DECODE, int FUSED, bool TMA, bool SHARED>
 __global__ void __launch_bounds__(NTHREADS)
 attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV) {
   static_assert(!FUSED || DECODE, "only the decode form takes the projection's K slices");
   static_assert(!TMA || (DECODE && D % 64 == 0), "the TMA form is for decode with head sizes 64 and 128");
   extern __shared__ __align__(16) uint8_t smem_raw[];
   __nv_bfloat16* smem = reinterpret_cast<__nv_bfloat16*>(smem_raw);
-  using S = Smem<D>;
+  static_assert(!SHARED || FUSED != 1, "rotated keys are not values");
+  using S = Smem<D, SHARED>;
   uint8_t* ring_base = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
   const int G = p.nh / p.nkv;
@@ -306,6 +311,9 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
   // Row offsets of a tile's 64 keys in the pools (-1: masked or without a page), one tile ahead of the copies:
   // the page-table lookups of tile i + 2 are in flight while tile i is computed, so no copy waits on one.
   __shared__ long long s_rowoff[STAGES][TILE];
+  // SHARED: the keys' factors (one slot more, since a slot is filled while the tile STAGES before may still be in use), and
+  // that of the row's own key
+  __shared__ float s_factor[SHARED && !TMA ? STAGES + 1 : 1][TILE], s_own_factor;
   const int bs_shift = __ffs(p.bs) - 1, bs_mask = p.bs - 1;
   // fused form: the CTA whose keys include the row's own position makes that key and value itself
   const bool owner = FUSED && p.has_kv && has_own;
@@ -320,8 +328,9 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
     }
     return ((((long long)blk * p.nkv + kvh) << bs_shift) + (kp & bs_mask)) * D;
   };
+  auto factor_at = [&](long long off) { return SHARED && off >= 0 ? __ldcg(p.key_scale + off / D) : 0.f; };
   auto load_tile = [&](int stage, int tile_index) {
-    __nv_bfloat16* ks = smem + (size_t)stage * 2 * S::TILE_ELEMS;
+    __nv_bfloat16* ks = smem + (size_t)stage * S::KV * S::TILE_ELEMS;
     __nv_bfloat16* vs = ks + S::TILE_ELEMS;
     const long long* ro = s_rowoff[tile_index % STAGES];
     constexpr int CH = D / 8;  // 16-byte chunks per row
@@ -332,7 +341,7 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
       bool valid = off >= 0;
       size_t o = valid ? (size_t)off + ch * 8 : 0;
       cp_async16(smem_u32(ks + key * S::RS + ch * 8), p.kpool + o, valid);
-      cp_async16(smem_u32(vs + key * S::RS + ch * 8), p.vpool + o, valid);
+      if (!SHARED) cp_async16(smem_u32(vs + key * S::RS + ch * 8), p.vpool + o, valid);
     }
   };
   // ---- TMA form: this warp's 16-key groups are (tile ti, keys 16 warp .. 16 warp + 15) for ti in [ti_lo, ti_hi)
@@ -340,6 +349,8 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
   __shared__ int w_abort;
   int ti_lo = 0, n_mine = 0, next_page = -1;
   uint8_t* ring = ring_base + (size_t)warp * S::WSTAGES * S::WSTAGE_BYTES;
+  // (behind the query rows and the row's own key and value)
+  float* factors = reinterpret_cast<float*>(ring_base + S::RING_BYTES + (S::Q_ELEMS + 2 * D) * 2) + warp * S::WSTAGES * 16;
   auto group_kp0 = [&](int j) { return tile_key0(ti_lo + j) + warp * 16; };
   auto group_seen = [&](int kp0) { return kp0 < range_hi && (kp0 + 16 > range_lo || kp0 < p.keep); };
   auto page_of = [&](int j) { return table[group_kp0(j) >> bs_shift]; };
@@ -353,9 +364,10 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
     const int row = ((page * p.nkv + kvh) << bs_shift) + (kp0 & bs_mask);
     const int st = j % S::WSTAGES;
     uint8_t* dst = ring + (size_t)st * S::WSTAGE_BYTES;
-    if (lane == 0) mbar_expect_tx(&w_full[warp][st], S::WSTAGE_BYTES);
+    if (lane == 0) mbar_expect_tx(&w_full[warp][st], S::WSTAGE_BYTES + S::FACTOR_BYTES);
     __syncwarp();
-    if (lane < 2 * S::HALVES) {
+    if (SHARED && lane == S::HALVES) bulk_load(factors + st * 16, p.key_scale + row, &w_full[warp][st], S::FACTOR_BYTES);
+    if (lane < S::KV * S::HALVES) {
       const int h = lane % S::HALVES;
       const bool values = lane >= S::HALVES;
       tma_load_2d(dst + lane * S::SUB_BYTES, values ? &tmV : &tmK, &w_full[warp][st], 64 * h, row);
@@ -377,7 +389,7 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
   const int f_rope_items = f_unit ? 0 : (G + (owner ? 1 : 0)) * f_hq;
   // (with unit norms an item is four columns of a head: the q heads, the row's own key and, if it has columns of its own,
   // the row's own value)
-  const int f_items = f_unit ? (G + (owner ? (p.v_col == p.nh * D ? 1 : 2) : 0)) * (D / 4)
+  const int f_items = f_unit ? (G + (owner ? (SHARED ? 1 : 2) : 0)) * (D / 4)
                              : f_rope_items + (owner ? D / 4 : 0);  // then the row's own value
   // columns of item `it`: ca (and ca + half for a rotated head); head index hh (G: the key), offset inside the head
   auto f_item = [&](int it, int& ca, int& hh, int& off) {
@@ -447,7 +459,11 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
     if (threadIdx.x < TILE) {
 #pragma unroll
       for (int i = 0; i < STAGES; ++i)
-        if (i < n_tiles) s_rowoff[i][threadIdx.x] = row_offset(i);
+        if (i < n_tiles) {
+          const long long off = row_offset(i);
+          s_rowoff[i][threadIdx.x] = off;
+          if (SHARED) s_factor[SHARED && !TMA ? i : 0][threadIdx.x] = factor_at(off);
+        }
     }
     __syncthreads();
 #pragma unroll
@@ -489,7 +505,7 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
   float4 gate_r = make_float4(0.f, 0.f, 0.f, 0.f);
   if (f_gated && (int)threadIdx.x < G * (D / 4) && (!p.cluster || n_used == 1 || cluster_rank() == 0)) gate_r = gate4(threadIdx.x);
   __nv_bfloat16* q_s = TMA ? reinterpret_cast<__nv_bfloat16*>(ring_base + S::RING_BYTES)
-                           : smem + (size_t)STAGES * 2 * S::TILE_ELEMS;  // [16][RS]: the group's rotated query heads
+                           : smem + (size_t)STAGES * S::KV * S::TILE_ELEMS;  // [16][RS]: the group's rotated query heads
   __nv_bfloat16* k_new = q_s + S::Q_ELEMS;                          // [D] rotated key of the row's own position
   __nv_bfloat16* v_new = k_new + D;                                 // [D] its value
   if (FUSED) {
@@ -528,8 +544,10 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
         if (hh < G) {
           put4(q_s + hh * S::RS + off, a, inv * (p.q_mul ? p.q_mul[kvh * G + hh] : 1.f));
         } else {
-          if (hh == G) put4(k_new + off, a, inv);
-          if (hh > G || p.v_col == p.nh * D) put4(v_new + off, a, 1.f);
+          // (a key that is the value too stays as projected, its norm becomes its factor)
+          if (hh == G) put4(k_new + off, a, SHARED ? 1.f : inv);
+          if (SHARED && off == 0) s_own_factor = inv;
+          if (hh > G) put4(v_new + off, a, 1.f);
         }
       }
     }
@@ -616,7 +634,8 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
         if (threadIdx.x == 0 && p.err) atomicExch(p.err, CUCA_ERR_BLOCK_RANGE);
       } else {
         const size_t off = ((((size_t)blk * p.nkv + kvh) << bs_shift) + (P & bs_mask)) * D;
-        for (int i = threadIdx.x; i < 2 * (D / 8); i += NTHREADS) {
+        if (SHARED && threadIdx.x == 0) p.key_scale[off / D] = s_own_factor;
+        for (int i = threadIdx.x; i < S::KV * (D / 8); i += NTHREADS) {
           const int which = i / (D / 8), ch = i % (D / 8);
           __nv_bfloat16* pool = const_cast<__nv_bfloat16*>(which ? p.vpool : p.kpool);
           *reinterpret_cast<uint4*>(pool + off + ch * 8) = *reinterpret_cast<const uint4*>((which ? v_new : k_new) + ch * 8);
@@ -631,7 +650,8 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
   constexpr int NT = 2 * SUBS;                    // 8-key n-tiles per update
   // One update with the keys [kp0, kp0 + 16 SUBS): kaddr / vaddr give the shared-memory address of (key, dim),
   // `key` counted from key0 within what they address.
-  auto update = [&](auto kaddr, auto vaddr, const int kp0, const int key0) {
+  // `factor` (SHARED): the factors of those keys.
+  auto update = [&](auto kaddr, auto vaddr, const int kp0, const int key0, const float* factor) {
     // ---- S = Q K^T
     float s[NT][4];
 #pragma unroll
@@ -663,7 +683,7 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
 #pragma unroll
       for (int nt = 0; nt < NT; ++nt)
 #pragma unroll
-        for (int e = 0; e < 2; ++e) s[nt][2 * h + e] = score_log2(s[nt][2 * h + e], p);
+        for (int e = 0; e < 2; ++e) s[nt][2 * h + e] = score_log2(SHARED ? s[nt][2 * h + e] * factor[nt * 8 + 2 * t + e] : s[nt][2 * h + e], p);
       if (p.slopes) {
         const float d0 = (float)(row_pos[h] - kp0 - 2 * t);  // the distance of the thread's first key
 #pragma unroll
@@ -743,7 +763,7 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
       ok = __all_sync(0xffffffffu, ok);
       if (!ok) break;
       const uint32_t kbase = smem_u32(ring + (size_t)st_i * S::WSTAGE_BYTES);
-      const uint32_t vbase = kbase + S::HALVES * S::SUB_BYTES;
+      const uint32_t vbase = SHARED ? kbase : kbase + S::HALVES * S::SUB_BYTES;
       // (key, dim) in a swizzled half: row `key` of 128 bytes, 16-byte chunk (dim % 64) / 8 XOR (key % 8)
       auto sw = [](uint32_t base, int key, int dim) {
         return base + (uint32_t)((dim >> 6) * S::SUB_BYTES + key * 128 + ((((dim & 63) >> 3) ^ (key & 7)) << 4));
@@ -752,7 +772,8 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
       if (owner && P >= kp0 && P < kp0 + 16) {
         // the row's own key and value take their place among the warp's keys (the page's row is stale)
         const int key = P - kp0;
-        for (int c = lane; c < 2 * (D / 8); c += 32) {
+        if (SHARED && lane == 0) factors[st_i * 16 + key] = s_own_factor;
+        for (int c = lane; c < S::KV * (D / 8); c += 32) {
           const int which = c / (D / 8), ch = c % (D / 8);
           const uint4 val = *reinterpret_cast<const uint4*>((which ? v_new : k_new) + ch * 8);
           const uint32_t dst = sw(which ? vbase : kbase, key, ch * 8);
@@ -761,7 +782,7 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
         __syncwarp();
       }
       update([&](int key, int dim) { return sw(kbase, key, dim); }, [&](int key, int dim) { return sw(vbase, key, dim); },
-             kp0, 0);
+             kp0, 0, factors + st_i * 16);
       __syncwarp();  // every lane has read the stage before lane 0 asks for the next group into it
     }
     if (w_abort) {
@@ -779,13 +800,16 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
       long long next_off = -1;
       const bool look_ahead = threadIdx.x < TILE && ti + STAGES < n_tiles;
       if (look_ahead) next_off = row_offset(ti + STAGES);
+      const float next_factor = factor_at(next_off);
+      float* tile_factor = s_factor[SHARED && !TMA ? ti % (STAGES + 1) : 0];
       const int start = tile_key0(ti);
-      const __nv_bfloat16* ks = smem + (size_t)stage * 2 * S::TILE_ELEMS;
-      const __nv_bfloat16* vs = ks + S::TILE_ELEMS;
+      const __nv_bfloat16* ks = smem + (size_t)stage * S::KV * S::TILE_ELEMS;
+      const __nv_bfloat16* vs = SHARED ? ks : ks + S::TILE_ELEMS;
       if (owner && P >= start && P < start + TILE) {
         // the row's own key and value take their place in the tile (the copy left zeros there)
         const int key = P - start;
-        for (int i = threadIdx.x; i < 2 * (D / 8); i += NTHREADS) {
+        if (SHARED && threadIdx.x == 0) tile_factor[key] = s_own_factor;
+        for (int i = threadIdx.x; i < S::KV * (D / 8); i += NTHREADS) {
           const int which = i / (D / 8), ch = i % (D / 8);
           __nv_bfloat16* dst = const_cast<__nv_bfloat16*>(which ? vs : ks) + key * S::RS + ch * 8;
           *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<const uint4*>((which ? v_new : k_new) + ch * 8);
@@ -798,8 +822,12 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
       if (!DECODE && kp0 > warp_pmax) active = false;  // every row of this warp lies before these keys (causal)
       if (active)
         update([&](int key, int dim) { return smem_u32(ks + key * S::RS + dim); },
-               [&](int key, int dim) { return smem_u32(vs + key * S::RS + dim); }, kp0, sub0 * 16);
-      if (look_ahead) s_rowoff[ti % STAGES][threadIdx.x] = next_off;  // this slot was last read to request tile ti
+               [&](int key, int dim) { return smem_u32(vs + key * S::RS + dim); }, kp0, sub0 * 16,
+               tile_factor + sub0 * 16);
+      if (look_ahead) {
+        s_rowoff[ti % STAGES][threadIdx.x] = next_off;  // this slot was last read to request tile ti
+        if (SHARED) s_factor[SHARED && !TMA ? (ti + STAGES) % (STAGES + 1) : 0][threadIdx.x] = next_factor;
+      }
       __syncthreads();  // the stage is overwritten by the load issued in the next iteration
     }
     cp_async_wait<0>();
@@ -1017,9 +1045,10 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
   if (threadIdx.x == 0) p.counters[blockIdx.z * p.nkv + kvh] = 0;
 }
 
-template <int D, bool DECODE, int FUSED, bool TMA>
+template <int D, bool DECODE, int FUSED, bool TMA, bool SHARED>
 int launch(const AttnParams& p, const CUtensorMap& tmK, const CUtensorMap& tmV, dim3 grid, cudaStream_t stream) {
-  int smem = TMA ? Smem<D>::TMA_BYTES : FUSED ? Smem<D>::FUSED_BYTES : Smem<D>::BYTES;
+  using S = Smem<D, SHARED>;
+  int smem = TMA ? S::TMA_BYTES : FUSED ? S::FUSED_BYTES : S::BYTES;
   if (DECODE) {
     // four warps' results, then the CTA's, then the output gate
     int need = (5 * 16 * (D + 2) + (FUSED == 2 ? 16 * D : 0)) * (int)sizeof(float) + (TMA ? 1024 : 0);
@@ -1027,7 +1056,7 @@ int launch(const AttnParams& p, const CUtensorMap& tmK, const CUtensorMap& tmV, 
   }
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(attn_mma_kernel<D, DECODE, FUSED, TMA>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    cudaError_t e = cudaFuncSetAttribute(attn_mma_kernel<D, DECODE, FUSED, TMA, SHARED>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) {
       cuca_set_error("attention: cannot reserve %d bytes of shared memory: %s", smem, cudaGetErrorString(e));
       return 2;
@@ -1035,16 +1064,16 @@ int launch(const AttnParams& p, const CUtensorMap& tmK, const CUtensorMap& tmV, 
     configured = true;
   }
   if (DECODE && p.cluster)
-    cuca_launch_cluster(attn_mma_kernel<D, DECODE, FUSED, TMA>, grid, dim3(NTHREADS), smem, stream, true, grid.x, p, tmK, tmV);
+    cuca_launch_cluster(attn_mma_kernel<D, DECODE, FUSED, TMA, SHARED>, grid, dim3(NTHREADS), smem, stream, true, grid.x, p, tmK, tmV);
   else
-    cuca_launch(attn_mma_kernel<D, DECODE, FUSED, TMA>, grid, dim3(NTHREADS), smem, stream, true, p, tmK, tmV);
+    cuca_launch(attn_mma_kernel<D, DECODE, FUSED, TMA, SHARED>, grid, dim3(NTHREADS), smem, stream, true, p, tmK, tmV);
   CUCA_CHECK_LAUNCH("attention_mma");
   return 0;
 }
 
 // tma: key/value groups by TMA (decode, head sizes 64 and 128, pages of at least 16 positions)
-template <bool DECODE, int FUSED = 0>
-int dispatch(int d, const AttnParams& p, dim3 grid, cudaStream_t stream, bool tma = false) {
+template <bool DECODE, int FUSED, bool SHARED>
+int dispatch_as(int d, const AttnParams& p, dim3 grid, cudaStream_t stream, bool tma) {
   CUtensorMap tmK, tmV;
   memset(&tmK, 0, sizeof(tmK));
   memset(&tmV, 0, sizeof(tmV));
@@ -1054,25 +1083,37 @@ int dispatch(int d, const AttnParams& p, dim3 grid, cudaStream_t stream, bool tm
       tma = false;
   }
   if constexpr (DECODE) {
-    if (tma && d == 64) return launch<64, true, FUSED, true>(p, tmK, tmV, grid, stream);
-    if (tma && d == 128) return launch<128, true, FUSED, true>(p, tmK, tmV, grid, stream);
+    if (tma && d == 64) return launch<64, true, FUSED, true, SHARED>(p, tmK, tmV, grid, stream);
+    if (tma && d == 128) return launch<128, true, FUSED, true, SHARED>(p, tmK, tmV, grid, stream);
   }
   switch (d) {
-    case 16: return launch<16, DECODE, FUSED, false>(p, tmK, tmV, grid, stream);
-    case 32: return launch<32, DECODE, FUSED, false>(p, tmK, tmV, grid, stream);
-    case 64: return launch<64, DECODE, FUSED, false>(p, tmK, tmV, grid, stream);
-    case 128: return launch<128, DECODE, FUSED, false>(p, tmK, tmV, grid, stream);
+    case 16: return launch<16, DECODE, FUSED, false, SHARED>(p, tmK, tmV, grid, stream);
+    case 32: return launch<32, DECODE, FUSED, false, SHARED>(p, tmK, tmV, grid, stream);
+    case 64: return launch<64, DECODE, FUSED, false, SHARED>(p, tmK, tmV, grid, stream);
+    case 128: return launch<128, DECODE, FUSED, false, SHARED>(p, tmK, tmV, grid, stream);
   }
   if constexpr (FUSED != 2) {  // (whose heads are a power of two lanes wide)
     switch (d) {
-      case 48: return launch<48, DECODE, FUSED, false>(p, tmK, tmV, grid, stream);
-      case 80: return launch<80, DECODE, FUSED, false>(p, tmK, tmV, grid, stream);
-      case 96: return launch<96, DECODE, FUSED, false>(p, tmK, tmV, grid, stream);
-      case 112: return launch<112, DECODE, FUSED, false>(p, tmK, tmV, grid, stream);
+      case 48: return launch<48, DECODE, FUSED, false, SHARED>(p, tmK, tmV, grid, stream);
+      case 80: return launch<80, DECODE, FUSED, false, SHARED>(p, tmK, tmV, grid, stream);
+      case 96: return launch<96, DECODE, FUSED, false, SHARED>(p, tmK, tmV, grid, stream);
+      case 112: return launch<112, DECODE, FUSED, false, SHARED>(p, tmK, tmV, grid, stream);
     }
   }
   cuca_set_error("attention_mma: head size %d is not one of 16, 32, ..., 128", d);
   return 1;
+}
+
+template <bool DECODE, int FUSED = 0>
+int dispatch(int d, const AttnParams& p, dim3 grid, cudaStream_t stream, bool tma = false) {
+  CUCA_REQUIRE(!p.key_scale || p.vpool == p.kpool, "attention: keys with factors of their own are the values too");
+  if constexpr (FUSED == 1) {
+    CUCA_REQUIRE(!p.key_scale, "attention_decode_fused: rotated keys are not values");
+    return dispatch_as<DECODE, FUSED, false>(d, p, grid, stream, tma);
+  } else {
+    return p.key_scale ? dispatch_as<DECODE, FUSED, true>(d, p, grid, stream, tma)
+                       : dispatch_as<DECODE, FUSED, false>(d, p, grid, stream, tma);
+  }
 }
 
 }  // namespace
@@ -1115,6 +1156,7 @@ void set_score_options(AttnParams& p, const CucaAttnOptions& o) {
   p.slopes = o.slopes;
   p.gate = (const __nv_bfloat16*)o.gate;
   p.gate_stride = o.gate_stride;
+  p.key_scale = o.key_scale;
   p.cap_log2e = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
   p.cap_arg = softcap > 0.f ? 2.f * scale * 1.4426950408889634f / softcap : 0.f;
   p.sink = o.sink ? 1 : 0;
@@ -1159,7 +1201,8 @@ int attention_decode_impl(const void* q, int q_stride, const FusedInput* fused, 
   static int env_tma = -1;
   if (env_tma < 0) { const char* e = getenv("CUCA_ATTN_TMA"); env_tma = e ? atoi(e) : 1; }
   // key/value groups of 16 positions by TMA: a group must lie in one page
-  const bool tma = env_tma && d % 64 == 0 && bs >= 16 && ((uintptr_t)kpool & 15) == 0 && ((uintptr_t)vpool & 15) == 0;
+  const bool tma = env_tma && d % 64 == 0 && bs >= 16 &&
+                   (((uintptr_t)kpool | (uintptr_t)vpool | (uintptr_t)opt.key_scale) & 15) == 0;
   if (!fused) return dispatch<true, 0>(d, p, dim3(n_splits, nkv, n_rows), stream, tma);
   CUCA_REQUIRE(fused->partial && fused->n_slices >= 1, "attention_decode_fused: no projection slices");
   CUCA_REQUIRE(fused->rot >= 0 && fused->rot <= d && fused->rot % 2 == 0,
@@ -1190,7 +1233,7 @@ CUCA_API int cuca_attention_decode(const void* q, int q_stride, void* out, int o
                                    const int* seq_of_row, const int* tables, int table_stride, const int* rows,
                                    int n_rows, int nh, int nkv, int d, float scale, int window, int chunk,
                                    int n_splits, float* part, int* counters, int* err, cudaStream_t stream) {
-  const CucaAttnOptions opt{scale, window, 0, 0.f, 0, 0, nullptr, nullptr, nullptr};
+  const CucaAttnOptions opt{scale, window, 0, 0.f, 0, 0, nullptr, nullptr, nullptr, nullptr};
   return attention_decode_impl(q, q_stride, nullptr, out, out_stride, kpool, vpool, n_blocks, bs, positions,
                                seq_of_row, tables, table_stride, rows, n_rows, nh, nkv, d, opt, chunk, n_splits, part,
                                counters, err, stream);
@@ -1217,7 +1260,7 @@ CUCA_API int cuca_attention_decode_sv(const void* q, int q_stride, void* out, in
                                       int n_rows, int nh, int nkv, int d, float scale, int window, float softcap,
                                       int sink, const float* sink_val, int chunk, int n_splits, float* part,
                                       int* counters, int* err, cudaStream_t stream) {
-  const CucaAttnOptions opt{scale, window, 0, softcap, sink, 0, sink_val, nullptr, nullptr};
+  const CucaAttnOptions opt{scale, window, 0, softcap, sink, 0, sink_val, nullptr, nullptr, nullptr};
   return attention_decode_impl(q, q_stride, nullptr, out, out_stride, kpool, vpool, n_blocks, bs, positions,
                                seq_of_row, tables, table_stride, rows, n_rows, nh, nkv, d, opt, chunk, n_splits, part,
                                counters, err, stream);
@@ -1248,15 +1291,15 @@ CUCA_API int cuca_attention_decode_fused(const float* partial, int n_slices, siz
                                          int* err, cudaStream_t stream) {
   FusedInput f{partial, n_slices, slice_stride, bias, cos_t, sin_t, table_rows, rot, has_kv,
                (nh + (has_kv ? 2 * nkv : 0)) * d, (nh + nkv) * d};
-  const CucaAttnOptions opt{scale, window, 0, 0.f, 0, 0, nullptr, nullptr, nullptr};
+  const CucaAttnOptions opt{scale, window, 0, 0.f, 0, 0, nullptr, nullptr, nullptr, nullptr};
   return attention_decode_impl(nullptr, 2, &f, out, out_stride, kpool, vpool, n_blocks, bs, positions, seq_of_row,
                                tables, table_stride, rows, n_rows, nh, nkv, d, opt, chunk, n_splits, part, counters, err,
                                stream);
 }
 
 // The same for layers without rotation whose queries and keys are divided by their root mean square per head (no weight):
-// slices of rows of `width` columns, q heads at 0, k heads at nh d, v heads at v_col (nh d: the values are the keys as
-// projected), the pre-activations of an output gate at gate_col (< 0: no gate). q_mul (or null): a factor on the queries of
+// slices of rows of `width` columns, q heads at 0, k heads at nh d, v heads at v_col (with opt->key_scale at nh d: the values
+// are the keys as projected), the pre-activations of an output gate at gate_col (< 0: no gate). q_mul (or null): a factor on the queries of
 // each head. Window, kept first keys, cap, distance bias and sink as `opt` says (its own gate must be null).
 CUCA_API int cuca_attention_decode_fused_unit(const float* partial, int n_slices, size_t slice_stride, const void* bias,
                                               int width, int v_col, int gate_col, float norm_eps, const float* q_mul,
@@ -1267,6 +1310,7 @@ CUCA_API int cuca_attention_decode_fused_unit(const float* partial, int n_slices
                                               int* counters, int* err, cudaStream_t stream) {
   CUCA_REQUIRE(opt != nullptr && opt->gate == nullptr, "attention_decode_fused: bad options");
   CUCA_REQUIRE(v_col >= nh * d && v_col + nkv * d <= width, "attention_decode_fused: values at column %d do not fit rows of %d", v_col, width);
+  CUCA_REQUIRE((opt->key_scale != nullptr) == (v_col == nh * d), "attention_decode_fused: keys that are the values have factors");
   FusedInput f{partial, n_slices, slice_stride, bias, nullptr, nullptr, 0, 0, 1, width, v_col, 1, norm_eps, q_mul, gate_col};
   return attention_decode_impl(nullptr, 2, &f, out, out_stride, kpool, vpool, n_blocks, bs, positions, seq_of_row, tables,
                                table_stride, rows, n_rows, nh, nkv, d, *opt, chunk, n_splits, part, counters, err, stream);
@@ -1305,7 +1349,7 @@ CUCA_API int cuca_attention_prefill_sv(const void* q, int q_stride, void* out, i
                                        const int* tile_row0, const int* tile_nrows, int n_tiles, int nh, int nkv, int d,
                                        float scale, int window, float softcap, int sink, const float* sink_val,
                                        int* err, cudaStream_t stream) {
-  const CucaAttnOptions opt{scale, window, 0, softcap, sink, 0, sink_val, nullptr, nullptr};
+  const CucaAttnOptions opt{scale, window, 0, softcap, sink, 0, sink_val, nullptr, nullptr, nullptr};
   return cuca_attention_prefill_o(q, q_stride, out, out_stride, kpool, vpool, n_blocks, bs, positions, seq_of_row, tables,
                                   table_stride, tile_row0, tile_nrows, n_tiles, nh, nkv, d, &opt, err, stream);
 }

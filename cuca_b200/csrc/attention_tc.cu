@@ -37,13 +37,16 @@ constexpr int BAR_BYTES = 256;                   // mbarriers, the TMEM address,
 constexpr int TMEM_COLS = 512;                   // two S buffers per query tile (4 x 64 columns), O of both (2 x D)
 constexpr int NTHREADS = 64 + NQ * 128 + 32;     // warp 0 TMA, warp 1 MMA of query tile 0, four softmax warps per query
                                                  // tile, last warp MMA of query tile 1
-// What depends on the head size D (64 or 128).
-template <int D>
+// What depends on the head size D (64 or 128). SHARED: the values are the keys: one tile serves both contractions, and every
+// key has a 32-bit factor on its scores.
+template <int D, bool SHARED>
 struct Shape {
   static constexpr int Q_BYTES = (D / 64) * Q_HALF;
   static constexpr int KV_TILE = (D / 64) * KV_HALF;
-  static constexpr int KV_STAGES = D == 128 ? 5 : 8;
-  static constexpr int TILES_BYTES = NQ * Q_BYTES + KV_STAGES * 2 * KV_TILE;   // 224 KB / 192 KB
+  static constexpr int KV_BYTES = (SHARED ? 1 : 2) * KV_TILE;                   // of a stage
+  static constexpr int FACTOR_BYTES = SHARED ? KEYS * 4 : 0;                    // of a stage's keys
+  static constexpr int KV_STAGES = SHARED ? 8 : D == 128 ? 5 : 8;
+  static constexpr int TILES_BYTES = NQ * Q_BYTES + KV_STAGES * (KV_BYTES + FACTOR_BYTES);   // 224 KB / 192 KB, 194 / 98
   static constexpr int DYN_SMEM = TILES_BYTES + BAR_BYTES + 1024;  // + what aligning the tiles to 1024 bytes may cost
 };
 
@@ -70,6 +73,7 @@ struct Params {
   const float* slopes;   // distance bias per query head (null: none): slopes[head] (position - key) is taken off a score
   const __nv_bfloat16* gate;  // with it the result is multiplied by sigmoid(gate[row][head D + dim])
   int gate_stride;
+  const float* key_scale;  // [pages][nkv][bs]: values that are the keys (see CucaAttnOptions), or null
   int* err;
 };
 
@@ -173,17 +177,18 @@ __host__ __device__ constexpr uint32_t instr_desc_b(bool b_mn, int n) {
          ((uint32_t)(128 >> 4) << 24);
 }
 
-template <int D>
+template <int D, bool SHARED>
 __global__ void __launch_bounds__(NTHREADS, 1)
 attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                const __grid_constant__ CUtensorMap tmV, const Params p) {
-  using SH = Shape<D>;
-  constexpr int Q_BYTES = SH::Q_BYTES, KV_TILE = SH::KV_TILE, KV_STAGES = SH::KV_STAGES;
+  using SH = Shape<D, SHARED>;
+  constexpr int Q_BYTES = SH::Q_BYTES, KV_TILE = SH::KV_TILE, KV_BYTES = SH::KV_BYTES, KV_STAGES = SH::KV_STAGES;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   uint8_t* q_s = smem;                                  // NQ Q tiles
-  uint8_t* kv_s = q_s + NQ * Q_BYTES;                   // KV_STAGES x (K tile + V tile)
-  uint64_t* bars = (uint64_t*)(kv_s + KV_STAGES * 2 * KV_TILE);
+  uint8_t* kv_s = q_s + NQ * Q_BYTES;                   // KV_STAGES x (K tile + V tile), or x the one tile of both
+  float* factor_s = (float*)(kv_s + KV_STAGES * KV_BYTES);  // SHARED: KV_STAGES x [KEYS]
+  uint64_t* bars = (uint64_t*)((uint8_t*)factor_s + KV_STAGES * SH::FACTOR_BYTES);
   uint64_t* q_full = bars;
   uint64_t* kv_full = bars + 1;              // [KV_STAGES]
   uint64_t* kv_empty = kv_full + KV_STAGES;  // [KV_STAGES]
@@ -284,15 +289,15 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
       int ok = 1;
       if (lane == 0 && j >= KV_STAGES) ok = mbar_wait(&kv_empty[s], ((j / KV_STAGES) & 1) ^ 1, p.err, abort_flag) ? 1 : 0;
       if (!__shfl_sync(0xffffffffu, ok, 0)) break;
-      uint8_t* ks = kv_s + s * 2 * KV_TILE;
+      uint8_t* ks = kv_s + s * KV_BYTES;
       uint8_t* vs = ks + KV_TILE;
-      if (lane == 0) mbar_expect_tx(&kv_full[s], 2 * KV_TILE);
+      if (lane == 0) mbar_expect_tx(&kv_full[s], KV_BYTES + SH::FACTOR_BYTES);
       __syncwarp();
       // one copy per lane: a page needs four (keys and values, two 64-wide halves each), a tile has up to 8 pages;
       // a single thread would need about as long to issue them as the tensor pipe needs for the tile
       const int pg = lane >> 2, which = lane & 3;
       int blk = __shfl_sync(0xffffffffu, entry, in_batch * pages + (pg < pages ? pg : 0));
-      if (pg < pages && (which & 1) < D / 64) {
+      if (pg < pages && (SHARED ? which < D / 64 || which == 3 : (which & 1) < D / 64)) {
         const int kp = tile_key0(j) + pg * p.bs;
         if (blk < 0 || blk >= p.n_blocks) {
           // keys before the window may have given their page back; they are masked. Anything else is an error.
@@ -300,6 +305,10 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
           blk = 0;
         }
         const int grow = (blk * p.nkv + kvh) * p.bs;  // row of the page in the pool seen as [rows][D]
+        if (SHARED && which == 3) {
+          bulk_load(factor_s + s * KEYS + pg * p.bs, p.key_scale + grow, &kv_full[s], p.bs * 4);
+          continue;
+        }
         uint8_t* dst = ((which & 2) ? vs : ks) + ((which & 1) ? KV_HALF : 0) + pg * p.bs * 128;  // bs rows of 128 B
         tma_load_2d(dst, (which & 2) ? &tmV : &tmK, &kv_full[s], (which & 1) ? 64 : 0, grow);
       }
@@ -321,8 +330,8 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
     uint64_t k_desc[KV_STAGES], v_desc[KV_STAGES];
 #pragma unroll
     for (int st = 0; st < KV_STAGES; ++st) {
-      k_desc[st] = smem_desc(smem_u32(kv_s + st * 2 * KV_TILE));
-      v_desc[st] = desc_mnmajor(smem_u32(kv_s + st * 2 * KV_TILE + KV_TILE), KV_HALF, 1024);
+      k_desc[st] = smem_desc(smem_u32(kv_s + st * KV_BYTES));
+      v_desc[st] = desc_mnmajor(smem_u32(kv_s + st * KV_BYTES + (SHARED ? 0 : KV_TILE)), KV_HALF, 1024);
     }
     auto stage_desc = [&](const uint64_t (&d)[KV_STAGES], int st) {  // registers, not local memory
       uint64_t r = d[0];
@@ -396,12 +405,15 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
     const int row_lo = (p.window > 0 && row_pos - (p.window - 1) > 0) ? row_pos - (p.window - 1) : 0;
     float m = -INFINITY, l = 0.f;
     bool ok = x < nq;
-    const bool biased = p.slopes != nullptr;
-    const float slope2 = (biased && ok) ? p.slopes[head0 + x] * CUCA_LOG2E : 0.f;
+    const bool biased = SHARED || p.slopes != nullptr;  // (scores with something of their own per key)
+    const float slope2 = (p.slopes && ok) ? p.slopes[head0 + x] * CUCA_LOG2E : 0.f;
     for (int j = 0; ok && j < n_tiles; ++j) {
       // the tcgen05.ld/st below are warp-wide: a warp leaves the loop together or not at all
       if (!__all_sync(0xffffffffu, mbar_wait(&s_full[2 * x + (j & 1)], (j >> 1) & 1, p.err, abort_flag))) { ok = false; break; }
       tc_fence_after();
+      // the copies' own barrier (long complete: the scores were made from the tile), for the factors that came with it
+      if (SHARED && !__all_sync(0xffffffffu, mbar_wait(&kv_full[j % KV_STAGES], (j / KV_STAGES) & 1, p.err, abort_flag))) { ok = false; break; }
+      const float* factor = factor_s + (j % KV_STAGES) * KEYS;
       const int key0 = tile_key0(j);
       const bool whole = key0 + KEYS - 1 <= pos0 &&
                          (p.window <= 0 || key0 >= pos0 + ROWS - 1 - (p.window - 1) || key0 + KEYS <= p.keep);
@@ -422,9 +434,10 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
 #pragma unroll
           for (int e = 0; e < 16; ++e) {
             const float2 bias2 = __ffma2_rn(make_float2((float)(c * 32 + 2 * e), (float)(c * 32 + 2 * e + 1)), slope22, c02);
-            const float r0 = __uint_as_float(raw[c][2 * e]), r1 = __uint_as_float(raw[c][2 * e + 1]);
-            const float2 s2 = capped ? __fadd2_rn(make_float2(capped_log2(r0, p.cap_arg, p.cap_log2e), capped_log2(r1, p.cap_arg, p.cap_log2e)), bias2)
-                                     : __ffma2_rn(make_float2(r0, r1), scale2, bias2);
+            float2 r2 = make_float2(__uint_as_float(raw[c][2 * e]), __uint_as_float(raw[c][2 * e + 1]));
+            if (SHARED) r2 = __fmul2_rn(r2, *reinterpret_cast<const float2*>(factor + c * 32 + 2 * e));
+            const float2 s2 = capped ? __fadd2_rn(make_float2(capped_log2(r2.x, p.cap_arg, p.cap_log2e), capped_log2(r2.y, p.cap_arg, p.cap_log2e)), bias2)
+                                     : __ffma2_rn(r2, scale2, bias2);
             raw[c][2 * e] = __float_as_uint(s2.x);
             raw[c][2 * e + 1] = __float_as_uint(s2.y);
           }
@@ -581,19 +594,19 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
 }
 
 // ------------------------------------------------------------------ host side
-template <int D>
+template <int D, bool SHARED>
 int launch_attn_tc(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, const Params& p, int n_tiles,
                    cudaStream_t stream) {
-  const int smem = Shape<D>::DYN_SMEM;
+  const int smem = Shape<D, SHARED>::DYN_SMEM;
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(attn_tc_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    cudaError_t e = cudaFuncSetAttribute(attn_tc_kernel<D, SHARED>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     CUCA_REQUIRE(e == cudaSuccess, "attention_prefill_tc: cannot reserve %d bytes of shared memory: %s", smem,
                  cudaGetErrorString(e));
     configured = true;
   }
   const int grid_x = p.pair_tiles ? (n_tiles + 1) / 2 : n_tiles;
-  cuca_launch(attn_tc_kernel<D>, dim3(grid_x, p.nh / p.heads_per_cta), dim3(NTHREADS), smem, stream, true, tmQ, tmK, tmV, p);
+  cuca_launch(attn_tc_kernel<D, SHARED>, dim3(grid_x, p.nh / p.heads_per_cta), dim3(NTHREADS), smem, stream, true, tmQ, tmK, tmV, p);
   CUCA_CHECK_LAUNCH("attention_prefill_tc");
   return 0;
 }
@@ -643,6 +656,8 @@ CUCA_API int cuca_attention_prefill_tc_o(const void* q, int q_stride, int n_rows
   p.n_blocks = n_blocks; p.bs = bs; p.nh = nh; p.nkv = nkv; p.scale_log2e = scale * 1.4426950408889634f;
   p.window = opt->window; p.keep = opt->window > 0 ? opt->keep : 0; p.slopes = opt->slopes; p.err = err;
   p.gate = (const __nv_bfloat16*)opt->gate; p.gate_stride = opt->gate_stride;
+  p.key_scale = opt->key_scale;
+  CUCA_REQUIRE(!p.key_scale || (vpool == kpool && ((uintptr_t)p.key_scale & 15) == 0), "attention_prefill_tc: keys with factors of their own are the values too");
   p.cap_log2e = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
   p.cap_arg = softcap > 0.f ? 2.f * scale * 1.4426950408889634f / softcap : 0.f;
   p.sink = opt->sink ? 1 : 0;
@@ -655,7 +670,9 @@ CUCA_API int cuca_attention_prefill_tc_o(const void* q, int q_stride, int n_rows
   const int head_ctas = nh / p.heads_per_cta, sms = cuca_device_sms();
   p.pair_tiles = n_tiles >= 2 && (pair_mode == 2 || (pair_mode == 1 && n_tiles * head_ctas > sms &&
                                                      ((n_tiles + 1) / 2) * head_ctas <= sms)) ? 1 : 0;
-  return d == 128 ? launch_attn_tc<128>(tmQ, tmK, tmV, p, n_tiles, stream) : launch_attn_tc<64>(tmQ, tmK, tmV, p, n_tiles, stream);
+  if (p.key_scale)
+    return d == 128 ? launch_attn_tc<128, true>(tmQ, tmK, tmV, p, n_tiles, stream) : launch_attn_tc<64, true>(tmQ, tmK, tmV, p, n_tiles, stream);
+  return d == 128 ? launch_attn_tc<128, false>(tmQ, tmK, tmV, p, n_tiles, stream) : launch_attn_tc<64, false>(tmQ, tmK, tmV, p, n_tiles, stream);
 }
 
 CUCA_API int cuca_attention_prefill_tc_sv(const void* q, int q_stride, int n_rows_total, void* out, int out_stride,
@@ -664,7 +681,7 @@ CUCA_API int cuca_attention_prefill_tc_sv(const void* q, int q_stride, int n_row
                                           int table_stride, const int* tile_row0, const int* tile_nrows, int n_tiles,
                                           int nh, int nkv, int d, float scale, int window, float softcap, int sink,
                                           const float* sink_val, int* err, cudaStream_t stream) {
-  const CucaAttnOptions opt{scale, window, 0, softcap, sink, 0, sink_val, nullptr, nullptr};
+  const CucaAttnOptions opt{scale, window, 0, softcap, sink, 0, sink_val, nullptr, nullptr, nullptr};
   return cuca_attention_prefill_tc_o(q, q_stride, n_rows_total, out, out_stride, kpool, vpool, n_blocks, bs, positions,
                                      seq_of_row, tables, table_stride, tile_row0, tile_nrows, n_tiles, nh, nkv, d, &opt,
                                      err, stream);

@@ -67,6 +67,12 @@ __device__ __forceinline__ void tma_load_2d(void* dst, const CUtensorMap* map, u
       ::"r"(smem_u32(dst)), "l"(map), "r"(smem_u32(bar)), "r"(c0), "r"(c1)
       : "memory");
 }
+// `bytes` consecutive bytes (a multiple of 16, both addresses 16-byte aligned) without a tensor map.
+__device__ __forceinline__ void bulk_load(void* dst, const void* src, uint64_t* bar, uint32_t bytes) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %3, [%2];"
+               ::"r"(smem_u32(dst)), "l"(src), "r"(smem_u32(bar)), "r"(bytes)
+               : "memory");
+}
 // The same with an L2 eviction policy (see l2_evict_first).
 __device__ __forceinline__ void tma_load_2d_hint(void* dst, const CUtensorMap* map, uint64_t* bar, int c0, int c1,
                                                  uint64_t policy) {

@@ -168,7 +168,7 @@ _SIGNATURES = {
     "cuca_attention_decode_fused_unit": [_P, _I, c_size_t, _P, _I, _I, _I, _F, _P, _P, _I, _P, _P, _I, _I, _P, _P, _P, _I,
                                          _P, _I, _I, _I, _I, _P, _I, _I, _P, _P, _P, _P],
     "cuca_norm_rope_store_u": [_P, _I, _I, _I, _I, _P, _I, _P, _P, _P, _I, _P, _P, _I, _I, _I, _P, _P, _I, _F, _P, _P,
-                               _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _P, _P, _P],
+                               _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _P, _P, _P, _P],
     "cuca_gemm_tc_act": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, c_size_t, _P, _I, _I, _P, _P],
     "cuca_activation": [_P, _I, c_size_t, _I, _P],
     "cuca_embed_pos": [_P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _F, _P, _P],

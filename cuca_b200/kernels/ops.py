@@ -169,16 +169,18 @@ class AttentionOptions(ctypes.Structure):
 
     _fields_ = [("scale", ctypes.c_float), ("window", ctypes.c_int), ("keep", ctypes.c_int), ("softcap", ctypes.c_float),
                 ("sink", ctypes.c_int), ("gate_stride", ctypes.c_int), ("sink_val", ctypes.c_void_p),
-                ("slopes", ctypes.c_void_p), ("gate", ctypes.c_void_p)]
+                ("slopes", ctypes.c_void_p), ("gate", ctypes.c_void_p), ("key_scale", ctypes.c_void_p)]
 
 
 def attention_options(n_heads, scale, window=None, softcap=0.0, sink=False, sink_values=None, keep_first=0, slopes=None,
-                      gate=None, gate_width=None) -> AttentionOptions:
+                      gate=None, gate_width=None, key_scale=None) -> AttentionOptions:
     """`window` w: a query sees the last w keys, itself included, and with `keep_first` k the first k of its request as
     well (None: all keys). `softcap` c > 0: a scaled score s becomes c tanh(s / c). `slopes` (32-bit, one per query
     head): slope * distance is taken off a score. `sink`: every row's denominator holds one more exp(0) that has no
     value, or exp(sink_values[head]) (32-bit, one number per query head) when those are given. `gate` ([rows,
-    gate_width], of the output's dtype): the result is multiplied by sigmoid(gate)."""
+    gate_width], of the output's dtype): the result is multiplied by sigmoid(gate). `key_scale` ([pages, key heads, positions
+    of a page], 32-bit): the values are the keys (the key pool is given as value pool too), and a score's q . k is
+    multiplied by its key's number before anything else."""
     o = AttentionOptions()
     o.scale, o.window, o.softcap = float(scale), int(window or 0), float(softcap or 0.0)
     o.keep = int(keep_first or 0) if window else 0
@@ -189,7 +191,17 @@ def attention_options(n_heads, scale, window=None, softcap=0.0, sink=False, sink
         if gate.dim() != 2 or gate.stride(1) != 1 or (gate_width is not None and gate.shape[1] < gate_width):
             raise library.KernelError(f"an output gate is [rows, {gate_width}] with contiguous rows, not {tuple(gate.shape)}")
         o.gate, o.gate_stride = gate.data_ptr(), gate.stride(0)
+    o.key_scale = _key_scale(key_scale)
     return o
+
+
+def _key_scale(key_scale):
+    if key_scale is None:
+        return None
+    if key_scale.dtype != torch.float32 or not key_scale.is_contiguous():
+        raise library.KernelError("the factors of keys are contiguous 32-bit numbers")
+    _cuda(key_scale)
+    return key_scale.data_ptr()
 
 
 def attention_generic(q, q_stride, out, kpool, vpool, positions, seq_of_row, tables, n_heads, n_kv_heads,
@@ -554,14 +566,14 @@ def attention_decode_fused_unit(partial, bias, v_col, gate_col, eps, q_mul, out,
     """The decode form fed by a stacked projection's unadded K slices for layers without rotation whose queries and keys are
     divided by their root mean square per head: adds the slices, norms, multiplies the queries by `q_mul` (one factor per
     query head, or None), stores the page rows, attends and applies the output gate whose pre-activations stand at column
-    `gate_col` (None: no gate), in one launch. Columns: q heads at 0, k heads behind them, v heads at `v_col` (the k heads'
-    column: the values are the keys as projected). Every row of the step is a single token."""
+    `gate_col` (None: no gate), in one launch. Columns: q heads at 0, k heads behind them, v heads at `v_col` (with the option
+    `key_scale` the k heads' column: the values are the keys as projected). Every row of the step is a single token."""
     part, cnt = _decode_scratch(out.device, n_rows, n_heads, n_kv_heads, head_dim, n_splits)
     opt = attention_options(n_heads, scale, window, **options)
     library.check(library.load().cuca_attention_decode_fused_unit(
         _p(partial.data), partial.slices, partial.slice_stride, _p(bias), partial.data.shape[2], int(v_col),
         -1 if gate_col is None else int(gate_col), float(eps), _per_head(q_mul, n_heads, "factors on the queries"), _p(out),
-        out.stride(0), _p(cache.k), _p(cache.v), cache.k.shape[0], cache.k.shape[2], _p(step.positions),
+        out.stride(0), _p(cache.k), _p(cache.k if cache.v is None else cache.v), cache.k.shape[0], cache.k.shape[2], _p(step.positions),
         _p(step.seq_of_row), _p(cache.tables), cache.tables.shape[1], None, n_rows, n_heads, n_kv_heads, head_dim,
         ctypes.addressof(opt), chunk, n_splits, _p(part), _p(cnt), _p(err), _stream()), "attention_decode_fused_unit")
 
@@ -1017,7 +1029,7 @@ def attention_generic_v(q, q_stride, out, kpool, vpool, positions, seq_of_row, t
 def norm_rope_store(qkv, k_col, v_col, positions, seq_of_row, tables, cos, sin, rotary_dim, adjacent, q_norm, k_norm,
                     v_norm: bool, eps: float, kpool, vpool, block_size, n_heads, n_kv_heads, head_dim, v_head_dim, err,
                     v_split: int = 1, q_out=None, v_row_dim: int = 0, whole: bool = False, q_temp=None,
-                    unit: bool = False, q_mul=None) -> None:
+                    unit: bool = False, q_mul=None, key_scale=None) -> None:
     """`rope_store_general` with norms per head in 32-bit before the rotation: q / rms(q) * q_norm, k likewise with
     k_norm (None: no norm), and with `v_norm` v / rms(v) before it is kept. q is rewritten in place, or goes to
     `q_out` [rows, heads * head_dim] of the pools' dtype (32-bit rows beside 16-bit pools). `v_row_dim` n > 0: a row's
@@ -1025,7 +1037,8 @@ def norm_rope_store(qkv, k_col, v_col, positions, seq_of_row, tables, cos, sin, 
     `whole`: the norm of q (and of k) is over the whole projection, all heads at once, with weights [heads * head_dim].
     `q_temp` (coef, every): the query at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1).
     `unit`: the norms per head have no weight. `q_mul` (32-bit, one per query head): a factor on the head's queries, after
-    the norm. `v_col` may be `k_col`: the values are then the keys as projected."""
+    the norm. `v_col` may be `k_col`: the values are then the keys as projected. `key_scale` (with `unit`, without rotation;
+    `vpool` None): the page rows hold the keys as projected and `key_scale` the factors their norms would have been."""
     _cuda(qkv, positions, seq_of_row, kpool, vpool, q_norm, k_norm, q_out)
     coef, every = (float(q_temp[0]), int(q_temp[1])) if q_temp else (0.0, 0)
     library.check(library.load().cuca_norm_rope_store_u(
@@ -1034,7 +1047,8 @@ def norm_rope_store(qkv, k_col, v_col, positions, seq_of_row, tables, cos, sin, 
         cos.shape[0] if cos is not None else 0, int(rotary_dim), int(bool(adjacent)), _p(q_norm), _p(k_norm),
         int(bool(v_norm)), float(eps), _p(kpool), _p(vpool), kpool.shape[0], int(block_size), qkv.shape[0], n_heads,
         n_kv_heads, head_dim, v_head_dim, int(v_split), int(v_row_dim), int(bool(whole)), coef, every, int(bool(unit)),
-        _per_head(q_mul, n_heads, "factors on the queries"), _p(err), _stream()), "norm_rope_store")
+        _per_head(q_mul, n_heads, "factors on the queries"), _key_scale(key_scale), _p(err), _stream()),
+        "norm_rope_store")
 
 
 def sigmoid_gate_(a, gate) -> None:

@@ -27,7 +27,9 @@ rows, the attention output and the output projection's input columns (zero colum
 the layer runs slab by slab like one whose values are a multiple. The norm on values is over the stored ones.
 
 More options of the general path. `qk_norm` "unit": the RMS norm per head has no weight. `values` "keys": there is no value
-projection, the values are the keys as projected (with their bias), before norm and rotation. `q_scale`: a stored factor
+projection, the values are the keys as projected (with their bias), before norm and rotation; where the keys are neither
+rotated nor normed with a weight, the pages hold one row for both and a 32-bit number per key, the factor of its norm,
+which multiplies the key's scores instead (half the cache, and half of what a decode step reads of it). `q_scale`: a stored factor
 per query head (`q_scale` [heads]) multiplies the head's scores; it goes into the queries, with the scale. `slopes` (one
 number per query head): slope * distance between query and key is taken off a score (after scale and cap). `keep_first` k
 beside a `window`: the first k keys of a request stay visible at their true distances; the pages that hold them stay with
@@ -111,6 +113,8 @@ class PagedAttention(Mixer):
         self.position = POSITIONS.get(pos.kind)(pos, runtime) if isinstance(pos, PartSpec) else None
         self.w_qkv = self.b_qkv = self.w_o = self.b_o = self.w_qn = self.w_kn = self.sink_values = None
         self.slopes = self.q_mul = None
+        # one row per key and value, and a factor per key
+        self.one_row = self.keys_as_values and self.norm_unit and self.position is None
         # what the stacked-projection kernels of the usual path do not take
         self.normed = self.qk_norm or self.v_norm or self.q_temp is not None or self.q_scaled
         self.general = (self.v_head_dim != self.head_dim or self.gated or self.head_gate or self.normed
@@ -122,7 +126,8 @@ class PagedAttention(Mixer):
                              "adjacent rotation pairs")
         # what the decode kernel that makes its own queries and keys takes
         self.fusable = (self.norm_unit and self.position is None and self.q_temp is None and not self.v_norm
-                        and not self.head_gate and self.v_head_dim == self.head_dim and self.head_dim in (16, 32, 64, 128))
+                        and not self.head_gate and self.v_head_dim == self.head_dim and self.head_dim in (16, 32, 64, 128)
+                        and self.one_row == self.keys_as_values)
         # the width of a value row in the pool: padded to a multiple of the key size for the tensor-core kernels
         self.v_pool_dim = self.v_head_dim
         d, dv = self.head_dim, self.v_head_dim
@@ -135,6 +140,8 @@ class PagedAttention(Mixer):
 
     # ------------------------------------------------------------ description
     def cache_needs(self):
+        if self.one_row:
+            return CacheNeeds(kv=KvNeeds(self.n_kv_heads, self.head_dim, self.window, 0, self.keep_first, key_scale=True))
         return CacheNeeds(kv=KvNeeds(self.n_kv_heads, self.head_dim, self.window,
                                      None if self.v_pool_dim == self.head_dim else self.v_pool_dim, self.keep_first))
 
@@ -236,6 +243,9 @@ class PagedAttention(Mixer):
         plan = self.plan(step) if split else None
         options = {"softcap": self.softcap, "sink": self.sink, "sink_values": self.sink_values, "keep_first": self.keep_first,
                    "slopes": self.slopes}
+        vpool = cache.v
+        if self.one_row:
+            vpool, options["key_scale"] = cache.k, cache.key_scale
         if (self.fusable and split == 1 and self.rt.use_partials and rows <= ops.ROPE_PARTIAL_MAX_ROWS
                 and ops.attention_decode_fused_supported(plan, cache, h.dtype, rows, nh, nkv, d)
                 and ops.gemm_partial_supported(h, self.w_qkv)):
@@ -259,7 +269,8 @@ class PagedAttention(Mixer):
             ops.norm_rope_store(proj, nh * d, v_col, step.positions, step.seq_of_row, cache.tables, cos, sin,
                                 rot, adjacent, self.w_qn, self.w_kn, self.v_norm, self.eps, cache.k, cache.v,
                                 cache.block_size, nh, nkv, d, dv, self.rt.err, v_split=split, v_row_dim=dv_row,
-                                whole=self.norm_whole, q_temp=self.q_temp, unit=self.norm_unit, q_mul=self.q_mul)
+                                whole=self.norm_whole, q_temp=self.q_temp, unit=self.norm_unit, q_mul=self.q_mul,
+                                key_scale=options.get("key_scale"))
         else:
             ops.rope_store_general(proj, nh * d, v_col, step.positions, step.seq_of_row, cache.tables, cos, sin,
                                    rot, adjacent, cache.k, cache.v, cache.block_size, nh, nkv, d, dv, self.rt.err,
@@ -267,7 +278,7 @@ class PagedAttention(Mixer):
         gate = proj[:, g_col:g_col + nh * dv] if self.gated else None  # (a layer with a gate per value is never padded)
         attn = self.rt.empty(rows, nh * dv)
         if tensor_cores:
-            slabs = cache.v.view(split, *cache.k.shape)
+            slabs = vpool.view(split, *cache.k.shape)
             parts = self.rt.empty(split, rows, nh * d) if split > 1 else attn.view(1, rows, nh * d)
             if split == 1:  # the gate is the attention kernels' own last step
                 options["gate"] = gate
@@ -277,7 +288,7 @@ class PagedAttention(Mixer):
             if parts.data_ptr() != attn.data_ptr():
                 ops.gate_merge(parts, gate, attn, nh, dv)
         else:
-            ops.attention_generic_v(proj, proj.stride(0), attn, cache.k, cache.v, step.positions, step.seq_of_row,
+            ops.attention_generic_v(proj, proj.stride(0), attn, cache.k, vpool, step.positions, step.seq_of_row,
                                     cache.tables, nh, nkv, d, dv, scale, self.window, self.rt.err, gate=gate, **options)
         if self.head_gate:
             ops.head_gate_(attn, proj[:, g_col:g_col + nh], nh, dv)

@@ -57,6 +57,7 @@ class KvNeeds:
     window: Optional[int] = None  # None: all keys; w: the last w keys
     v_head_dim: Optional[int] = None  # None: values as wide as keys; 0: no value slab (the mixer reads values out of its key rows)
     keep_first: int = 0  # beside the window, the first positions of a request stay visible
+    key_scale: bool = False  # a 32-bit number per position and key head beside the rows (the factor of a key's norm)
 
 
 @dataclass(frozen=True)

@@ -61,8 +61,9 @@ def test_run_order_caches_and_tensors():
     model = Model(spec)
     needs = model.cache_needs()
     assert len(needs) == 6 and all(n.state["shift"].shape == (60,) and n.state["shift"].dtype == "float32" for n in needs.values())
-    assert [(n.kv.window, n.kv.keep_first, n.kv.v_head_dim) for n in needs.values()] == \
-        [(13, 3, None), (5, 1, None), (13, 3, None), (40, 9, None), (5, 1, None), (13, 3, None)]
+    # (one row per key and value, and a factor per key)
+    assert all(n.kv.v_head_dim == 0 and n.kv.key_scale for n in needs.values())
+    assert [(n.kv.window, n.kv.keep_first) for n in needs.values()] == [(13, 3), (5, 1), (13, 3), (40, 9), (5, 1), (13, 3)]
     names = set(model.tensor_needs())
     want = {"embed", "pos", "head", "final.norm"}
     for i in (0, 1, 3):

@@ -230,7 +230,8 @@ class _Cache:
         shape = (sum(per) + 3, kv.n_kv_heads, bs)
         fill = float("nan") if rt.dtype == torch.float32 else 0.0
         self.k = torch.full((*shape, kv.head_dim), fill, dtype=rt.dtype, device=rt.device)
-        self.v = torch.full((*shape, kv.v_head_dim or kv.head_dim), fill, dtype=rt.dtype, device=rt.device)
+        self.v = None if kv.v_head_dim == 0 else torch.full((*shape, kv.v_head_dim or kv.head_dim), fill, dtype=rt.dtype, device=rt.device)
+        self.key_scale = torch.full(shape, float("nan"), device=rt.device) if kv.key_scale else None
         table = np.full((max(slots) + 2, max(per) + 2), -1)
         for n, s in zip(per, slots):
             table[s, :n] = [order.pop() for _ in range(n)]
@@ -247,7 +248,7 @@ class _Cache:
 
     def view(self, step):
         from cuca_b200.cache.device import CacheView
-        return CacheView(self.k, self.v, self.tables, self.bs, 0, None, step.slots)
+        return CacheView(self.k, self.v, self.tables, self.bs, 0, None, step.slots, self.key_scale)
 
 
 def _run_attention(part, rt, cache, xs, cuts, slots, E, dtype):
@@ -312,6 +313,11 @@ def test_unit_norm_and_page_write(eps):
             v_col = (nh + nkv) * d if own_v else nh * d
             ops.norm_rope_store(proj, nh * d, v_col, step.positions, step.seq_of_row, tables, None, None, 0, False, None, None, False,
                                 eps, k, v, bs, nh, nkv, d, d, rt.err, unit=True, q_mul=_t(mul, dev))
+            # one row for both, and the norm's factor beside it
+            again, k1, f1 = _t(src, dev, dtype), torch.zeros_like(k), torch.zeros(8, nkv, bs, device=dev)
+            ops.norm_rope_store(again, nh * d, nh * d, step.positions, step.seq_of_row, tables, None, None, 0, False, None, None, False,
+                                eps, k1, None, bs, nh, nkv, d, d, rt.err, unit=True, q_mul=_t(mul, dev), key_scale=f1)
+            assert torch.equal(again, proj)
             tol = 1e-5 if dtype == torch.float32 else 1e-2
             q = src[:, :nh * d].reshape(rows, nh, d)
             want = pp.rms(q, eps) * mul[:, None]
@@ -324,7 +330,9 @@ def test_unit_norm_and_page_write(eps):
                 at = (tb[s, p // bs], slice(None), p % bs)
                 assert np.abs(k[at].float().cpu().numpy() - pp.rms(kk, eps)).max() < tol * 8
                 assert np.array_equal(v[at].float().cpu().numpy(), vv.astype(np.float32))
-            assert int(rt.err.item()) == 0
+                assert np.array_equal(k1[at].float().cpu().numpy(), kk.astype(np.float32))
+                assert np.allclose(f1[at].cpu().numpy(), 1 / np.sqrt(np.mean(kk * kk, axis=1) + eps), rtol=1e-5)
+            assert int(rt.err.item()) == 0 and int((f1 != 0).sum()) == 21 * nkv
 
 
 def _planted(dtype, m, n, far, askers, E=40, eps=1e-6):
@@ -410,11 +418,12 @@ def _plain_options(q, k, v, o):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("d", [24, 32, 64, 128])
+@pytest.mark.parametrize("one_row", [False, True])
 @pytest.mark.parametrize("window, keep, cap, slopes, sink, gate", [
-    (None, 0, 0.0, True, False, False), (50, 3, 3.0, True, True, True), (130, 66, 0.0, False, True, False), (300, 20, 5.0, True, False, True),
+    (None, 0, 0.0, True, False, False), (50, 3, 3.0, True, True, True), (90, 0, 0.0, False, False, False), (130, 66, 0.0, False, True, False), (300, 20, 5.0, True, False, True),
     (None, 0, 2.0, True, True, True), (20, 200, 0.0, True, False, True)])
-def test_attention_options_in_every_form(dtype, d, window, keep, cap, slopes, sink, gate):
-    """Every option with every other through the plain kernel, the two prompt forms and the split-key decode form (one
+def test_attention_options_in_every_form(dtype, d, window, keep, cap, slopes, sink, gate, one_row):
+    """Every option with every other, rows of keys and values apart or one row for both with a factor per key, through the plain kernel, the two prompt forms and the split-key decode form (one
     chunk, several merged as a cluster, several through memory); positions up to 600; pages the window has passed gone."""
     from cuca_b200.cache.device import CacheView
     from cuca_b200.kernels import ops
@@ -425,7 +434,8 @@ def test_attention_options_in_every_form(dtype, d, window, keep, cap, slopes, si
     q, k, v = r(T, H, d), r(T, G, d), r(T, G, d)
     o = {"window": window, "keep": keep, "scale": 1.7 * d ** -0.5, "cap": cap, "slopes": rs.uniform(0.0, 0.1, H) if slopes else None,
          "sink": rs.normal(0, 2, H) if sink else None, "gate": r(T, H, d) if gate else None}
-    want = _plain_options(q, k, v, o)
+    factors = rs.uniform(0.2, 2.0, (T, G)).astype(np.float32)
+    want = _plain_options(q, k * factors[:, :, None] if one_row else k, k if one_row else v, o)
     order = rs.permutation(T // bs + 2)[:-(-T // bs)]
     kp, vp = torch.zeros(T // bs + 2, G, bs, d, dtype=dtype, device=dev), torch.zeros(T // bs + 2, G, bs, d, dtype=dtype, device=dev)
     pos = np.arange(T)
@@ -435,6 +445,9 @@ def test_attention_options_in_every_form(dtype, d, window, keep, cap, slopes, si
     tables[1, :len(order)] = torch.tensor(order, dtype=torch.int32)
     opts = {"softcap": cap, "slopes": None if o["slopes"] is None else _t(o["slopes"], dev), "keep_first": keep, "sink": sink,
             "sink_values": None if o["sink"] is None else _t(o["sink"], dev)}
+    if one_row:
+        vp, opts["key_scale"] = kp, torch.full((T // bs + 2, G, bs), float("nan"), device=dev)
+        opts["key_scale"][order[pos // bs], :, pos % bs] = _t(factors, dev)
 
     def run(rows, step, plan):
         qq = _t(q[rows].reshape(len(rows), -1), dev, dtype)
@@ -494,18 +507,23 @@ def test_decode_that_makes_its_own_queries_and_keys(H, G, d, gate, own_v, mul):
         kp, vp = torch.zeros(4 * pages, G, bs, d, dtype=torch.bfloat16, device=dev), torch.zeros(4 * pages, G, bs, d, dtype=torch.bfloat16, device=dev)
         tables = torch.tensor(rs.permutation(4 * pages).reshape(4, pages), dtype=torch.int32, device=dev)
         tb = tables.cpu().numpy()
+        fp = torch.full((4 * pages, G, bs), float("nan"), device=dev)
         raw = rs.normal(0, 1, (5, 4, cols))
         total = raw.sum(0) + bias
         want = np.zeros((4, H, d))
         for r, (n, s) in enumerate(zip(lengths, slots)):
             k, v, at = ks[r % 2, :n], vs[r % 2, :n], np.arange(n)
-            kp[tb[s, at // bs], :, at % bs] = _t(k, dev, torch.bfloat16)
+            if not own_v:  # the page holds the values, which are the keys before their factors
+                f = rs.uniform(0.3, 2.0, (n, G)).astype(np.float32)
+                k = v * f[:, :, None]
+                fp[tb[s, at // bs], :, at % bs] = _t(f, dev)
+            kp[tb[s, at // bs], :, at % bs] = _t(k if own_v else v, dev, torch.bfloat16)
             vp[tb[s, at // bs], :, at % bs] = _t(v, dev, torch.bfloat16)
             q = pp.rms(total[r, :H * d].reshape(H, d), eps) * (factor[:, None] if mul else 1.0)
             kn = total[r, H * d:(H + G) * d].reshape(1, G, d)
             vn = total[r, v_col:v_col + G * d].reshape(1, G, d)
             o = {"window": window, "keep": keep, "scale": 0.4, "cap": 0.0, "slopes": slopes, "sink": None, "gate": None}
-            kk, vv = pu.bf16_round(np.concatenate([k, pp.rms(kn, eps)])), pu.bf16_round(np.concatenate([v, vn]))
+            kk, vv = np.concatenate([k, pp.rms(kn, eps)]), pu.bf16_round(np.concatenate([v, vn]))
             qq = np.zeros((n + 1, H, d))
             qq[n] = pu.bf16_round(q)
             js = pp.visible(n, {"size": window, "keep_first": keep} if window else None)
@@ -518,17 +536,22 @@ def test_decode_that_makes_its_own_queries_and_keys(H, G, d, gate, own_v, mul):
             assert o["window"] == window
         step = _step(dev, [(n, 1) for n in lengths], slots)
         for chunk, n_splits in ((0, 1), (0, 2), (0, 4), (0, 8), (0, 6), (64, 8)):
-            cache = CacheView(kp.clone(), vp.clone(), tables, bs, 0, None, step.slots)
+            cache = CacheView(kp.clone(), vp.clone() if own_v else None, tables, bs, 0, None, step.slots, None if own_v else fp.clone())
             out = torch.empty(4, H * d, dtype=torch.bfloat16, device=dev)
             parts = ops.PartialSums(_t(raw, dev), 5)
             ops.attention_decode_fused_unit(parts, _t(bias, dev, torch.bfloat16), v_col, g_col if gate else None, eps,
                                             _t(factor, dev) if mul else None, out, cache, step, 4, H, G, d, 0.4, window, chunk,
-                                            n_splits, rt.err, slopes=_t(slopes, dev), keep_first=keep)
+                                            n_splits, rt.err, slopes=_t(slopes, dev), keep_first=keep,
+                                            key_scale=cache.key_scale)
             got = out.float().cpu().numpy().reshape(4, H, d)
             assert np.abs(got - want).max() < 2e-2 * np.abs(want).max(), (window, chunk, n_splits)
             for r, (n, s) in enumerate(zip(lengths, slots)):
-                row = cache.k[tb[s, n // bs], :, n % bs].float().cpu().numpy()
-                assert np.abs(row - pp.rms(total[r, H * d:(H + G) * d].reshape(G, d), eps)).max() < 2e-2 * np.abs(row).max()
+                row, key = cache.k[tb[s, n // bs], :, n % bs].float().cpu().numpy(), total[r, H * d:(H + G) * d].reshape(G, d)
+                if not own_v:
+                    assert np.abs(row - key).max() < 1e-2 * np.abs(row).max()
+                    assert np.allclose(cache.key_scale[tb[s, n // bs], :, n % bs].cpu().numpy(), 1 / np.sqrt(np.mean(key * key, axis=1) + eps), rtol=1e-4)
+                    continue
+                assert np.abs(row - pp.rms(key, eps)).max() < 2e-2 * np.abs(row).max()
                 row = cache.v[tb[s, n // bs], :, n % bs].float().cpu().numpy()
                 assert np.abs(row - total[r, v_col:v_col + G * d].reshape(G, d)).max() < 1e-2 * np.abs(row).max()
     assert int(rt.err.item()) == 0
