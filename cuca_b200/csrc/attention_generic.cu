@@ -403,7 +403,7 @@ norm_rope_store_kernel(T* __restrict__ qkv, int ld, int k_col, int v_col, TP* __
 // The same without rotation for bfloat16 rows with heads of a multiple of eight values and value heads as wide as keys:
 // `group` lanes (a power of two) take one head of one row, 16 bytes a lane. Values that are the keys as projected
 // (v_col == k_col) are written by the lanes that have them.
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(768)
 norm_store_kernel(__nv_bfloat16* __restrict__ qkv, int ld, int k_col, int v_col, const int* __restrict__ positions,
                   const int* __restrict__ seq_of_row, const int* __restrict__ tables, int table_stride,
                   const float* __restrict__ q_norm, const float* __restrict__ k_norm, int v_norm, float eps,
@@ -496,8 +496,8 @@ CUCA_API int cuca_norm_rope_store_u(void* qkv, int dtype, int ld, int k_col, int
     int group = 1;
     while (group * 8 < d) group *= 2;
     const int lanes = (nh + nkv * (v_col == k_col ? 1 : 2)) * group;
-    const int threads = lanes < 256 ? (lanes + 31) / 32 * 32 : 256;
-    cuca_launch(norm_store_kernel, dim3(n_rows, (lanes + threads - 1) / threads), dim3(threads), 0, stream, true, (__nv_bfloat16*)qkv, ld,
+    const int blocks = (lanes + 767) / 768, threads = ((lanes + blocks - 1) / blocks + 31) / 32 * 32;  // of a row
+    cuca_launch(norm_store_kernel, dim3(n_rows, blocks), dim3(threads), 0, stream, true, (__nv_bfloat16*)qkv, ld,
                 k_col, v_col, positions, seq_of_row, tables, table_stride, q_norm, k_norm, v_norm, eps,
                 (__nv_bfloat16*)kpool, (__nv_bfloat16*)vpool, n_blocks, bs, nh, nkv, d, group, qt_coef, qt_every, unit,
                 q_mul, key_scale, err);

@@ -57,9 +57,10 @@ __device__ __forceinline__ void block_sums(float (&s)[N], float* red) {
 }
 
 // One block per row. R > 0: a thread holds R packs of V values (blockDim R V >= E); R = 0: the sum stays in x between the
-// passes (rows wider than a block can hold).
-template <typename TO, int V, int R>
-__global__ void __launch_bounds__(1024, 1)
+// passes (rows wider than a block can hold). AHEAD: slices asked for at once (many: few rows, whose time is latency; one:
+// many rows, whose terms are whole tensors, so that more blocks fit an SM).
+template <typename TO, int V, int R, int AHEAD>
+__global__ void __launch_bounds__(1024, AHEAD == 1 ? 2 : 1)
 sum_norm_kernel(const SumNorm p, float* __restrict__ x, TO* __restrict__ out) {
   __shared__ float red[32];
   pdl_trigger();
@@ -82,13 +83,13 @@ sum_norm_kernel(const SumNorm p, float* __restrict__ x, TO* __restrict__ out) {
       const int i = threadIdx.x * V + r * step;
       if (i >= p.E) continue;
       wv[r] = ld<V>(p.w + i);
-      z[r] = summed<V, R == 1 ? 8 : 4>(p, row, i);
+      z[r] = summed<V, AHEAD>(p, row, i);
 #pragma unroll
       for (int k = 0; k < V; ++k) q[0] = fmaf(z[r].v[k], z[r].v[k], q[0]);
     }
   } else {
     for (int i = threadIdx.x * V; i < p.E; i += step) {
-      const Pack<V> v = summed<V>(p, row, i);
+      const Pack<V> v = summed<V, AHEAD>(p, row, i);
       st<V>(x + row * p.E + i, v);
 #pragma unroll
       for (int k = 0; k < V; ++k) q[0] = fmaf(v.v[k], v.v[k], q[0]);
@@ -140,6 +141,7 @@ sum_norm_shift_kernel(const SumNorm p, const Shift sh, float* __restrict__ x_out
   float q[ROWS + 1];
   // one row a block (single tokens, mostly): what the rest of the row needs is asked for before the reduction
   constexpr bool EARLY = ROWS == 1 && R == 1;
+  constexpr int AHEAD = EARLY ? 6 : ROWS > 1 ? 1 : 2;
   Pack<V> wv, mixv, keptv;
   const int i0 = threadIdx.x * V;
   if (EARLY && i0 < p.E && seq[1] >= 0) {
@@ -156,7 +158,7 @@ sum_norm_shift_kernel(const SumNorm p, const Shift sh, float* __restrict__ x_out
 #pragma unroll
       for (int k = 0; k < V; ++k) z[j][r].v[k] = 0.f;
       if (seq[j] < 0 || i >= p.E) continue;
-      z[j][r] = summed<V, EARLY ? 8 : 4>(p, r0 - 1 + j, i);
+      z[j][r] = summed<V, AHEAD>(p, r0 - 1 + j, i);
 #pragma unroll
       for (int k = 0; k < V; ++k) q[j] = fmaf(z[j][r].v[k], z[j][r].v[k], q[j]);
     }
@@ -211,7 +213,7 @@ sum_norm_shift_kernel(const SumNorm p, const Shift sh, float* __restrict__ x_out
   for (int r = 0; r < R; ++r) {
     const int i = threadIdx.x * V + r * step;
     if (i >= p.E) continue;
-    z[0][r] = summed<V>(p, row, i);
+    z[0][r] = summed<V, AHEAD>(p, row, i);
 #pragma unroll
     for (int k = 0; k < V; ++k) t[0] = fmaf(z[0][r].v[k], z[0][r].v[k], t[0]);
   }
@@ -277,11 +279,16 @@ template <typename TO, int V>
 void launch_sum_norm(const SumNorm& p, float* x, TO* out, int n_rows, cudaStream_t stream) {
   int threads, held;
   shape_for(p.E / V, &threads, &held);
-#define SN(R) cuca_launch(sum_norm_kernel<TO, V, R>, dim3(n_rows), dim3(threads), 0, stream, true, p, x, out)
-  if (held == 1) SN(1);
-  else if (held == 2) SN(2);
-  else if (held == 4) SN(4);
-  else SN(0);
+  const bool many = n_rows > 512;  // (beyond what leaves K slices)
+#define SN(R, AHEAD)                                                                                                    \
+  do {                                                                                                                  \
+    if (many) cuca_launch(sum_norm_kernel<TO, V, R, 1>, dim3(n_rows), dim3(threads), 0, stream, true, p, x, out);       \
+    else cuca_launch(sum_norm_kernel<TO, V, R, AHEAD>, dim3(n_rows), dim3(threads), 0, stream, true, p, x, out);        \
+  } while (0)
+  if (held == 1) SN(1, 8);
+  else if (held == 2) SN(2, 4);
+  else if (held == 4) SN(4, 2);
+  else SN(0, 4);
 #undef SN
 }
 
