@@ -142,10 +142,19 @@ struct Smem {
   static constexpr int HALVES = D / 64;
   static constexpr int SUB_BYTES = 16 * 128;
   static constexpr int WSTAGE_BYTES = KV * (HALVES > 0 ? HALVES : 1) * SUB_BYTES;
-  static constexpr int WSTAGES = SHARED ? 4 : 3;
+  // groups of one round (two where one tile is key and value: the chain of a round, scores, maximum, exponents, products, is
+  // what a warp waits for) and three rounds of stages: two in flight while one is worked on
+  static constexpr int PER_ROUND = SHARED ? 2 : 1;
+  static constexpr int WSTAGES = 3 * PER_ROUND;
   static constexpr int FACTOR_BYTES = SHARED ? 16 * 4 : 0;  // of a stage's keys
   static constexpr int RING_BYTES = 4 * WSTAGES * WSTAGE_BYTES;
   static constexpr int TMA_BYTES = RING_BYTES + 1024 /*alignment*/ + (Q_ELEMS + 2 * D) * 2 + 4 * WSTAGES * FACTOR_BYTES;
+};
+
+// Where the groups of 16 keys of an update start.
+template <int N>
+struct KeyGroups {
+  int at[N];
 };
 
 // One warp's state over its 16 MMA rows: thread (g, t) holds rows g and g + 8.
@@ -347,7 +356,7 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
   // ---- TMA form: this warp's 16-key groups are (tile ti, keys 16 warp .. 16 warp + 15) for ti in [ti_lo, ti_hi)
   __shared__ __align__(8) uint64_t w_full[4][S::WSTAGES];
   __shared__ int w_abort;
-  int ti_lo = 0, n_mine = 0, next_page = -1;
+  int ti_lo = 0, n_mine = 0, next_page[S::PER_ROUND];
   uint8_t* ring = ring_base + (size_t)warp * S::WSTAGES * S::WSTAGE_BYTES;
   // (behind the query rows and the row's own key and value)
   float* factors = reinterpret_cast<float*>(ring_base + S::RING_BYTES + (S::Q_ELEMS + 2 * D) * 2) + warp * S::WSTAGES * 16;
@@ -451,9 +460,10 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
         pg[j] = __shfl_sync(0xffffffffu, pg[j], 0);
       }
 #pragma unroll
-      for (int j = 0; j < S::WSTAGES - 1; ++j)
+      for (int j = 0; j < S::WSTAGES - S::PER_ROUND; ++j)
         if (j < n_mine) issue_group(j, pg[j]);
-      next_page = pg[S::WSTAGES - 1];
+#pragma unroll
+      for (int u = 0; u < S::PER_ROUND; ++u) next_page[u] = pg[S::WSTAGES - S::PER_ROUND + u];
     }
   } else {
     if (threadIdx.x < TILE) {
@@ -646,12 +656,13 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
 
   // decode: a warp owns 16 keys of each tile and updates its softmax per 16 keys; prefill: every warp takes all
   // 64 keys of the tile in one softmax update
-  constexpr int SUBS = DECODE ? 1 : TILE / 16;   // 16-key groups per update
+  constexpr int SUBS = !DECODE ? TILE / 16 : TMA ? S::PER_ROUND : 1;  // 16-key groups per update
   constexpr int NT = 2 * SUBS;                    // 8-key n-tiles per update
-  // One update with the keys [kp0, kp0 + 16 SUBS): kaddr / vaddr give the shared-memory address of (key, dim),
-  // `key` counted from key0 within what they address.
+  // One update with SUBS groups of 16 keys, group u from position kps.at[u] on (for a prompt consecutive): kaddr / vaddr give the
+  // shared-memory address of (key, dim), `key` counted from key0 within what they address.
   // `factor` (SHARED): the factors of those keys.
-  auto update = [&](auto kaddr, auto vaddr, const int kp0, const int key0, const float* factor) {
+  auto update = [&](auto kaddr, auto vaddr, const KeyGroups<SUBS> kps, const int key0, const float* factor) {
+    const int kp0 = kps.at[0];
     // ---- S = Q K^T
     float s[NT][4];
 #pragma unroll
@@ -685,11 +696,12 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
 #pragma unroll
         for (int e = 0; e < 2; ++e) s[nt][2 * h + e] = score_log2(SHARED ? s[nt][2 * h + e] * factor[nt * 8 + 2 * t + e] : s[nt][2 * h + e], p);
       if (p.slopes) {
-        const float d0 = (float)(row_pos[h] - kp0 - 2 * t);  // the distance of the thread's first key
 #pragma unroll
-        for (int nt = 0; nt < NT; ++nt)
+        for (int nt = 0; nt < NT; ++nt) {
+          const float d0 = (float)(row_pos[h] - kps.at[nt >> 1] - (nt & 1) * 8 - 2 * t);
 #pragma unroll
-          for (int e = 0; e < 2; ++e) s[nt][2 * h + e] = fmaf(-slope2[h], d0 - (float)(nt * 8 + e), s[nt][2 * h + e]);
+          for (int e = 0; e < 2; ++e) s[nt][2 * h + e] = fmaf(-slope2[h], d0 - (float)e, s[nt][2 * h + e]);
+        }
       }
       if (whole) {
 #pragma unroll
@@ -702,7 +714,7 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
         for (int nt = 0; nt < NT; ++nt)
 #pragma unroll
           for (int e = 0; e < 2; ++e) {
-            const int kp = kp0 + nt * 8 + 2 * t + e;
+            const int kp = kps.at[nt >> 1] + (nt & 1) * 8 + 2 * t + e;
             const bool ok = row_ok[h] && kp <= row_pos[h] && (kp >= lo_row || kp < p.keep);
             if (!ok) s[nt][2 * h + e] = -INFINITY;
             mx = fmaxf(mx, s[nt][2 * h + e]);
@@ -746,44 +758,54 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
     }
   };
 
-  if (TMA) {
+  if constexpr (TMA) {
     // every warp walks its own groups through its own ring: no block-wide barrier in the loop
     bool ok = true;
-    for (int i = 0; i < n_mine && ok; ++i) {
-      {
-        // group i + WSTAGES - 1 goes into the stage that group i - 1 left; the page of the one after is looked up now
-        // (by lane 0, which hands it to the warp one round later)
-        const int j = i + S::WSTAGES - 1;
-        const int page_j = __shfl_sync(0xffffffffu, next_page, 0);
-        if (lane == 0 && j + 1 < n_mine) next_page = page_of(j + 1);
+    constexpr int PR = S::PER_ROUND;
+    for (int i = 0; i < n_mine && ok; i += PR) {
+      // The groups two rounds on go into the stages that the last round left; the pages of those after them are looked up
+      // now (by lane 0, which hands them to the warp one round later).
+#pragma unroll
+      for (int u = 0; u < PR; ++u) {
+        const int j = i + S::WSTAGES - PR + u;
+        const int page_j = __shfl_sync(0xffffffffu, next_page[u], 0);
+        if (lane == 0 && j + PR < n_mine) next_page[u] = page_of(j + PR);
         if (j < n_mine) issue_group(j, page_j);
       }
-      const int st_i = i % S::WSTAGES;
-      ok = mbar_wait(&w_full[warp][st_i], (i / S::WSTAGES) & 1, p.err, &w_abort);
-      ok = __all_sync(0xffffffffu, ok);
+      const int st_i = i % S::WSTAGES, n_here = min(PR, n_mine - i);
+      for (int u = 0; u < n_here && ok; ++u)
+        ok = __all_sync(0xffffffffu, mbar_wait(&w_full[warp][st_i + u], (i / S::WSTAGES) & 1, p.err, &w_abort));
       if (!ok) break;
       const uint32_t kbase = smem_u32(ring + (size_t)st_i * S::WSTAGE_BYTES);
       const uint32_t vbase = SHARED ? kbase : kbase + S::HALVES * S::SUB_BYTES;
+      // a round without its second group takes the first one's rows in its place, at a position that no row sees
+      const uint32_t second = n_here == PR ? S::WSTAGE_BYTES : 0;
       // (key, dim) in a swizzled half: row `key` of 128 bytes, 16-byte chunk (dim % 64) / 8 XOR (key % 8)
-      auto sw = [](uint32_t base, int key, int dim) {
-        return base + (uint32_t)((dim >> 6) * S::SUB_BYTES + key * 128 + ((((dim & 63) >> 3) ^ (key & 7)) << 4));
+      auto sw = [second](uint32_t base, int key, int dim) {
+        if (PR > 1) base += key >= 16 ? second : 0;
+        const int k = PR > 1 ? key & 15 : key;
+        return base + (uint32_t)((dim >> 6) * S::SUB_BYTES + k * 128 + ((((dim & 63) >> 3) ^ (k & 7)) << 4));
       };
-      const int kp0 = group_kp0(i);
-      if (owner && P >= kp0 && P < kp0 + 16) {
+      KeyGroups<PR> kps;
+#pragma unroll
+      for (int u = 0; u < PR; ++u) kps.at[u] = u < n_here ? group_kp0(i + u) : (1 << 30);
+#pragma unroll
+      for (int u = 0; u < PR; ++u) {
+        if (!(owner && P >= kps.at[u] && P < kps.at[u] + 16)) continue;
         // the row's own key and value take their place among the warp's keys (the page's row is stale)
-        const int key = P - kp0;
-        if (SHARED && lane == 0) factors[st_i * 16 + key] = s_own_factor;
+        const int key = P - kps.at[u];
+        if (SHARED && lane == 0) factors[(st_i + u) * 16 + key] = s_own_factor;
         for (int c = lane; c < S::KV * (D / 8); c += 32) {
           const int which = c / (D / 8), ch = c % (D / 8);
           const uint4 val = *reinterpret_cast<const uint4*>((which ? v_new : k_new) + ch * 8);
-          const uint32_t dst = sw(which ? vbase : kbase, key, ch * 8);
+          const uint32_t dst = sw(which ? vbase : kbase, 16 * u + key, ch * 8);
           asm volatile("st.shared.v4.b32 [%0], {%1, %2, %3, %4};" ::"r"(dst), "r"(val.x), "r"(val.y), "r"(val.z), "r"(val.w) : "memory");
         }
-        __syncwarp();
       }
-      update([&](int key, int dim) { return sw(kbase, key, dim); }, [&](int key, int dim) { return sw(vbase, key, dim); },
-             kp0, 0, factors + st_i * 16);
-      __syncwarp();  // every lane has read the stage before lane 0 asks for the next group into it
+      if (owner) __syncwarp();
+      update([&](int key, int dim) { return sw(kbase, key, dim); }, [&](int key, int dim) { return sw(vbase, key, dim); }, kps, 0,
+             factors + st_i * 16);
+      __syncwarp();  // every lane has read the stages before lane 0 asks for the next groups into them
     }
     if (w_abort) {
       // copies in flight land before the shared memory is used again
@@ -820,10 +842,14 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
       const int kp0 = start + sub0 * 16;              // first key of this update
       bool active = kp0 < range_hi && (kp0 + 16 * SUBS > range_lo || kp0 < p.keep);
       if (!DECODE && kp0 > warp_pmax) active = false;  // every row of this warp lies before these keys (causal)
-      if (active)
+      if (active) {
+        KeyGroups<SUBS> kps;
+#pragma unroll
+        for (int u = 0; u < SUBS; ++u) kps.at[u] = kp0 + 16 * u;
         update([&](int key, int dim) { return smem_u32(ks + key * S::RS + dim); },
-               [&](int key, int dim) { return smem_u32(vs + key * S::RS + dim); }, kp0, sub0 * 16,
+               [&](int key, int dim) { return smem_u32(vs + key * S::RS + dim); }, kps, sub0 * 16,
                tile_factor + sub0 * 16);
+      }
       if (look_ahead) {
         s_rowoff[ti % STAGES][threadIdx.x] = next_off;  // this slot was last read to request tile ti
         if (SHARED) s_factor[SHARED && !TMA ? (ti + STAGES) % (STAGES + 1) : 0][threadIdx.x] = next_factor;
