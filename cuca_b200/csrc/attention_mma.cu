@@ -122,6 +122,12 @@ __device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], 
       : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
+// the 8 x 8 matrix of 16-bit values that the warp holds (thread (g, t): row g, columns 2 t and 2 t + 1), transposed
+__device__ __forceinline__ uint32_t transpose_8x8(uint32_t a) {
+  uint32_t d;
+  asm volatile("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(d) : "r"(a));
+  return d;
+}
 __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
   __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
   return *reinterpret_cast<uint32_t*>(&v);
@@ -178,13 +184,17 @@ __device__ __forceinline__ float sink_term(float m, const AttnParams& p, int hea
 }
 
 // FUSED: 1: decode fed by the projection's K slices, with rotation; 2: with unit norms per head instead (and an output gate)
-template <int D, bool DECODE, int FUSED, bool TMA, bool SHARED>
+// TURNED (decode, up to eight query heads per key head): the keys are the 16 MMA rows and the heads the 8 columns, S^T = K Q^T
+// and O^T = V^T P^T, so that half as many MMAs work on padding. mma.sync sets the pace where one page row serves as key and
+// value: a step's bytes are half of what they are else (64 rows of 8,000 keys, 4 heads a group: 158 us for 532 MB before).
+template <int D, bool DECODE, int FUSED, bool TMA, bool SHARED, bool TURNED>
 __global__ void __launch_bounds__(NTHREADS)
 attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV) {
   static_assert(!FUSED || DECODE, "only the decode form takes the projection's K slices");
   static_assert(!TMA || (DECODE && D % 64 == 0), "the TMA form is for decode with head sizes 64 and 128");
   extern __shared__ __align__(16) uint8_t smem_raw[];
   __nv_bfloat16* smem = reinterpret_cast<__nv_bfloat16*>(smem_raw);
+  static_assert(!TURNED || (DECODE && TMA && SHARED), "the turned form is for decode with TMA over one-row pages");
   static_assert(!SHARED || FUSED != 1, "rotated keys are not values");
   using S = Smem<D, SHARED>;
   uint8_t* ring_base = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
@@ -284,9 +294,17 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
   const int* table = p.tables + (size_t)seq * p.table_stride;
 
   // ---------------------------------------------------------------- query fragments (A operand), from global
-  uint32_t qf[D / 16][4];
+  uint32_t qf[D / 16][TURNED ? 2 : 4];  // (turned: the B operand, thread (g, t) has head g and dimensions 2t, 2t + 1 and 8 on)
 #pragma unroll
   for (int ks = 0; ks < D / 16; ++ks) {
+    if constexpr (TURNED) {
+      qf[ks][0] = qf[ks][1] = 0;
+      if (!FUSED && row_ok[0]) {  // (g < G)
+        const __nv_bfloat16* qp = p.q + (size_t)dec_row * p.q_stride + (size_t)row_head[0] * D + ks * 16 + 2 * t;
+        qf[ks][0] = *reinterpret_cast<const uint32_t*>(qp);
+        qf[ks][1] = *reinterpret_cast<const uint32_t*>(qp + 8);
+      }
+    } else {
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
       uint32_t lo = 0, hi = 0;
@@ -298,11 +316,13 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
       qf[ks][h] = lo;       // a0 (row g) / a1 (row g + 8): k = 2t, 2t + 1
       qf[ks][2 + h] = hi;   // a2 / a3: k = 2t + 8, 2t + 9
     }
+    }
   }
 
-  WarpState<D> st;
+  // turned: acc[j] is dimensions 16 j + g (and + 8 in the second half) of heads 2t and 2t + 1, m and l are those heads'
+  WarpState<TURNED ? D / 2 : D> st;
 #pragma unroll
-  for (int j = 0; j < D / 8; ++j)
+  for (int j = 0; j < (TURNED ? D / 16 : D / 8); ++j)
 #pragma unroll
     for (int c = 0; c < 4; ++c) st.acc[j][c] = 0.f;
   st.m[0] = st.m[1] = -INFINITY;
@@ -315,7 +335,10 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
   };
   float slope2[2];  // the distance bias of the owned rows, in log2 units
 #pragma unroll
-  for (int h = 0; h < 2; ++h) slope2[h] = (p.slopes && row_ok[h]) ? p.slopes[row_head[h]] * CUCA_LOG2E : 0.f;
+  for (int h = 0; h < 2; ++h) {
+    if (TURNED) slope2[h] = (p.slopes && 2 * t + h < G) ? p.slopes[kvh * G + 2 * t + h] * CUCA_LOG2E : 0.f;
+    else slope2[h] = (p.slopes && row_ok[h]) ? p.slopes[row_head[h]] * CUCA_LOG2E : 0.f;
+  }
 
   // Row offsets of a tile's 64 keys in the pools (-1: masked or without a page), one tile ahead of the copies:
   // the page-table lookups of tile i + 2 are in flight while tile i is computed, so no copy waits on one.
@@ -632,10 +655,10 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
 #pragma unroll
     for (int ks = 0; ks < D / 16; ++ks)
 #pragma unroll
-      for (int h = 0; h < 2; ++h) {
+      for (int h = 0; h < (TURNED ? 1 : 2); ++h) {
         const __nv_bfloat16* qp = q_s + (g + 8 * h) * S::RS + ks * 16 + 2 * t;
         qf[ks][h] = *reinterpret_cast<const uint32_t*>(qp);
-        qf[ks][2 + h] = *reinterpret_cast<const uint32_t*>(qp + 8);
+        qf[ks][(TURNED ? 1 : 2) + h] = *reinterpret_cast<const uint32_t*>(qp + 8);
       }
     if (owner) {
       // the page keeps the new key and value for the steps to come
@@ -663,6 +686,79 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
   // `factor` (SHARED): the factors of those keys.
   auto update = [&](auto kaddr, auto vaddr, const KeyGroups<SUBS> kps, const int key0, const float* factor) {
     const int kp0 = kps.at[0];
+    if constexpr (TURNED) {
+      // ---- S^T = K Q^T: per group of 16 keys two accumulators (even and odd K steps), thread (g, t) gets keys g and g + 8 of
+      // heads 2t and 2t + 1
+      float sc[SUBS][2][4];
+#pragma unroll
+      for (int u = 0; u < SUBS; ++u)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) sc[u][0][c] = sc[u][1][c] = 0.f;
+      const int mat = lane >> 3, r = lane & 7;
+#pragma unroll
+      for (int kk = 0; kk < D / 16; ++kk)
+#pragma unroll
+        for (int u = 0; u < SUBS; ++u) {
+          uint32_t a[4];
+          ldsm_x4(a, kaddr(u * 16 + (mat & 1) * 8 + r, kk * 16 + (mat >> 1) * 8));
+          mma_bf16(sc[u][kk & 1], a, qf[kk][0], qf[kk][1]);
+        }
+      // ---- scale, mask, online softmax per head over the keys, which lie across the eight g
+      float v[SUBS][4];
+      const int lo_row = range_lo;
+#pragma unroll
+      for (int u = 0; u < SUBS; ++u)
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          const int kp = kps.at[u] + g + 8 * half;
+          const bool seen = kp <= P && (kp >= lo_row || kp < p.keep);
+          const float f = factor[u * 16 + g + 8 * half];
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            float x = score_log2((sc[u][0][2 * half + e] + sc[u][1][2 * half + e]) * f, p);
+            if (p.slopes) x = fmaf(-slope2[e], (float)(P - kp), x);
+            v[u][2 * half + e] = seen ? x : -INFINITY;
+          }
+        }
+      float corr[2];
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        float mx = -INFINITY;
+#pragma unroll
+        for (int u = 0; u < SUBS; ++u) mx = fmaxf(mx, fmaxf(v[u][e], v[u][2 + e]));
+#pragma unroll
+        for (int o = 4; o < 32; o <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+        const float m_new = fmaxf(st.m[e], mx), m_use = m_new == -INFINITY ? 0.f : m_new;
+        corr[e] = (m_new == -INFINITY) ? 1.f : exp2f(st.m[e] - m_new);
+        float sum = 0.f;
+#pragma unroll
+        for (int u = 0; u < SUBS; ++u)
+#pragma unroll
+          for (int half = 0; half < 2; ++half) {
+            const float x = exp2f(v[u][2 * half + e] - m_use);  // (exp2(-inf) is 0)
+            v[u][2 * half + e] = x;
+            sum += x;
+          }
+        st.l[e] = st.l[e] * corr[e] + sum;
+        st.m[e] = m_new;
+      }
+#pragma unroll
+      for (int j = 0; j < D / 16; ++j)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) st.acc[j][c] *= corr[c & 1];
+      // ---- O^T += V^T P^T: the tile read transposed is the A operand, P turned round the B operand
+#pragma unroll
+      for (int u = 0; u < SUBS; ++u) {
+        const uint32_t b0 = transpose_8x8(pack_bf16(v[u][0], v[u][1])), b1 = transpose_8x8(pack_bf16(v[u][2], v[u][3]));
+#pragma unroll
+        for (int j = 0; j < D / 16; ++j) {
+          uint32_t a[4];
+          ldsm_x4_trans(a, vaddr(u * 16 + (mat >> 1) * 8 + r, j * 16 + (mat & 1) * 8));
+          mma_bf16(st.acc[j], a, b0, b1);
+        }
+      }
+      return;
+    } else {
     // ---- S = Q K^T
     float s[NT][4];
 #pragma unroll
@@ -755,6 +851,7 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
         mma_bf16(st.acc[j], pa[sub], b[0], b[1]);
         mma_bf16(st.acc[j + 1], pa[sub], b[2], b[3]);
       }
+    }
     }
   };
 
@@ -861,11 +958,16 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
   // row sums live spread over the four threads of a quad
 #pragma unroll
   for (int h = 0; h < 2; ++h) {
-    st.l[h] += __shfl_xor_sync(0xffffffffu, st.l[h], 1);
-    st.l[h] += __shfl_xor_sync(0xffffffffu, st.l[h], 2);
+    if constexpr (TURNED) {  // (over the eight g)
+#pragma unroll
+      for (int o = 4; o < 32; o <<= 1) st.l[h] += __shfl_xor_sync(0xffffffffu, st.l[h], o);
+    } else {
+      st.l[h] += __shfl_xor_sync(0xffffffffu, st.l[h], 1);
+      st.l[h] += __shfl_xor_sync(0xffffffffu, st.l[h], 2);
+    }
   }
 
-  if (!DECODE) {
+  if constexpr (!DECODE) {
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
       if (!row_ok[h]) continue;
@@ -901,6 +1003,19 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
   };
 #pragma unroll
   for (int h = 0; h < 2; ++h) {
+    if constexpr (TURNED) {
+      float* dst = fs + ((size_t)warp * 16 + 2 * t + h) * FR;
+#pragma unroll
+      for (int j = 0; j < D / 16; ++j) {
+        dst[j * 16 + g] = st.acc[j][h];
+        dst[j * 16 + 8 + g] = st.acc[j][2 + h];
+      }
+      if (g == 0) {
+        dst[D] = st.m[h];
+        dst[D + 1] = st.l[h];
+      }
+      continue;
+    } else {
     int rowi = g + 8 * h;
     float* dst = fs + ((size_t)warp * 16 + rowi) * FR;
 #pragma unroll
@@ -911,6 +1026,7 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
     if (t == 0) {
       dst[D] = st.m[h];
       dst[D + 1] = st.l[h];
+    }
     }
   }
   __syncthreads();
@@ -1071,7 +1187,7 @@ attn_mma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap tmK, con
   if (threadIdx.x == 0) p.counters[blockIdx.z * p.nkv + kvh] = 0;
 }
 
-template <int D, bool DECODE, int FUSED, bool TMA, bool SHARED>
+template <int D, bool DECODE, int FUSED, bool TMA, bool SHARED, bool TURNED = false>
 int launch(const AttnParams& p, const CUtensorMap& tmK, const CUtensorMap& tmV, dim3 grid, cudaStream_t stream) {
   using S = Smem<D, SHARED>;
   int smem = TMA ? S::TMA_BYTES : FUSED ? S::FUSED_BYTES : S::BYTES;
@@ -1082,7 +1198,7 @@ int launch(const AttnParams& p, const CUtensorMap& tmK, const CUtensorMap& tmV, 
   }
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(attn_mma_kernel<D, DECODE, FUSED, TMA, SHARED>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    cudaError_t e = cudaFuncSetAttribute(attn_mma_kernel<D, DECODE, FUSED, TMA, SHARED, TURNED>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) {
       cuca_set_error("attention: cannot reserve %d bytes of shared memory: %s", smem, cudaGetErrorString(e));
       return 2;
@@ -1090,9 +1206,9 @@ int launch(const AttnParams& p, const CUtensorMap& tmK, const CUtensorMap& tmV, 
     configured = true;
   }
   if (DECODE && p.cluster)
-    cuca_launch_cluster(attn_mma_kernel<D, DECODE, FUSED, TMA, SHARED>, grid, dim3(NTHREADS), smem, stream, true, grid.x, p, tmK, tmV);
+    cuca_launch_cluster(attn_mma_kernel<D, DECODE, FUSED, TMA, SHARED, TURNED>, grid, dim3(NTHREADS), smem, stream, true, grid.x, p, tmK, tmV);
   else
-    cuca_launch(attn_mma_kernel<D, DECODE, FUSED, TMA, SHARED>, grid, dim3(NTHREADS), smem, stream, true, p, tmK, tmV);
+    cuca_launch(attn_mma_kernel<D, DECODE, FUSED, TMA, SHARED, TURNED>, grid, dim3(NTHREADS), smem, stream, true, p, tmK, tmV);
   CUCA_CHECK_LAUNCH("attention_mma");
   return 0;
 }
@@ -1107,6 +1223,12 @@ int dispatch_as(int d, const AttnParams& p, dim3 grid, cudaStream_t stream, bool
     const uint64_t rows = (uint64_t)p.n_blocks * p.nkv * p.bs;
     if (!cuca_tensor_map_bf16(p.kpool, rows, d, d, 16, &tmK) || !cuca_tensor_map_bf16(p.vpool, rows, d, d, 16, &tmV))
       tma = false;
+  }
+  if constexpr (DECODE && SHARED) {
+    if (tma && p.nh / p.nkv <= 8) {
+      if (d == 64) return launch<64, true, FUSED, true, true, true>(p, tmK, tmV, grid, stream);
+      if (d == 128) return launch<128, true, FUSED, true, true, true>(p, tmK, tmV, grid, stream);
+    }
   }
   if constexpr (DECODE) {
     if (tma && d == 64) return launch<64, true, FUSED, true, SHARED>(p, tmK, tmV, grid, stream);

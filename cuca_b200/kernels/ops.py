@@ -390,14 +390,15 @@ class AttentionPlan:
         if want_rows:
             self._decode_rows = rows
 
-    def chunk(self, n_kv_heads: int, head_dim: int, window=None, keep_first: int = 0):
-        """(chunk, most chunks of a row) of the decode form; a window bounds the 64-key tiles that a row walks."""
+    def chunk(self, n_kv_heads: int, head_dim: int, window=None, keep_first: int = 0, one_row: bool = False):
+        """(chunk, most chunks of a row) of the decode form; a window bounds the 64-key tiles that a row walks. `one_row`:
+        a page row is key and value."""
         max_len = self.max_len
         if window:
             max_len = min(max_len, (-(-int(keep_first or 0) // 64) + -(-int(window) // 64) + 1) * 64)
-        key = (n_kv_heads, head_dim, max_len)
+        key = (n_kv_heads, head_dim, max_len, one_row)
         if key not in self._chunking:
-            self._chunking[key] = decode_chunking(self.n_decode, n_kv_heads, max_len, head_dim)
+            self._chunking[key] = decode_chunking(self.n_decode, n_kv_heads, max_len, head_dim, one_row=one_row)
         return self._chunking[key]
 
 
@@ -464,12 +465,15 @@ def sm_count() -> int:
     return _sms[dev]
 
 
-def decode_chunking(n_rows: int, n_kv_heads: int, max_len: int, head_dim: int = 128, sms: int | None = None):
+def decode_chunking(n_rows: int, n_kv_heads: int, max_len: int, head_dim: int = 128, sms: int | None = None,
+                    one_row: bool = False):
     """(chunk, n_splits) of the decode attention. chunk 0: every row spreads its own keys evenly over the
     chunks it uses (the kernel repeats this choice per row from the row's own length, never above n_splits).
     n_splits minimises the time on the critical path in units of one 64-key tile: rounds of CTAs the GPU needs
     (a CTA holds three stages of a key and a value tile in shared memory) times (tiles per chunk + about three
-    tiles' worth of fixed work per CTA); at most 32 and at most one chunk per tile of the longest row."""
+    tiles' worth of fixed work per CTA); at most 32 and at most one chunk per tile of the longest row. A tile of rows that
+    are key and value at once (`one_row`) takes half the time, so the fixed parts count double (8 rows of 1,055 keys, 4 key
+    heads: 4 chunks as clusters 10.7 us, 9 through memory 11.8)."""
     if sms is None:
         sms = sm_count()
     tiles = max(1, -(-max_len // 64))
@@ -479,13 +483,14 @@ def decode_chunking(n_rows: int, n_kv_heads: int, max_len: int, head_dim: int = 
         return -(-tiles // n) * 64, n
     slots = _decode_slots(head_dim, sms)
     pairs = max(1, n_rows * n_kv_heads)
+    fixed, through_memory = (6, 26) if one_row else (3, 10)
     best, best_cost = 1, None
     for n in range(1, min(32, tiles) + 1):
         rounds = -(-pairs * n // slots)
         # the merge: none for one chunk, through distributed shared memory where a row's chunks run as a cluster,
         # through global memory and a last arriver else (measured: about a tile's time more, growing with the chunks)
-        merge = 0 if n == 1 else 2 if _merge_as_cluster(pairs, n, slots) else 10 + n // 2
-        cost = rounds * (-(-tiles // n) + 3) * 8 + merge
+        merge = 0 if n == 1 else 2 if _merge_as_cluster(pairs, n, slots) else through_memory + n // 2
+        cost = rounds * (-(-tiles // n) + fixed) * 8 + merge
         if best_cost is None or cost < best_cost:
             best, best_cost = n, cost
     return 0, best
@@ -651,7 +656,8 @@ def attention(qkv, out, cache, step, plan, n_heads, n_kv_heads, head_dim, scale,
                                   cache.tables, row0, nrows, n, n_heads, n_kv_heads, head_dim, scale, window, err,
                                   **options)
         if plan.n_decode:
-            chunk, n_splits = plan.chunk(n_kv_heads, head_dim, window, options.get("keep_first", 0))
+            chunk, n_splits = plan.chunk(n_kv_heads, head_dim, window, options.get("keep_first", 0),
+                                         options.get("key_scale") is not None)
             attention_decode(qkv, qkv.stride(0), out, cache.k, cache.v, step.positions, step.seq_of_row,
                              cache.tables, plan.decode_rows, plan.n_decode, n_heads, n_kv_heads, head_dim, scale,
                              window, chunk, n_splits, err, **options)

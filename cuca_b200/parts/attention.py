@@ -253,7 +253,7 @@ class PagedAttention(Mixer):
             # attention and the gate are one launch
             parts = ops.gemm_partial(h, self.w_qkv, self.rt.err)
             attn = self.rt.empty(rows, nh * d)
-            chunk, n_splits = plan.chunk(nkv, d, self.window, self.keep_first)
+            chunk, n_splits = plan.chunk(nkv, d, self.window, self.keep_first, self.one_row)
             ops.attention_decode_fused_unit(parts, self.b_qkv, v_col, g_col if self.gated else None, self.eps, self.q_mul,
                                             attn, cache, step, rows, nh, nkv, d, scale, self.window, chunk, n_splits,
                                             self.rt.err, **options)
