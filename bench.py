@@ -391,7 +391,7 @@ def design_table(args) -> int:
             for gi, grp in enumerate(core.groups):
                 seen = mean_ctx if grp.window is None else min(mean_ctx, grp.window + grp.keep_first)
                 vd = grp.head_dim if grp.v_head_dim is None else grp.v_head_dim
-                per_request += seen * len(grp.cache_ids) * grp.n_kv_heads * (grp.head_dim + vd) * 2
+                per_request += seen * len(grp.cache_ids) * grp.n_kv_heads * ((grp.head_dim + vd) * 2 + (4 if grp.key_scale else 0))
             per_request += 2 * core.cache.state_bytes_per_request()
             step_bytes = core.model.weight_bytes() + B * per_request
             ms_step = ms / steps
